@@ -398,6 +398,62 @@ int b200attn_stack_rows(b200attn_stack st, int* n_active_out, int* h_row_slots);
  * cuda_engine.cu:327-352): the captured graph when it was captured for n_rows, eager launches otherwise. */
 int b200attn_stack_step(b200attn_stack st, int n_rows, b200attn_stream stream);
 
+/* ------------------------------------------------------------------------------------------------
+ * Stacks built from layer descriptions.
+ * The same handle, caches, continuous batching and captured decode step as above, for models whose layers are given as a
+ * list: every layer is x += norm1(mixer(x)), then (with a feed-forward) x += norm2(ff(x)), RMS norms with plain weights on
+ * the sublayers' outputs; logits = embedding . norm(x) * logit_scale.  None of this has a counterpart in the reference.
+ *
+ * Mixers: B200ATTN_MIXER_MLSTM, a matrix memory with exponential gates (state per sequence and head: [dim][vdim], [dim],
+ * one running maximum, fp32); B200ATTN_MIXER_LATENT, attention with keys and values up-projected from a cached latent of
+ * kv_rank values and one rotated key part shared by all heads, over a sliding window.  A latent layer with kv_from >= 0
+ * reads the cache of that earlier layer.
+ * Feed-forward: down(gelu_tanh(gate x) * up x).
+ * ---------------------------------------------------------------------------------------------- */
+typedef enum { B200ATTN_DTYPE_BF16 = 0, B200ATTN_DTYPE_F32 = 1 } b200attn_dtype;
+typedef enum { B200ATTN_MIXER_MLSTM = 1, B200ATTN_MIXER_LATENT = 2 } b200attn_mixer;
+
+typedef struct {
+    int width, vocab_size;
+    int max_seqs;          /* sequences resident on this GPU                                              */
+    int max_seq_len;       /* tokens per sequence                                                         */
+    int num_pages;         /* cache pages of 64 tokens; 0 = max_seq_len for every sequence.  With fewer pages the stack serves
+                              continuous batching only                                                    */
+    int max_pass_rows;     /* tokens per prefill pass (bounds the working buffers); longer prompts run in several passes */
+    int dtype;             /* b200attn_dtype of weights, activations and cached latents                   */
+    double norm_eps, embed_scale, logit_scale;
+} b200attn_model_config;
+
+typedef struct {
+    int mixer;             /* b200attn_mixer                                                              */
+    int heads, dim, vdim;  /* query / key size per head (latent: its unrotated part), value size per head  */
+    double gate_cap;       /* mLSTM: soft cap of the gate pre-activations                                  */
+    int kv_rank, rot_dim;  /* latent attention                                                             */
+    int window;            /* a position sees itself and the window - 1 positions before it; 0 = all       */
+    int kv_from;           /* index of the layer whose latents this one reads, -1 = its own                */
+    double rot_base, scale;/* rotation base, score factor                                                  */
+    int ff;                /* feed-forward size, 0 = no feed-forward                                       */
+} b200attn_layer_desc;
+
+/* Builds the stack: caches, state, working buffers, zeroed weights.  No reference counterpart. */
+int b200attn_stack_create_layers(const b200attn_model_config* cfg, const b200attn_layer_desc* layers, int num_layers, b200attn_stack* out);
+/* Gives one weight by name, host data in bf16 or fp32, row-major [rows, cols] (vectors: rows values, cols = 1).  Names:
+ * "embed", "final.norm", and per layer i "l<i>.norm1", ".norm2", ".mlp.{gate,up,down}", ".mix.{q,k,v,g,o,norm,i,i.b,f,f.b}"
+ * (mLSTM) or ".mix.{q,dkv,dkv.norm,uk,uv,o}" (latent).  A wrong name or shape is refused.  No reference counterpart. */
+int b200attn_stack_set_tensor(b200attn_stack st, const char* name, const void* h_data, int dtype, long long rows, long long cols);
+/* Admits a sequence without running a prompt (continuous batching): takes a slot and a row, reserves pages for
+ * reserve_tokens (may be 0: they are reserved as the sequence grows), clears its state.  No reference counterpart. */
+int b200attn_stack_open(b200attn_stack st, int reserve_tokens, int* row_out, b200attn_stream stream);
+/* Runs the next n_tokens tokens (device int32) of the sequence in `row` behind what it already holds: one token through the
+ * decode kernels, more through the prefill kernels.  Logits of the places h_want (ascending, < n_tokens) go to d_logits
+ * fp32 [n_want, vocab]; with d_next the greedy token behind the last of these tokens is stored there.  No reference counterpart. */
+int b200attn_stack_extend(b200attn_stack st, int row, const int* d_tokens, int n_tokens, const int* h_want, int n_want, float* d_logits,
+                          int* d_next, b200attn_stream stream);
+/* The residual stream of the last pass's rows (fp32 [rows, width]; rows = 0: none), for checks of single layers:
+ * stop_after >= 0 makes the following passes end behind that many layers, -1 runs all again, -2 changes nothing.
+ * No reference counterpart. */
+int b200attn_stack_residual(b200attn_stack st, int rows, float* d_out, int stop_after, b200attn_stream stream);
+
 /* Number of kernels this library launched on behalf of the calling thread since the last call
  * with reset != 0 (graph replays count the nodes of the captured step).  No reference counterpart. */
 long long b200attn_launch_count(int reset);

@@ -99,7 +99,7 @@ class StackBackend:
         self.torch = torch
         self.stack = stack
         self.ops = ops_module
-        self.n_rows = stack.cfg.max_seqs
+        self.n_rows = stack.max_seqs
         self.captured = False
 
     def begin_batching(self) -> None:
@@ -124,3 +124,14 @@ class StackBackend:
 
     def read_tokens(self, n_active: int):
         return self.stack.get_tokens(self.n_rows)[:n_active].cpu().tolist()
+
+
+def generate(stack, prompts, max_new_tokens: int, eos: int | None = None) -> list[list[int]]:
+    """Greedy continuations of prompts (sequences of token ids) through the batcher and the captured decode step, in the
+    order of the prompts.  Call it on a non-default stream (the step is captured)."""
+    import torch
+    from . import ops
+    cb = ContinuousBatcher(StackBackend(stack, ops), stack.max_seqs)
+    for i, p in enumerate(prompts):
+        cb.submit(Request(i, torch.tensor(list(p), dtype=torch.int32, device="cuda"), max_new_tokens, eos))
+    return [r.tokens for r in sorted(cb.run(), key=lambda r: r.rid)]

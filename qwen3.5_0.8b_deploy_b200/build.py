@@ -17,7 +17,8 @@ CSRC = os.path.join(HERE, "csrc")
 OUT = os.path.join(HERE, "libb200attn.so")
 OBJ = os.path.join(HERE, "build")
 SOURCES = ["gemm.cu", "kv_cache.cu", "fa_decode.cu", "fa_prefill.cu", "fa_ops.cu", "la_kernels.cu", "la_chunk.cu",
-           "la_ops.cu", "stack.cu", "fa_decode_static.cu", "gemm_tc.cu"]
+           "la_ops.cu", "stack.cu", "fa_decode_static.cu", "gemm_tc.cu",
+           "block_model.cu", "block_kernels.cu", "mlstm.cu", "mlstm_chunk.cu", "latent.cu", "latent_decode.cu", "latent_prefill.cu"]
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "-Xcompiler", "-fPIC",
          "--expt-relaxed-constexpr", "-Xptxas", "-v"]
@@ -48,16 +49,26 @@ def _compile(src: str, force: bool, verbose: bool) -> str:
     return obj
 
 
-def build(force: bool = False, verbose: bool = False) -> str:
+def build_library(force: bool = False, verbose: bool = False) -> str:
+    """libb200attn.so alone: all that running a model needs."""
     os.makedirs(OBJ, exist_ok=True)
     srcs = [s for s in SOURCES if os.path.exists(os.path.join(CSRC, s))]
-    with cf.ThreadPoolExecutor(max_workers=min(8, len(srcs))) as ex:
+    if (not force and os.path.exists(OUT) and os.path.getmtime(OUT) >= _newest_header()
+            and all(os.path.getmtime(OUT) >= os.path.getmtime(os.path.join(CSRC, s)) for s in srcs)):
+        return OUT
+    with cf.ThreadPoolExecutor(max_workers=min(max(8, os.cpu_count() or 1), len(srcs))) as ex:
         objs = list(ex.map(lambda s: _compile(s, force, verbose), srcs))
-    if force or not os.path.exists(OUT) or any(os.path.getmtime(o) > os.path.getmtime(OUT) for o in objs):
-        cmd = [NVCC, "-shared", "-o", OUT, *objs, "-lcublas", "-Xlinker", "-rpath,/usr/local/cuda/lib64"]
-        p = subprocess.run(cmd, capture_output=True, text=True)
-        if p.returncode != 0:
-            raise RuntimeError(f"link failed:\n{p.stderr[-4000:]}")
+    part = f"{OUT}.{os.getpid()}"          # linked beside its place, then moved: a reader never sees half a library
+    cmd = [NVCC, "-shared", "-o", part, *objs, "-lcublas", "-Xlinker", "-rpath,/usr/local/cuda/lib64"]
+    p = subprocess.run(cmd, capture_output=True, text=True)
+    if p.returncode != 0:
+        raise RuntimeError(f"link failed:\n{p.stderr[-4000:]}")
+    os.replace(part, OUT)
+    return OUT
+
+
+def build(force: bool = False, verbose: bool = False) -> str:
+    build_library(force, verbose)
     build_compat(force)
     return OUT
 

@@ -142,6 +142,15 @@ inline int ceil_div(int a, int b) { return (a + b - 1) / b; }
 // Y = alpha * X W^T + beta * Y; ld_out > 0 gives the row pitch of Y (elements) when it is a column block of a wider matrix.
 int gemm_xwT(cudaStream_t stream, const void* X, bool x_fp16, const void* W, bool w_fp16, void* Y,
              bool y_fp16, int rows, int out, int in, float beta = 0.f, float alpha = 1.f, int ld_out = 0);
+// The same product with named element types (accumulation fp32; fp32 inputs in full fp32 math): X has row pitch ldx, Y row pitch ldy.
+enum ElemType { ELEM_F16 = 0, ELEM_BF16, ELEM_F32 };
+inline size_t elem_bytes(ElemType t) { return t == ELEM_F32 ? 4 : 2; }
+int gemm_typed(cudaStream_t stream, const void* X, int ldx, const void* W, void* Y, int ldy, ElemType in_type, ElemType out_type, int rows,
+               int out, int in, float beta = 0.f, float alpha = 1.f);
+// One product per head, strided batched: Y_h[rows, out] = X_h[rows, in] W_h^T with W_h [out, in], or X_h W_h with W_h [in, out]
+// when w_in_major.  Head h starts x_stride / y_stride elements behind head h - 1 inside a row; the W_h lie back to back.
+int gemm_heads(cudaStream_t stream, const void* X, int ldx, int x_stride, const void* W, bool w_in_major, void* Y, int ldy, int y_stride,
+               ElemType in_type, ElemType out_type, int rows, int out, int in, int heads);
 int cublas_init();   // creates the current device's handle and its capture-safe workspace (call outside stream capture)
 
 // ---- small elementwise helpers (elementwise.cu) ----------------------------------------------------
@@ -162,6 +171,14 @@ struct KvView {            // what kernels need, passed by value
     const int* capacity;     // [max_seqs] tokens reserved
     int* error;              // device error word
     int num_pages, max_seqs, max_pages_per_seq, is_fp16;
+};
+struct LatentView {        // one layer of a latent pool
+    void* rows;              // [page][page_tokens][pitch]
+    int pitch;               // elements per row
+    const int* block_table;  // [max_seqs][max_pages_per_seq]
+    const int* capacity;     // [max_seqs] tokens reserved
+    int* error;              // device error word
+    int num_pages, max_seqs, max_pages_per_seq;
 };
 
 }  // namespace b200
@@ -186,6 +203,11 @@ struct b200attn_kv_pool_s {
     std::vector<int> free_pages;
     std::vector<int> h_block_table;
     std::vector<int> h_capacity;
+    // Latent pools (kv_pool_create_latent): one row per token and layer instead of K and V heads; d_k holds
+    // [layer][page][page_tokens][pitch] rows, every layer with a pitch of its own.
+    std::vector<size_t> latent_offset;   // bytes from d_k to the layer's first page
+    std::vector<int> latent_pitch;       // elements per row
+    b200::LatentView latent_view(int layer) const;
     b200::KvView view() const;
     int sync_lens();                // refresh h_lens from the device when dirty
     size_t layer_stride_elems() const {
@@ -238,6 +260,9 @@ struct b200attn_la_state_s {
     b200attn_la_state_config cfg{};
     float* d_recurrent = nullptr;   // [layer][slot][16][128][128]
     float* d_conv = nullptr;        // [layer][slot][3][6144]
+    // Pools of per-layer state blocks (state_pool_create_blocks): d_recurrent is [layer][slot][block_floats[layer]], no conv part.
+    std::vector<size_t> block_floats;   // floats per (layer, slot); empty in a DeltaNet pool
+    std::vector<size_t> block_offset;   // floats from d_recurrent to the layer's first block
     size_t rec_stride_slot() const { return (size_t)cfg.num_heads * cfg.key_dim * cfg.value_dim; }
     size_t conv_stride_slot() const {
         return (size_t)(cfg.conv_kernel - 1) * cfg.num_heads * (2 * cfg.key_dim + cfg.value_dim);

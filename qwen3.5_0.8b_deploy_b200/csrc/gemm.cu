@@ -137,22 +137,45 @@ static int cublas_for_current_device(cublasHandle_t* out) {
 
 int cublas_init() { return cublas_for_current_device(nullptr); }
 
-int gemm_xwT(cudaStream_t stream, const void* X, bool x_fp16, const void* W, bool w_fp16, void* Y, bool y_fp16, int rows,
-             int out, int in, float beta, float alpha, int ld_out) {
-    if (rows <= 0) return 0;
+static cudaDataType cuda_type(ElemType t) { return t == ELEM_F16 ? CUDA_R_16F : t == ELEM_BF16 ? CUDA_R_16BF : CUDA_R_32F; }
+
+int gemm_typed(cudaStream_t stream, const void* X, int ldx, const void* W, void* Y, int ldy, ElemType in_type, ElemType out_type, int rows,
+               int out, int in, float beta, float alpha) {
+    if (rows <= 0 || out <= 0) return 0;
     cublasHandle_t handle = nullptr;
     B2_TRY(cublas_for_current_device(&handle));
-    if (x_fp16 != w_fp16) B2_FAIL(B200ATTN_ERR_INVALID, "gemm: activation and weight types must match");
     cublasStatus_t st = cublasSetStream(handle, stream);
     if (st != CUBLAS_STATUS_SUCCESS) B2_FAIL(B200ATTN_ERR_CUDA, "cublasSetStream failed with status %d", (int)st);
-    const cudaDataType_t in_t = x_fp16 ? CUDA_R_16F : CUDA_R_32F;
-    const cudaDataType_t out_t = y_fp16 ? CUDA_R_16F : CUDA_R_32F;
     // Row-major Y[rows,out] = X[rows,in] W[out,in]^T  ==  column-major Y^T[out,rows] = W^T(op T) X^T.
-    st = cublasGemmEx(handle, CUBLAS_OP_T, CUBLAS_OP_N, out, rows, in, &alpha, W, in_t, in, X, in_t, in, &beta, Y, out_t,
-                      ld_out > 0 ? ld_out : out, CUBLAS_COMPUTE_32F, CUBLAS_GEMM_DEFAULT);
+    st = cublasGemmEx(handle, CUBLAS_OP_T, CUBLAS_OP_N, out, rows, in, &alpha, W, cuda_type(in_type), in, X, cuda_type(in_type), ldx, &beta, Y,
+                      cuda_type(out_type), ldy, CUBLAS_COMPUTE_32F, CUBLAS_GEMM_DEFAULT);
     if (st != CUBLAS_STATUS_SUCCESS) B2_FAIL(B200ATTN_ERR_CUDA, "cublasGemmEx(%d,%d,%d) failed with status %d", rows, out, in, (int)st);
     count_launch();
     return 0;
+}
+
+int gemm_heads(cudaStream_t stream, const void* X, int ldx, int x_stride, const void* W, bool w_in_major, void* Y, int ldy, int y_stride,
+               ElemType in_type, ElemType out_type, int rows, int out, int in, int heads) {
+    if (rows <= 0) return 0;
+    cublasHandle_t handle = nullptr;
+    B2_TRY(cublas_for_current_device(&handle));
+    cublasStatus_t st = cublasSetStream(handle, stream);
+    if (st != CUBLAS_STATUS_SUCCESS) B2_FAIL(B200ATTN_ERR_CUDA, "cublasSetStream failed with status %d", (int)st);
+    const float one = 1.f, zero = 0.f;
+    st = cublasGemmStridedBatchedEx(handle, w_in_major ? CUBLAS_OP_N : CUBLAS_OP_T, CUBLAS_OP_N, out, rows, in, &one, W, cuda_type(in_type),
+                                    w_in_major ? out : in, (long long)out * in, X, cuda_type(in_type), ldx, x_stride, &zero, Y,
+                                    cuda_type(out_type), ldy, y_stride, heads, CUBLAS_COMPUTE_32F, CUBLAS_GEMM_DEFAULT);
+    if (st != CUBLAS_STATUS_SUCCESS)
+        B2_FAIL(B200ATTN_ERR_CUDA, "cublasGemmStridedBatchedEx(%d,%d,%d x %d) failed with status %d", rows, out, in, heads, (int)st);
+    count_launch();
+    return 0;
+}
+
+int gemm_xwT(cudaStream_t stream, const void* X, bool x_fp16, const void* W, bool w_fp16, void* Y, bool y_fp16, int rows,
+             int out, int in, float beta, float alpha, int ld_out) {
+    if (x_fp16 != w_fp16) B2_FAIL(B200ATTN_ERR_INVALID, "gemm: activation and weight types must match");
+    return gemm_typed(stream, X, in, W, Y, ld_out > 0 ? ld_out : out, x_fp16 ? ELEM_F16 : ELEM_F32, y_fp16 ? ELEM_F16 : ELEM_F32, rows, out,
+                      in, beta, alpha);
 }
 
 // x -> hi = fp16(x), lo = fp16((x - hi) * 2^11): hi + lo * 2^-11 carries about 22 significant bits of x.

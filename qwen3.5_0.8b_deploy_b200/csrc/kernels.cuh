@@ -29,6 +29,9 @@ void build_append_tiles(const std::vector<int>& base, const int* h_counts, int n
 int pool_prepare_append(b200attn_kv_pool p, int layer, const int* h_slots, const int* h_counts, int n_seqs,
                         std::vector<int>& base, int* total_rows);
 int ensure_meta(int** d_meta, int* cap, int need);
+// A pool of the same pages, tables and lengths whose layers hold one row of row_pitch[layer] elements per token.
+int kv_pool_create_latent(const std::vector<int>& row_pitch, ElemType elem, int num_pages, int max_seqs, int max_pages_per_seq,
+                          b200attn_kv_pool* out);
 
 // ---- decode attention (fa_decode.cu) -----------------------------------------------------------------------
 constexpr int kFaDecodeParts = 16;      // partial slots per (sequence, kv head) pair the decode kernel may use; sizes part_o / part_ml
@@ -57,6 +60,8 @@ struct LaSeqMeta {  // per sequence, device array
     int row0;
     int count;
 };
+// A state pool whose layers hold blocks of block_floats[layer] floats per slot (zeroed by b200attn_la_state_clear).
+int state_pool_create_blocks(const std::vector<size_t>& block_floats, int max_seqs, b200attn_la_state* out);
 int launch_la_conv_seq(const float* mixed, const int* d_row_seq, const LaSeqMeta* d_seqs, const float* conv_layer,
                        size_t conv_stride, const float* conv_w, const float* a_log, const float* dt_bias, int rows,
                        float* q, float* k, __half* qh, __half* kh, float* v, __half* vh, float* g, float* beta, cudaStream_t s);

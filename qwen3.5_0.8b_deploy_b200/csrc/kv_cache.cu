@@ -423,6 +423,61 @@ int b200attn_kv_pool_s::sync_lens() {
     return 0;
 }
 
+b200::LatentView b200attn_kv_pool_s::latent_view(int layer) const {
+    return LatentView{static_cast<char*>(d_k) + latent_offset[layer], latent_pitch[layer], d_block_table, d_capacity, d_error,
+                      cfg.num_pages, cfg.max_seqs, cfg.max_pages_per_seq};
+}
+
+// Page tables, lengths, capacities and the status word, common to all kinds of pools; the data is allocated by the caller.
+static int pool_init_bookkeeping(b200attn_kv_pool p) {
+    const auto* cfg = &p->cfg;
+    const size_t bt = (size_t)cfg->max_seqs * cfg->max_pages_per_seq, nl = (size_t)cfg->num_layers * cfg->max_seqs;
+    B2_CUDA(cudaMalloc(&p->d_block_table, bt * sizeof(int)));
+    B2_CUDA(cudaMemset(p->d_block_table, 0, bt * sizeof(int)));
+    B2_CUDA(cudaMalloc(&p->d_lens, nl * sizeof(int)));
+    B2_CUDA(cudaMemset(p->d_lens, 0, nl * sizeof(int)));
+    B2_CUDA(cudaMalloc(&p->d_capacity, cfg->max_seqs * sizeof(int)));
+    B2_CUDA(cudaMemset(p->d_capacity, 0, cfg->max_seqs * sizeof(int)));
+    B2_CUDA(cudaMalloc(&p->d_error, sizeof(int)));
+    B2_CUDA(cudaMemset(p->d_error, 0, sizeof(int)));
+    p->h_lens.assign(nl, 0);
+    p->seq_pages.assign(cfg->max_seqs, {});
+    p->slot_used.assign(cfg->max_seqs, 0);
+    p->h_block_table.assign(bt, 0);
+    p->h_capacity.assign(cfg->max_seqs, 0);
+    p->free_pages.reserve(cfg->num_pages);
+    for (int i = cfg->num_pages - 1; i >= 0; --i) p->free_pages.push_back(i);   // pop_back hands out page 0 first
+    return 0;
+}
+
+namespace b200 {
+int kv_pool_create_latent(const std::vector<int>& row_pitch, ElemType elem, int num_pages, int max_seqs, int max_pages_per_seq,
+                          b200attn_kv_pool* out) {
+    B2_CHECK_ARG(out && !row_pitch.empty() && num_pages > 0 && max_seqs > 0 && max_pages_per_seq > 0, "latent pool: bad argument");
+    auto* p = new (std::nothrow) b200attn_kv_pool_s();
+    if (!p) B2_FAIL(B200ATTN_ERR_NOMEM, "latent pool: host allocation failed");
+    p->cfg = b200attn_kv_config{(int)row_pitch.size(), 1, 0, kPageTokens, num_pages, max_seqs, max_pages_per_seq, B200ATTN_KV_FP16};
+    p->elem_bytes = (int)elem_bytes(elem);
+    p->latent_pitch = row_pitch;
+    size_t total = 0;
+    for (int pitch : row_pitch) {
+        p->latent_offset.push_back(total);
+        total += ((size_t)num_pages * kPageTokens * pitch * p->elem_bytes + 1023) / 1024 * 1024;
+    }
+    cudaError_t e = cudaMalloc(&p->d_k, total);
+    if (e == cudaSuccess) e = cudaMemset(p->d_k, 0, total);
+    int st = 0;
+    if (e != cudaSuccess) {
+        set_error("latent pool: %s", cudaGetErrorString(e));
+        st = e == cudaErrorMemoryAllocation ? B200ATTN_ERR_NOMEM : B200ATTN_ERR_CUDA;
+    }
+    if (st == 0) st = pool_init_bookkeeping(p);
+    if (st != 0) { b200attn_kv_pool_destroy(p); return st; }
+    *out = p;
+    return 0;
+}
+}  // namespace b200
+
 extern "C" int b200attn_kv_pool_create(const b200attn_kv_config* cfg, b200attn_kv_pool* out) {
     B2_CHECK_ARG(cfg && out, "kv_pool_create: null argument");
     B2_CHECK_ARG(cfg->num_layers > 0 && cfg->num_pages > 0 && cfg->max_seqs > 0 && cfg->max_pages_per_seq > 0,
@@ -450,24 +505,8 @@ extern "C" int b200attn_kv_pool_create(const b200attn_kv_config* cfg, b200attn_k
         POOL_CUDA(cudaMemset(p->d_ks, 0, nscale * sizeof(float)));
         POOL_CUDA(cudaMemset(p->d_vs, 0, nscale * sizeof(float)));
     }
-    const size_t bt = (size_t)cfg->max_seqs * cfg->max_pages_per_seq;
-    POOL_CUDA(cudaMalloc(&p->d_block_table, bt * sizeof(int)));
-    POOL_CUDA(cudaMemset(p->d_block_table, 0, bt * sizeof(int)));
-    POOL_CUDA(cudaMalloc(&p->d_lens, (size_t)cfg->num_layers * cfg->max_seqs * sizeof(int)));
-    POOL_CUDA(cudaMemset(p->d_lens, 0, (size_t)cfg->num_layers * cfg->max_seqs * sizeof(int)));
-    POOL_CUDA(cudaMalloc(&p->d_capacity, cfg->max_seqs * sizeof(int)));
-    POOL_CUDA(cudaMemset(p->d_capacity, 0, cfg->max_seqs * sizeof(int)));
-    POOL_CUDA(cudaMalloc(&p->d_error, sizeof(int)));
-    POOL_CUDA(cudaMemset(p->d_error, 0, sizeof(int)));
 #undef POOL_CUDA
-    (void)st;
-    p->h_lens.assign((size_t)cfg->num_layers * cfg->max_seqs, 0);
-    p->seq_pages.assign(cfg->max_seqs, {});
-    p->slot_used.assign(cfg->max_seqs, 0);
-    p->h_block_table.assign(bt, 0);
-    p->h_capacity.assign(cfg->max_seqs, 0);
-    p->free_pages.reserve(cfg->num_pages);
-    for (int i = cfg->num_pages - 1; i >= 0; --i) p->free_pages.push_back(i);   // pop_back hands out page 0 first
+    if ((st = pool_init_bookkeeping(p)) != 0) return fail(st);
     *out = p;
     return 0;
 }
@@ -656,6 +695,7 @@ int pool_prepare_append(b200attn_kv_pool p, int layer, const int* h_slots, const
 extern "C" int b200attn_kv_append(b200attn_kv_pool p, int layer, const int* h_slots, const int* h_counts, int n_seqs,
                                   const float* d_k, const float* d_v, b200attn_stream stream) {
     B2_CHECK_ARG(d_k && d_v, "kv_append: null K/V");
+    B2_CHECK_ARG(!p || p->latent_pitch.empty(), "kv_append: the pool holds latent rows");
     std::vector<int> base;
     int rows = 0;
     B2_TRY(pool_prepare_append(p, layer, h_slots, h_counts, n_seqs, base, &rows));

@@ -178,6 +178,15 @@ extern "C" int b200attn_la_state_clear(b200attn_la_state st, int slot, b200attn_
     B2_CHECK_ARG(st, "la_state_clear: null state");
     B2_CHECK_ARG(slot < st->cfg.max_seqs, "la_state_clear: slot out of range");
     cudaStream_t s = as_stream(stream);
+    if (!st->block_floats.empty()) {
+        for (size_t l = 0; l < st->block_floats.size(); ++l) {
+            float* layer = st->d_recurrent + st->block_offset[l];
+            const size_t n = st->block_floats[l];
+            if (slot < 0) B2_CUDA(cudaMemsetAsync(layer, 0, n * st->cfg.max_seqs * 4, s));
+            else B2_CUDA(cudaMemsetAsync(layer + n * slot, 0, n * 4, s));
+        }
+        return 0;
+    }
     if (slot < 0) {
         B2_CUDA(cudaMemsetAsync(st->d_recurrent, 0, (size_t)st->cfg.num_layers * st->cfg.max_seqs * st->rec_stride_slot() * 4, s));
         B2_CUDA(cudaMemsetAsync(st->d_conv, 0, (size_t)st->cfg.num_layers * st->cfg.max_seqs * st->conv_stride_slot() * 4, s));
@@ -191,8 +200,30 @@ extern "C" int b200attn_la_state_clear(b200attn_la_state st, int slot, b200attn_
     return 0;
 }
 
+namespace b200 {
+int state_pool_create_blocks(const std::vector<size_t>& block_floats, int max_seqs, b200attn_la_state* out) {
+    B2_CHECK_ARG(out && !block_floats.empty() && max_seqs > 0, "state pool: bad argument");
+    auto* st = new (std::nothrow) b200attn_la_state_s();
+    if (!st) B2_FAIL(B200ATTN_ERR_NOMEM, "state pool: host allocation failed");
+    st->cfg.num_layers = (int)block_floats.size();
+    st->cfg.max_seqs = max_seqs;
+    st->block_floats = block_floats;
+    size_t total = 0;
+    for (size_t n : block_floats) { st->block_offset.push_back(total); total += n * max_seqs; }
+    cudaError_t e = cudaMalloc(&st->d_recurrent, total * 4);
+    if (e == cudaSuccess) e = cudaMemset(st->d_recurrent, 0, total * 4);
+    if (e != cudaSuccess) {
+        set_error("state pool: %s", cudaGetErrorString(e));
+        b200attn_la_state_destroy(st);
+        return e == cudaErrorMemoryAllocation ? B200ATTN_ERR_NOMEM : B200ATTN_ERR_CUDA;
+    }
+    *out = st;
+    return 0;
+}
+}  // namespace b200
+
 static int la_state_index(b200attn_la_state st, int layer, int slot, size_t* idx) {
-    B2_CHECK_ARG(st, "la_state: null state");
+    B2_CHECK_ARG(st && st->block_floats.empty(), "la_state: null state or a pool of another kind");
     B2_CHECK_ARG(layer >= 0 && layer < st->cfg.num_layers, "la_state: layer %d out of range", layer);
     B2_CHECK_ARG(slot >= 0 && slot < st->cfg.max_seqs, "la_state: slot %d out of range", slot);
     *idx = (size_t)layer * st->cfg.max_seqs + slot;

@@ -1,0 +1,217 @@
+// Matrix memory with exponential gating (mLSTM): the token-serial recurrence and the head norm.
+//
+// Per head, with log input gate i = cap tanh(. / cap) and log forget gate f = logsigmoid(cap tanh(. / cap)):
+//     m_t = max(f_t + m_{t-1}, i_t),   S_t = e^{f_t + m_{t-1} - m_t} S_{t-1} + e^{i_t - m_t} k_t v_t^T,   n_t likewise with k_t
+//     o_t = S_t^T q_t / (max(|n_t . q_t|, e^{-m_t}) + 1e-6)
+// and all of S, n, m start at zero.  The state of a head lies in tiles of up to 128 value columns, each with a copy of n
+// and m of its own, so that CTAs that share a head never read what another one writes.
+#include "block_model.cuh"
+#include "elem.cuh"
+#include "mlstm.cuh"
+#include "ptx_utils.cuh"
+
+#include <algorithm>
+
+namespace b200 {
+
+// grid (sequences, heads, tiles), block 256.  Lane l of every warp owns value columns 4l .. 4l+3 of the tile, warp w the
+// key rows w, w + 8, ...; with dim <= 8 NR a thread's part of the state stays in registers over the whole run of tokens
+// (decode: one token), else it is streamed through for every token.  Decode loads its state ahead of the wait on the
+// preceding kernel: the state was last written one step earlier.
+template <int NR, typename T, bool kFuseNorm>
+__global__ void __launch_bounds__(256)
+mlstm_step_kernel(const MlstmStepArgs a, unsigned long long* stamp) {
+    extern __shared__ float sm[];
+    const MlstmShape& sh = a.sh;
+    const int D = sh.dim, h = blockIdx.y, tile = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    float* s_q = sm;
+    const int D4 = (D + 3) / 4 * 4;
+    float* s_k = s_q + D4;
+    float* s_n = s_k + D4;
+    float* s_red = s_n + D4;                // [8][128]
+    float* s_x = s_red + 8 * kMlstmTile;    // 16 words
+    int slot, row0 = blockIdx.x, count = 1;
+    if (a.seqs) {
+        pdl_wait();
+        const LaSeqMeta q = a.seqs[blockIdx.x];
+        slot = q.slot; row0 = q.row0; count = q.count;
+    } else {
+        slot = a.d_slots[blockIdx.x];
+    }
+    if (slot < 0 || slot >= a.max_seqs || count <= 0) { pdl_enter(); return; }
+    float* S = a.state + (size_t)slot * sh.state_floats() + (size_t)(h * sh.n_vt + tile) * sh.tile_floats();
+    float* gn = S + (size_t)D * sh.vt;
+    float* gm = gn + D4;
+    const int c0 = 4 * lane, vcol = tile * kMlstmTile + c0;       // column in the tile / in the head
+    const bool act = c0 < sh.vt;
+    const bool resident = D <= 8 * NR;
+    float4 st[NR];
+    if (resident && act) {
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {
+            const int d = warp + 8 * i;
+            if (d < D) st[i] = __ldcs(reinterpret_cast<const float4*>(S + (size_t)d * sh.vt + c0));
+        }
+    }
+    float m = *gm;
+    for (int d = tid; d < D; d += 256) s_n[d] = gn[d];
+    pdl_enter();
+    stamp_begin(stamp);
+    const float q_scale = 1.0f / sqrtf((float)D);
+    const int V = sh.vdim;
+    for (int t = 0; t < count; ++t) {
+        const size_t row = row0 + t;
+        const float* pr = a.proj + row * sh.pitch();
+        for (int d = tid; d < D; d += 256) {
+            s_q[d] = pr[sh.off_q() + h * sh.dp + d] * q_scale;
+            s_k[d] = pr[sh.off_k() + h * sh.dp + d];
+        }
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (act && vcol < sh.vp) v = *reinterpret_cast<const float4*>(pr + sh.off_v() + h * sh.vp + vcol);
+        const float ig = mlstm_log_input(pr[sh.off_i() + h] + a.bias[h], sh.gate_cap);
+        const float fg = mlstm_log_forget(pr[sh.off_f() + h] + a.bias[sh.heads + h], sh.gate_cap);
+        const float m_new = fmaxf(fg + m, ig);
+        const float keep = expf(fg + m - m_new), add = expf(ig - m_new);
+        m = m_new;
+        __syncthreads();
+        float4 num = make_float4(0.f, 0.f, 0.f, 0.f);
+        auto row_step = [&](float4 x, int d) -> float4 {
+            const float kd = add * s_k[d], qd = s_q[d];
+            x.x = keep * x.x + kd * v.x; x.y = keep * x.y + kd * v.y;
+            x.z = keep * x.z + kd * v.z; x.w = keep * x.w + kd * v.w;
+            num.x += x.x * qd; num.y += x.y * qd; num.z += x.z * qd; num.w += x.w * qd;
+            return x;
+        };
+        if (act) {
+            if (resident) {
+#pragma unroll
+                for (int i = 0; i < NR; ++i) {
+                    const int d = warp + 8 * i;
+                    if (d < D) st[i] = row_step(st[i], d);
+                }
+            } else {
+                for (int d = warp; d < D; d += 8) {
+                    float4* p = reinterpret_cast<float4*>(S + (size_t)d * sh.vt + c0);
+                    *p = row_step(*p, d);
+                }
+            }
+        }
+        float nq = 0.f;
+        for (int d = tid; d < D; d += 256) {
+            const float nn = keep * s_n[d] + add * s_k[d];
+            s_n[d] = nn;
+            nq += nn * s_q[d];
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) nq += __shfl_xor_sync(0xffffffffu, nq, o);
+        if (lane == 0) s_x[warp] = nq;
+        *reinterpret_cast<float4*>(s_red + warp * kMlstmTile + c0) = num;
+        __syncthreads();
+        float o = 0.f;
+        const int vc = tile * kMlstmTile + tid;
+        const bool mine = tid < kMlstmTile && tid < sh.vt && vc < V;
+        if (tid < kMlstmTile) {
+            nq = ((s_x[0] + s_x[1]) + (s_x[2] + s_x[3])) + ((s_x[4] + s_x[5]) + (s_x[6] + s_x[7]));
+            if (mine) {
+#pragma unroll
+                for (int w = 0; w < 8; ++w) o += s_red[w * kMlstmTile + tid];
+                o /= fmaxf(fabsf(nq), expf(-m)) + 1e-6f;
+            }
+        }
+        if constexpr (kFuseNorm) {
+            if (tid < kMlstmTile) {
+                float ss = o * o;
+#pragma unroll
+                for (int k = 16; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
+                if (lane == 0) s_x[8 + warp] = ss;
+            }
+            __syncthreads();
+            if (mine) {
+                const float rms = sqrtf(((s_x[8] + s_x[9]) + (s_x[10] + s_x[11])) / (float)V + sh.eps);
+                const float g = pr[sh.off_g() + h * sh.vp + vc];
+                const float r = o / rms * a.norm_w[h * sh.vp + vc] / (1.0f + expf(-g));
+                static_cast<T*>(a.gated)[row * (sh.heads * sh.vp) + h * sh.vp + vc] = from_f32<T>(r);
+            }
+        } else {
+            if (mine) a.core[row * (sh.heads * sh.vp) + h * sh.vp + vc] = o;
+        }
+        if (t + 1 < count) __syncthreads();       // s_q, s_k and the partial sums are free again
+    }
+    if (resident && act) {
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {
+            const int d = warp + 8 * i;
+            if (d < D) __stcs(reinterpret_cast<float4*>(S + (size_t)d * sh.vt + c0), st[i]);
+        }
+    }
+    for (int d = tid; d < D; d += 256) gn[d] = s_n[d];
+    if (tid == 0) *gm = m;
+    if (stamp) { __syncthreads(); stamp_end(stamp); }
+}
+
+int launch_mlstm_step(ElemType t, const MlstmStepArgs& a, int n, cudaStream_t s) {
+    const MlstmShape& sh = a.sh;
+    const size_t smem = (3 * (size_t)round_up(sh.dim, 4) + 8 * kMlstmTile + 16) * 4;
+    const dim3 grid(n, sh.heads, sh.n_vt);
+    unsigned long long* stamp = a.seqs ? nullptr : prof_stamp_slot(PROF_LA_DECODE);
+    dispatch_elem(t, [&](auto tag) {
+        using T = decltype(tag);
+        auto go = [&](auto kernel) { launch_pdl(kernel, grid, dim3(256), smem, s, a, stamp); };
+        auto pick = [&](auto fuse) {
+            constexpr bool kFuse = decltype(fuse)::value;
+            if (sh.dim <= 32) go(mlstm_step_kernel<4, T, kFuse>);
+            else if (sh.dim <= 64) go(mlstm_step_kernel<8, T, kFuse>);
+            else if (sh.dim <= 128) go(mlstm_step_kernel<16, T, kFuse>);
+            else go(mlstm_step_kernel<32, T, kFuse>);
+        };
+        if (sh.n_vt == 1) pick(std::true_type{}); else pick(std::false_type{});
+    });
+    B2_LAUNCH_CHECK();
+    return 0;
+}
+
+// One warp per (row, head): the head's outputs over their root mean square, times the norm weight, times sigmoid(g).
+template <typename T, typename G>
+__global__ void __launch_bounds__(256)
+mlstm_head_norm_kernel(const float* __restrict__ core, const G* __restrict__ g, int g_pitch, int off_g, const float* __restrict__ norm_w,
+                       float eps, int heads, int vdim, int vp, int units, T* __restrict__ out) {
+    pdl_enter();
+    const int u = (blockIdx.x * 256 + threadIdx.x) >> 5, lane = threadIdx.x & 31;
+    if (u >= units) return;
+    const int row = u / heads, h = u % heads;
+    const float* c = core + (size_t)row * heads * vp + h * vp;
+    const G* gr = g + (size_t)row * g_pitch + off_g + h * vp;
+    T* o = out + (size_t)row * heads * vp + h * vp;
+    float ss = 0.f;
+    for (int v = 4 * lane; v < vp; v += 128) {                   // columns from vdim on are zero
+        const float4 x = load4(c + v);
+        ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+    }
+#pragma unroll
+    for (int k = 16; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
+    const float rms = sqrtf(ss / (float)vdim + eps);
+    for (int v = 4 * lane; v < vp; v += 128) {
+        const float4 x = load4(c + v), w = load4(norm_w + h * vp + v), z = load4(gr + v);
+        store4(o + v, make_float4(x.x / rms * w.x / (1.0f + expf(-z.x)), x.y / rms * w.y / (1.0f + expf(-z.y)),
+                                  x.z / rms * w.z / (1.0f + expf(-z.z)), x.w / rms * w.w / (1.0f + expf(-z.w))));
+    }
+}
+
+int launch_mlstm_head_norm(ElemType t, const MlstmShape& sh, const float* core, const void* g, bool g_f32, int g_pitch, const float* norm_w,
+                           int rows, void* gated, cudaStream_t s) {
+    const int units = rows * sh.heads;
+    const dim3 grid(ceil_div(units, 8));
+    dispatch_elem(t, [&](auto tag) {
+        using T = decltype(tag);
+        if (g_f32)
+            launch_pdl(mlstm_head_norm_kernel<T, float>, grid, dim3(256), 0, s, core, (const float*)g, g_pitch, sh.off_g(), norm_w, sh.eps, sh.heads,
+                       sh.vdim, sh.vp, units, (T*)gated);
+        else
+            launch_pdl(mlstm_head_norm_kernel<T, T>, grid, dim3(256), 0, s, core, (const T*)g, g_pitch, sh.off_g(), norm_w, sh.eps, sh.heads, sh.vdim,
+                       sh.vp, units, (T*)gated);
+    });
+    B2_LAUNCH_CHECK();
+    return 0;
+}
+
+}  // namespace b200

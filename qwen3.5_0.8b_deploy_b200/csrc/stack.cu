@@ -7,54 +7,12 @@
 // per-layer weights, prefill over token batches, a decode step for the whole batch, reset_cache, and a
 // graph-captured step (there: prefill, :391-479; here: decode with device-resident lengths and tokens).
 // The residual stream is fp32; GEMM operands are fp16 with fp32 accumulation (cuBLAS).
-#include "kernels.cuh"
+#include "stack.cuh"
 #include "ptx_utils.cuh"
 
 #include <algorithm>
 #include <new>
 #include <vector>
-
-struct b200attn_stack_s {
-    b200attn_stack_config cfg{};
-    int n_fa = 0, n_la = 0;
-    std::vector<int> layer_kind;      // 1 = full attention, 0 = DeltaNet
-    std::vector<int> layer_sub;       // index inside the kv pool / state pool
-    std::vector<b200attn_fa> fa;
-    std::vector<b200attn_la> la;
-    std::vector<float*> d_in_norm, d_post_norm;
-    std::vector<__half*> d_wgu, d_wdown;   // [2*inter, hidden], [hidden, inter]
-    std::vector<char> layer_ready;
-    __half* d_embed = nullptr;  // [vocab, hidden]
-    float* d_final_norm = nullptr;
-    bool embed_ready = false;
-    b200attn_kv_pool pool = nullptr;
-    b200attn_la_state state = nullptr;
-    b200::Scratch op_scratch;
-    int max_rows = 0;
-    float* d_h = nullptr;              // [max_rows, hidden] residual stream
-    __half* d_xb = nullptr;     // [max_rows, hidden]
-    __half* d_gu = nullptr;     // [max_rows, 2*inter]
-    __half* d_act = nullptr;    // [max_rows, inter]
-    float* d_last = nullptr;           // [max_seqs, hidden]
-    float* d_logits = nullptr;         // [max_seqs, vocab]
-    int* d_tokens = nullptr;           // [max_seqs] decode token buffer (in place)
-    int* d_slots = nullptr;            // [max_seqs] identity slots
-    __half* d_xh = nullptr;            // [128, hidden] fp16 copy of the residual stream in the fused decode step
-    float* d_rowsq = nullptr;          // [128][kRowsqParts] partial sums of squares of the residual rows
-    unsigned long long* d_packed = nullptr;   // [128] running argmax words of the LM head
-    int* d_error = nullptr;            // device status word of the stack's own tcgen05 GEMMs
-    int* d_last_idx = nullptr;         // [max_seqs] row of every sequence's last prompt token inside a prefill pass
-    // Continuous batching: row r of a decode step is bound to slot row_slot[r] (its KV pages and DeltaNet state), -1 =
-    // inactive.  Empty in the plain mode, where row r is slot r.
-    bool batching = false;
-    std::vector<int> row_slot;
-    std::vector<int> free_slots;
-    int n_active = 0;
-    cudaGraph_t graph = nullptr;
-    cudaGraphExec_t graph_exec = nullptr;
-    int graph_nseqs = 0;
-    long long graph_nodes = 0;
-};
 
 namespace b200 {
 
@@ -213,6 +171,12 @@ argmax_kernel(const float* __restrict__ logits, int vocab, int* __restrict__ out
     }
 }
 
+int launch_argmax_rows(const float* logits, int rows, int vocab, int* out, cudaStream_t s) {
+    argmax_kernel<<<rows, 1024, 0, s>>>(logits, vocab, out);
+    B2_LAUNCH_CHECK();
+    return 0;
+}
+
 // Embedding ~ N(0, std) from a counter-based hash (Box-Muller), written as fp16.
 __global__ void init_normal_fp16_kernel(__half* __restrict__ out, size_t n, uint64_t seed, float std_dev) {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -290,7 +254,7 @@ extern "C" int b200attn_stack_destroy(b200attn_stack st) {
     cudaFree(st->op_scratch.base);
     cudaFree(st->d_h); cudaFree(st->d_xb); cudaFree(st->d_gu); cudaFree(st->d_act); cudaFree(st->d_last);
     cudaFree(st->d_logits); cudaFree(st->d_tokens); cudaFree(st->d_slots);
-    cudaFree(st->d_xh); cudaFree(st->d_rowsq); cudaFree(st->d_packed); cudaFree(st->d_error); cudaFree(st->d_last_idx);
+    cudaFree(st->d_xh); cudaFree(st->d_rowsq); cudaFree(st->d_packed); cudaFree(st->d_error); cudaFree(st->d_last_idx); cudaFree(st->d_want);
     delete st;
     return 0;
 }
@@ -375,6 +339,7 @@ extern "C" int b200attn_stack_create(const b200attn_stack_config* cfg, b200attn_
 
 extern "C" int b200attn_stack_set_layer_weights(b200attn_stack st, int layer, const b200attn_layer_weights* w) {
     B2_CHECK_ARG(st && w, "stack_set_layer_weights: null argument");
+    B2_CHECK_ARG(!st->blocks, "stack_set_layer_weights: a layer-described stack takes its weights by name");
     B2_CHECK_ARG(layer >= 0 && layer < st->cfg.num_layers, "stack_set_layer_weights: layer %d out of range", layer);
     B2_CHECK_ARG(w->input_norm && w->post_norm && w->ffn_gate && w->ffn_up && w->ffn_down, "stack_set_layer_weights: null weight pointer");
     const bool q8 = st->cfg.int8_weights != 0;
@@ -455,6 +420,7 @@ extern "C" int b200attn_stack_set_layer_weights(b200attn_stack st, int layer, co
 
 extern "C" int b200attn_stack_set_embedding(b200attn_stack st, const float* h_embed, const float* h_final_norm) {
     B2_CHECK_ARG(st && h_embed && h_final_norm, "stack_set_embedding: null argument");
+    B2_CHECK_ARG(!st->blocks, "stack_set_embedding: a layer-described stack takes its weights by name");
     cudaFree(st->d_embed); cudaFree(st->d_final_norm);
     st->d_embed = nullptr; st->d_final_norm = nullptr; st->embed_ready = false;
     B2_TRY(upload_matrix(h_embed, st->cfg.vocab_size, kHidden, st->cfg.int8_weights != 0, &st->d_embed));
@@ -465,6 +431,7 @@ extern "C" int b200attn_stack_set_embedding(b200attn_stack st, const float* h_em
 
 extern "C" int b200attn_stack_init_embedding_random(b200attn_stack st, uint64_t seed, float std_dev, const float* h_final_norm) {
     B2_CHECK_ARG(st && h_final_norm, "stack_init_embedding_random: null argument");
+    B2_CHECK_ARG(!st->blocks, "stack_init_embedding_random: a layer-described stack takes its weights by name");
     cudaFree(st->d_embed); cudaFree(st->d_final_norm);
     st->d_embed = nullptr; st->d_final_norm = nullptr; st->embed_ready = false;
     const size_t n = (size_t)st->cfg.vocab_size * kHidden;
@@ -483,6 +450,11 @@ extern "C" int b200attn_stack_device_status(b200attn_stack st, int* code_out) {
     int c = 0;
     if (st->pool) { B2_TRY(b200attn_kv_device_status(st->pool, &c)); if (c && !*code_out) *code_out = c; }
     for (auto l : st->la) { B2_TRY(b200attn_la_device_status(l, &c)); if (c && !*code_out) *code_out = c; }
+    if (st->blocks) {
+        B2_TRY(block_model_status(*st->blocks, &c));
+        if (c && !*code_out) *code_out = c;
+        return 0;
+    }
     B2_CUDA(cudaDeviceSynchronize());
     B2_CUDA(cudaMemcpy(&c, st->d_error, sizeof(int), cudaMemcpyDeviceToHost));
     if (c) { B2_CUDA(cudaMemset(st->d_error, 0, sizeof(int))); if (!*code_out) *code_out = c; }
@@ -496,7 +468,7 @@ extern "C" int b200attn_stack_reset(b200attn_stack st, b200attn_stream stream) {
     if (st->batching) {     // back to the plain mode: row r is slot r, every slot holds pages for max_seq_len tokens
         st->batching = false;
         st->n_active = 0;
-        if (st->pool)
+        if (st->pool && !(st->blocks && st->blocks->cfg.num_pages > 0))
             for (int i = 0; i < st->cfg.max_seqs; ++i) B2_TRY(b200attn_kv_seq_reserve(st->pool, i, st->cfg.max_seq_len));
         iota_kernel<<<ceil_div(st->cfg.max_seqs, 128), 128, 0, b200::as_stream(stream)>>>(st->d_slots, st->cfg.max_seqs);
         B2_LAUNCH_CHECK();
@@ -508,6 +480,7 @@ namespace b200 {
 
 static int stack_ready(b200attn_stack st) {
     B2_CHECK_ARG(st, "stack: null handle");
+    if (st->blocks) return block_model_ready(*st->blocks);
     if (!st->embed_ready) B2_FAIL(B200ATTN_ERR_NOT_READY, "stack: embedding not set");
     for (int i = 0; i < st->cfg.num_layers; ++i)
         if (!st->layer_ready[i]) B2_FAIL(B200ATTN_ERR_NOT_READY, "stack: weights of layer %d not set", i);
@@ -564,6 +537,11 @@ static int stack_layers(b200attn_stack st, int rows, const int* h_slots, const i
 
 // Final norm of the selected rows, tied LM head, greedy argmax.
 static int stack_head(b200attn_stack st, int n_seqs, const int* d_row_index, int* d_next, float* d_hidden_out, cudaStream_t s) {
+    if (st->blocks) {
+        if (d_hidden_out) B2_FAIL(B200ATTN_ERR_UNSUPPORTED, "a layer-described stack does not return hidden states");
+        B2_TRY(block_logits(*st->blocks, n_seqs, d_row_index, st->d_logits, s));
+        return launch_argmax_rows(st->d_logits, n_seqs, st->cfg.vocab_size, d_next, s);
+    }
     launch_pdl(rmsnorm_kernel, dim3(n_seqs), dim3(256), 0, s, st->d_h, d_row_index, st->d_final_norm, st->cfg.rms_eps, n_seqs, st->d_xb,
                d_hidden_out);
     B2_LAUNCH_CHECK();
@@ -577,15 +555,33 @@ static int stack_head(b200attn_stack st, int n_seqs, const int* d_row_index, int
     return 0;
 }
 
-static int stack_decode_step(b200attn_stack st, int n_seqs, const int* d_tokens_in, int* d_tokens_out, cudaStream_t s) {
+// The layers of one decode step over n rows whose slots are d_slots[0 .. n).
+static int stack_decode_layers(b200attn_stack st, int n_seqs, const int* d_tokens_in, const int* d_slots, cudaStream_t s) {
+    if (st->blocks) {
+        if (st->pool) st->pool->lens_dirty = true;
+        return block_decode_rows(*st->blocks, n_seqs, d_tokens_in, d_slots, s);
+    }
     if (n_seqs <= 128 && gemm_tc_enabled())
         launch_pdl(embed_gather_fused_kernel, dim3(n_seqs), dim3(256), 0, s, d_tokens_in, st->d_embed, st->cfg.vocab_size, st->d_h, st->d_xh,
                    st->d_rowsq);
     else
         launch_pdl(embed_gather_kernel, dim3(n_seqs), dim3(256), 0, s, d_tokens_in, st->d_embed, st->cfg.vocab_size, st->d_h);
     B2_LAUNCH_CHECK();
-    B2_TRY(stack_layers(st, n_seqs, nullptr, nullptr, n_seqs, st->d_slots, true, s));
+    if (st->pool) st->pool->lens_dirty = true;
+    return stack_layers(st, n_seqs, nullptr, nullptr, n_seqs, d_slots, true, s);
+}
+
+static int stack_decode_step(b200attn_stack st, int n_seqs, const int* d_tokens_in, int* d_tokens_out, cudaStream_t s) {
+    B2_TRY(stack_decode_layers(st, n_seqs, d_tokens_in, st->d_slots, s));
     return stack_head(st, n_seqs, nullptr, d_tokens_out, nullptr, s);
+}
+
+// Logits (fp32 [n, vocab]) of selected rows of the last pass.
+static int stack_logits(b200attn_stack st, int n, const int* d_row_index, float* d_logits, cudaStream_t s) {
+    if (st->blocks) return block_logits(*st->blocks, n, d_row_index, d_logits, s);
+    launch_pdl(rmsnorm_kernel, dim3(n), dim3(256), 0, s, st->d_h, d_row_index, st->d_final_norm, st->cfg.rms_eps, n, st->d_xb, nullptr);
+    B2_LAUNCH_CHECK();
+    return gemm_xwT(s, st->d_xb, true, st->d_embed, true, d_logits, false, n, st->cfg.vocab_size, kHidden);
 }
 
 }  // namespace b200
@@ -595,16 +591,33 @@ namespace b200 {
 // i goes to d_next[i].
 static int stack_prefill_slots(b200attn_stack st, const int* h_slots, int n_seqs, int prompt_len, const int* d_tokens, int* d_next,
                                float* d_hidden_out, cudaStream_t s) {
+    if (st->blocks && prompt_len > st->max_rows) {     // one sequence at a time, in portions of a pass
+        for (int i = 0; i < n_seqs; ++i)
+            for (int t = 0, n; t < prompt_len; t += n) {
+                n = std::min(st->max_rows, prompt_len - t);
+                B2_TRY(block_prefill_rows(*st->blocks, 1, h_slots + i, &n, d_tokens + (size_t)i * prompt_len + t, s));
+                if (t + n < prompt_len) continue;
+                last_row_index_kernel<<<1, 128, 0, s>>>(st->d_last_idx, 1, n);
+                count_launch();
+                B2_TRY(stack_head(st, 1, st->d_last_idx, d_next + i, d_hidden_out, s));
+            }
+        return 0;
+    }
     const int chunk = std::max(1, std::min(n_seqs, st->max_rows / prompt_len));
     std::vector<int> counts(chunk, prompt_len);
     int* d_idx = st->d_last_idx;   // row of each sequence's last token inside the pass
     int rc = 0;
-    for (int s0 = 0; s0 < n_seqs && rc == 0; s0 += chunk) {
-        const int n = std::min(chunk, n_seqs - s0);
+    for (int s0 = 0, n = 0; s0 < n_seqs && rc == 0; s0 += n) {
+        n = std::min(chunk, n_seqs - s0);
         const int rows = n * prompt_len;
-        launch_pdl(embed_gather_kernel, dim3(rows), dim3(256), 0, s, d_tokens + (size_t)s0 * prompt_len, st->d_embed, st->cfg.vocab_size, st->d_h);
-        count_launch();
-        rc = stack_layers(st, rows, h_slots + s0, counts.data(), n, nullptr, false, s);
+        if (st->blocks) {
+            B2_TRY(block_pass_sequences(*st->blocks, n, h_slots + s0, counts.data(), &n));
+            rc = block_prefill_rows(*st->blocks, n, h_slots + s0, counts.data(), d_tokens + (size_t)s0 * prompt_len, s);
+        } else {
+            launch_pdl(embed_gather_kernel, dim3(rows), dim3(256), 0, s, d_tokens + (size_t)s0 * prompt_len, st->d_embed, st->cfg.vocab_size, st->d_h);
+            count_launch();
+            rc = stack_layers(st, rows, h_slots + s0, counts.data(), n, nullptr, false, s);
+        }
         if (rc != 0) break;
         last_row_index_kernel<<<ceil_div(n, 128), 128, 0, s>>>(d_idx, n, prompt_len);
         count_launch();
@@ -624,6 +637,38 @@ extern "C" int b200attn_stack_prefill(b200attn_stack st, int n_seqs, int prompt_
     std::vector<int> slots(n_seqs);
     for (int i = 0; i < n_seqs; ++i) slots[i] = i;
     return stack_prefill_slots(st, slots.data(), n_seqs, prompt_len, d_tokens, d_next, d_hidden_out, as_stream(stream));
+}
+
+extern "C" int b200attn_stack_create_layers(const b200attn_model_config* cfg, const b200attn_layer_desc* layers, int num_layers,
+                                            b200attn_stack* out) {
+    B2_CHECK_ARG(cfg && layers && out, "stack_create_layers: null argument");
+    B2_CHECK_ARG(num_layers > 0 && cfg->width > 0 && cfg->vocab_size > 0 && cfg->max_seqs > 0 && cfg->max_seq_len > 0 && cfg->num_pages >= 0 &&
+                     cfg->max_pass_rows >= 0, "stack_create_layers: bad sizes");
+    refresh_runtime_flags();
+    auto* st = new (std::nothrow) b200attn_stack_s();
+    if (!st) B2_FAIL(B200ATTN_ERR_NOMEM, "stack_create_layers: host allocation failed");
+    st->cfg.num_layers = num_layers;
+    st->cfg.vocab_size = cfg->vocab_size;
+    st->cfg.max_seqs = cfg->max_seqs;
+    st->cfg.max_seq_len = cfg->max_seq_len;
+    int rc = block_model_create(cfg, layers, num_layers, st);
+    auto alloc = [&](auto** p, size_t bytes) {
+        if (rc == 0 && cudaMalloc(p, bytes) != cudaSuccess) { set_error("stack_create_layers: out of device memory"); rc = B200ATTN_ERR_NOMEM; }
+        if (rc == 0) cudaMemset(*p, 0, bytes);
+    };
+    const size_t n = cfg->max_seqs;
+    alloc(&st->d_logits, n * cfg->vocab_size * 4);
+    alloc(&st->d_tokens, n * 4);
+    alloc(&st->d_slots, n * 4);
+    alloc(&st->d_last_idx, n * 4);
+    if (rc == 0) {
+        iota_kernel<<<ceil_div(cfg->max_seqs, 128), 128>>>(st->d_slots, cfg->max_seqs);
+        count_launch();
+        if (cudaDeviceSynchronize() != cudaSuccess) { set_error("stack_create_layers: %s", cudaGetErrorString(cudaGetLastError())); rc = B200ATTN_ERR_CUDA; }
+    }
+    if (rc != 0) { b200attn_stack_destroy(st); return rc; }
+    *out = st;
+    return 0;
 }
 
 // ---- continuous batching ---------------------------------------------------------------------------------------------
@@ -651,6 +696,25 @@ extern "C" int b200attn_stack_begin_batching(b200attn_stack st, b200attn_stream 
     return push_row_slots(st, s);
 }
 
+extern "C" int b200attn_stack_open(b200attn_stack st, int reserve_tokens, int* row_out, b200attn_stream stream) {
+    B2_TRY(stack_ready(st));
+    B2_CHECK_ARG(row_out, "stack_open: null argument");
+    if (!st->batching) B2_FAIL(B200ATTN_ERR_INVALID, "stack_open: call b200attn_stack_begin_batching first");
+    B2_CHECK_ARG(reserve_tokens >= 0 && reserve_tokens <= st->cfg.max_seq_len, "stack_open: %d tokens outside [0, max_seq_len %d]", reserve_tokens,
+                 st->cfg.max_seq_len);
+    if (st->free_slots.empty()) B2_FAIL(B200ATTN_ERR_NOMEM, "stack_open: all %d rows are in use", st->cfg.max_seqs);
+    const int slot = st->free_slots.back();
+    if (st->pool) B2_TRY(b200attn_kv_seq_reserve(st->pool, slot, reserve_tokens));      // NOMEM when the page pool cannot hold it: nothing changed
+    st->free_slots.pop_back();
+    if (st->state) B2_TRY(b200attn_la_state_clear(st->state, slot, stream));
+    const int row = st->n_active;
+    st->row_slot[row] = slot;
+    st->n_active = row + 1;
+    B2_TRY(push_row_slots(st, as_stream(stream)));
+    *row_out = row;
+    return 0;
+}
+
 extern "C" int b200attn_stack_admit(b200attn_stack st, const int* d_prompt, int prompt_len, int reserve_tokens, int* row_out,
                                     b200attn_stream stream) {
     B2_TRY(stack_ready(st));
@@ -658,19 +722,58 @@ extern "C" int b200attn_stack_admit(b200attn_stack st, const int* d_prompt, int 
     if (!st->batching) B2_FAIL(B200ATTN_ERR_INVALID, "stack_admit: call b200attn_stack_begin_batching first");
     B2_CHECK_ARG(prompt_len > 0 && prompt_len <= reserve_tokens && reserve_tokens <= st->cfg.max_seq_len,
                  "stack_admit: need 0 < prompt_len (%d) <= reserve_tokens (%d) <= max_seq_len (%d)", prompt_len, reserve_tokens, st->cfg.max_seq_len);
-    B2_CHECK_ARG(prompt_len <= st->max_rows, "stack_admit: prompt of %d tokens exceeds the prefill scratch (%d rows)", prompt_len, st->max_rows);
-    if (st->free_slots.empty()) B2_FAIL(B200ATTN_ERR_NOMEM, "stack_admit: all %d rows are in use", st->cfg.max_seqs);
-    cudaStream_t s = as_stream(stream);
-    const int slot = st->free_slots.back();
-    if (st->pool) B2_TRY(b200attn_kv_seq_reserve(st->pool, slot, reserve_tokens));      // NOMEM when the page pool cannot hold it: nothing changed
-    st->free_slots.pop_back();
-    if (st->state) B2_TRY(b200attn_la_state_clear(st->state, slot, stream));
-    const int row = st->n_active;
-    B2_TRY(stack_prefill_slots(st, &slot, 1, prompt_len, d_prompt, st->d_tokens + row, nullptr, s));
-    st->row_slot[row] = slot;
-    st->n_active = row + 1;
-    B2_TRY(push_row_slots(st, s));
+    B2_CHECK_ARG(st->blocks || prompt_len <= st->max_rows, "stack_admit: prompt of %d tokens exceeds the prefill scratch (%d rows)", prompt_len,
+                 st->max_rows);
+    int row = -1;
+    B2_TRY(b200attn_stack_open(st, reserve_tokens, &row, stream));
+    B2_TRY(stack_prefill_slots(st, &st->row_slot[row], 1, prompt_len, d_prompt, st->d_tokens + row, nullptr, as_stream(stream)));
     *row_out = row;
+    return 0;
+}
+
+extern "C" int b200attn_stack_extend(b200attn_stack st, int row, const int* d_tokens, int n_tokens, const int* h_want, int n_want,
+                                     float* d_logits, int* d_next, b200attn_stream stream) {
+    B2_TRY(stack_ready(st));
+    B2_CHECK_ARG(d_tokens && n_tokens > 0 && n_want >= 0 && (n_want == 0 || (h_want && d_logits)), "stack_extend: bad argument");
+    if (!st->batching) B2_FAIL(B200ATTN_ERR_INVALID, "stack_extend: call b200attn_stack_begin_batching first");
+    B2_CHECK_ARG(row >= 0 && row < st->n_active, "stack_extend: row %d is not active (%d active rows)", row, st->n_active);
+    for (int i = 0; i < n_want; ++i)
+        B2_CHECK_ARG(h_want[i] >= (i ? h_want[i - 1] : 0) && h_want[i] < n_tokens, "stack_extend: wanted places must ascend within the tokens");
+    cudaStream_t s = as_stream(stream);
+    const int slot = st->row_slot[row];
+    if (st->pool) {
+        int len = 0;
+        B2_TRY(b200attn_kv_seq_len(st->pool, 0, slot, &len));
+        B2_CHECK_ARG(len + n_tokens <= st->cfg.max_seq_len, "stack_extend: %d + %d tokens exceed max_seq_len %d", len, n_tokens, st->cfg.max_seq_len);
+        B2_TRY(b200attn_kv_seq_reserve(st->pool, slot, len + n_tokens));
+    }
+    B2_TRY(ensure_meta(&st->d_want, &st->want_cap, n_want + 1));
+    size_t out = 0;
+    for (int t = 0, w = 0, n; t < n_tokens; t += n) {
+        n = std::min(st->max_rows, n_tokens - t);
+        if (n == 1) {
+            B2_TRY(stack_decode_layers(st, 1, d_tokens + t, st->d_slots + row, s));
+        } else if (st->blocks) {
+            B2_TRY(block_prefill_rows(*st->blocks, 1, &slot, &n, d_tokens + t, s));
+        } else {
+            launch_pdl(embed_gather_kernel, dim3(n), dim3(256), 0, s, d_tokens + t, st->d_embed, st->cfg.vocab_size, st->d_h);
+            B2_LAUNCH_CHECK();
+            B2_TRY(stack_layers(st, n, &slot, &n, 1, nullptr, false, s));
+        }
+        std::vector<int> idx;
+        for (; w < n_want && h_want[w] < t + n; ++w) idx.push_back(h_want[w] - t);
+        if (t + n == n_tokens && d_next) idx.push_back(n - 1);
+        const int have = (int)idx.size() - ((t + n == n_tokens && d_next) ? 1 : 0);
+        if (idx.empty()) continue;
+        B2_CUDA(cudaMemcpyAsync(st->d_want, idx.data(), idx.size() * sizeof(int), cudaMemcpyHostToDevice, s));
+        for (int r0 = 0, k; r0 < have; r0 += k) {                  // the head's row buffer holds max_rows rows
+            k = std::min(st->max_rows, have - r0);
+            B2_TRY(stack_logits(st, k, st->d_want + r0, d_logits + out * st->cfg.vocab_size, s));
+            out += k;
+        }
+        if ((int)idx.size() > have) B2_TRY(stack_head(st, 1, st->d_want + have, d_next, nullptr, s));
+        B2_CUDA(cudaStreamSynchronize(s));                          // the index vector goes out of scope
+    }
     return 0;
 }
 

@@ -20,6 +20,8 @@ LIB_PATH = os.path.join(_HERE, "libb200attn.so")
 OK, ERR_INVALID, ERR_CUDA, ERR_NOMEM, ERR_NOT_READY, ERR_UNSUPPORTED, ERR_DEVICE = 0, -1, -2, -3, -4, -5, -6
 PROJ_FP32, PROJ_FP16 = 0, 1
 KV_INT8, KV_FP16 = 0, 1
+DTYPE_BF16, DTYPE_F32 = 0, 1
+MIXER_MLSTM, MIXER_LATENT = 1, 2
 
 # Every symbol include/b200attn.h declares (tests check the library exports exactly these).
 ABI_SYMBOLS = [
@@ -39,6 +41,7 @@ ABI_SYMBOLS = [
     "b200attn_stack_prefill", "b200attn_stack_decode", "b200attn_decode_graph_capture",
     "b200attn_decode_graph_launch", "b200attn_stack_set_tokens", "b200attn_stack_get_tokens",
     "b200attn_stack_begin_batching", "b200attn_stack_admit", "b200attn_stack_retire", "b200attn_stack_rows", "b200attn_stack_step",
+    "b200attn_stack_create_layers", "b200attn_stack_set_tensor", "b200attn_stack_open", "b200attn_stack_extend", "b200attn_stack_residual",
 ]
 
 
@@ -138,6 +141,16 @@ class StackConfig(C.Structure):
                 ("vocab_size", C.c_int), ("max_seqs", C.c_int), ("max_seq_len", C.c_int),
                 ("prefill_chunk_seqs", C.c_int), ("kv_dtype", C.c_int), ("int8_weights", C.c_int),
                 ("rms_eps", C.c_float)]
+
+
+class ModelConfig(C.Structure):
+    _fields_ = [(n, C.c_int) for n in ("width", "vocab_size", "max_seqs", "max_seq_len", "num_pages", "max_pass_rows", "dtype")] + \
+               [(n, C.c_double) for n in ("norm_eps", "embed_scale", "logit_scale")]
+
+
+class LayerDesc(C.Structure):
+    _fields_ = [("mixer", C.c_int), ("heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("gate_cap", C.c_double), ("kv_rank", C.c_int),
+                ("rot_dim", C.c_int), ("window", C.c_int), ("kv_from", C.c_int), ("rot_base", C.c_double), ("scale", C.c_double), ("ff", C.c_int)]
 
 
 class LayerWeights(C.Structure):
@@ -369,38 +382,11 @@ class LinearAttention:
 
 
 # ---- hybrid stack + graph-captured decode -------------------------------------------------------------------------
-class HybridStack:
-    """CudaEngine for the attention-facing part: set_layer_weights, forward_batch_prefill,
-    forward_batch_decode, reset_cache, and the captured decode step."""
+class Stack:
+    """What every stack offers whatever its layers are: batched prefill and decode, the captured decode step, continuous batching."""
 
-    def __init__(self, num_layers=24, intermediate_size=3584, vocab_size=248320, max_seqs=128, max_seq_len=1536,
-                 prefill_chunk_seqs=8, kv_dtype=KV_FP16, int8_weights=True, rms_eps=1e-6):
-        self.cfg = StackConfig(num_layers, 1024, intermediate_size, vocab_size, max_seqs, max_seq_len, prefill_chunk_seqs,
-                               kv_dtype, 1 if int8_weights else 0, rms_eps)
-        self.h = C.c_void_p()
-        _check(_lib.b200attn_stack_create(C.byref(self.cfg), C.byref(self.h)))
-
-    def set_layer_weights(self, layer: int, norms: dict, ffn: dict, fa: dict | None = None, la: dict | None = None) -> None:
-        keep = [_host_f32(norms["input_norm"]), _host_f32(norms["post_norm"]), _host_f32(ffn["gate"]),
-                _host_f32(ffn["up"]), _host_f32(ffn["down"])]
-        fa_s = la_s = None
-        if fa is not None:
-            fa_s, k2 = _fa_weights_struct(fa)
-            keep.append(k2)
-        if la is not None:
-            la_s, k3 = _la_weights_struct(la)
-            keep.append(k3)
-        lw = LayerWeights(*[a.ctypes.data_as(_f32p) for a in keep[:5]],
-                          C.pointer(fa_s) if fa_s is not None else None, C.pointer(la_s) if la_s is not None else None)
-        _check(_lib.b200attn_stack_set_layer_weights(self.h, C.c_int(layer), C.byref(lw)))
-
-    def set_embedding(self, embed: np.ndarray, final_norm: np.ndarray) -> None:
-        e, f = _host_f32(embed), _host_f32(final_norm)
-        _check(_lib.b200attn_stack_set_embedding(self.h, e.ctypes.data_as(_f32p), f.ctypes.data_as(_f32p)))
-
-    def init_embedding_random(self, seed: int, std: float, final_norm: np.ndarray) -> None:
-        f = _host_f32(final_norm)
-        _check(_lib.b200attn_stack_init_embedding_random(self.h, C.c_uint64(seed), C.c_float(std), f.ctypes.data_as(_f32p)))
+    vocab_size: int
+    max_seqs: int
 
     def device_status(self) -> int:
         code = C.c_int(0)
@@ -451,9 +437,25 @@ class HybridStack:
 
     def rows(self) -> tuple[int, list[int]]:
         n = C.c_int(0)
-        slots = (C.c_int * self.cfg.max_seqs)()
+        slots = (C.c_int * self.max_seqs)()
         _check(_lib.b200attn_stack_rows(self.h, C.byref(n), slots))
         return n.value, list(slots)
+
+    def open(self, reserve_tokens: int = 0) -> int:
+        """Admit one sequence without a prompt; returns its row."""
+        row = C.c_int(-1)
+        _check(_lib.b200attn_stack_open(self.h, C.c_int(reserve_tokens), C.byref(row), _stream()))
+        return row.value
+
+    def extend(self, row: int, tokens: torch.Tensor, want=(), want_next: bool = False):
+        """Run the next tokens (int32 device tensor) of the sequence in `row`; returns the logits [len(want), vocab] of the
+        ascending places `want` and, with want_next, the greedy next token as a device tensor."""
+        w = _host_i32(want)
+        logits = torch.empty((len(w), self.vocab_size), dtype=torch.float32, device="cuda")
+        nxt = torch.empty(1, dtype=torch.int32, device="cuda") if want_next else None
+        _check(_lib.b200attn_stack_extend(self.h, C.c_int(row), _dev(tokens), C.c_int(tokens.numel()), w.ctypes.data_as(_i32p), C.c_int(len(w)),
+                                          _dev(logits) if len(w) else C.c_void_p(0), _dev(nxt), _stream()))
+        return (logits, nxt) if want_next else logits
 
     def step(self, n_rows: int) -> None:
         _check(_lib.b200attn_stack_step(self.h, C.c_int(n_rows), _stream()))
@@ -464,6 +466,71 @@ class HybridStack:
                 _lib.b200attn_stack_destroy(self.h)
         except Exception:
             pass
+
+
+class HybridStack(Stack):
+    """CudaEngine for the attention-facing part: set_layer_weights, forward_batch_prefill,
+    forward_batch_decode, reset_cache, and the captured decode step."""
+
+    def __init__(self, num_layers=24, intermediate_size=3584, vocab_size=248320, max_seqs=128, max_seq_len=1536,
+                 prefill_chunk_seqs=8, kv_dtype=KV_FP16, int8_weights=True, rms_eps=1e-6):
+        self.cfg = StackConfig(num_layers, 1024, intermediate_size, vocab_size, max_seqs, max_seq_len, prefill_chunk_seqs,
+                               kv_dtype, 1 if int8_weights else 0, rms_eps)
+        self.vocab_size, self.max_seqs = vocab_size, max_seqs
+        self.h = C.c_void_p()
+        _check(_lib.b200attn_stack_create(C.byref(self.cfg), C.byref(self.h)))
+
+    def set_layer_weights(self, layer: int, norms: dict, ffn: dict, fa: dict | None = None, la: dict | None = None) -> None:
+        keep = [_host_f32(norms["input_norm"]), _host_f32(norms["post_norm"]), _host_f32(ffn["gate"]),
+                _host_f32(ffn["up"]), _host_f32(ffn["down"])]
+        fa_s = la_s = None
+        if fa is not None:
+            fa_s, k2 = _fa_weights_struct(fa)
+            keep.append(k2)
+        if la is not None:
+            la_s, k3 = _la_weights_struct(la)
+            keep.append(k3)
+        lw = LayerWeights(*[a.ctypes.data_as(_f32p) for a in keep[:5]],
+                          C.pointer(fa_s) if fa_s is not None else None, C.pointer(la_s) if la_s is not None else None)
+        _check(_lib.b200attn_stack_set_layer_weights(self.h, C.c_int(layer), C.byref(lw)))
+
+    def set_embedding(self, embed: np.ndarray, final_norm: np.ndarray) -> None:
+        e, f = _host_f32(embed), _host_f32(final_norm)
+        _check(_lib.b200attn_stack_set_embedding(self.h, e.ctypes.data_as(_f32p), f.ctypes.data_as(_f32p)))
+
+    def init_embedding_random(self, seed: int, std: float, final_norm: np.ndarray) -> None:
+        f = _host_f32(final_norm)
+        _check(_lib.b200attn_stack_init_embedding_random(self.h, C.c_uint64(seed), C.c_float(std), f.ctypes.data_as(_f32p)))
+
+
+class LayerStack(Stack):
+    """A stack built from layer descriptions (LayerDesc); weights are given by name."""
+
+    def __init__(self, cfg: ModelConfig, layers: list[LayerDesc]):
+        self.cfg = cfg
+        self.vocab_size, self.max_seqs = cfg.vocab_size, cfg.max_seqs
+        self.h = C.c_void_p()
+        arr = (LayerDesc * len(layers))(*layers)
+        _check(_lib.b200attn_stack_create_layers(C.byref(cfg), arr, C.c_int(len(layers)), C.byref(self.h)))
+
+    def set_tensor(self, name: str, a: np.ndarray) -> None:
+        """`a`: float32, or uint16 holding bf16 bits; one or two dimensions."""
+        a = np.ascontiguousarray(a)
+        if a.dtype != np.uint16:
+            a = np.ascontiguousarray(a, dtype=np.float32)
+        rows, cols = (a.shape[0], 1) if a.ndim == 1 else a.shape
+        _check(_lib.b200attn_stack_set_tensor(self.h, name.encode(), C.c_void_p(a.ctypes.data), C.c_int(DTYPE_BF16 if a.dtype == np.uint16 else DTYPE_F32),
+                                              C.c_longlong(rows), C.c_longlong(cols)))
+
+    def residual(self, rows: int) -> torch.Tensor:
+        """Residual stream of the last pass's rows, fp32 [rows, width]."""
+        out = torch.empty((rows, self.cfg.width), dtype=torch.float32, device="cuda")
+        _check(_lib.b200attn_stack_residual(self.h, C.c_int(rows), _dev(out), C.c_int(-2), _stream()))
+        return out
+
+    def stop_after(self, layers: int) -> None:
+        """The following passes end behind that many layers (-1: all)."""
+        _check(_lib.b200attn_stack_residual(self.h, C.c_int(0), C.c_void_p(0), C.c_int(layers), _stream()))
 
 
 def fa_decode_core_static(q: torch.Tensor, kv: KVCache, layer: int, d_slots: torch.Tensor, out: torch.Tensor) -> None:
