@@ -57,25 +57,30 @@ def mlstm_recurrence(q, k, v, ig, fg, state=None):
     return o, (S, n, m)
 
 
-def mlstm_mixer(h, W, c, eps, state=None):
-    """W: dict of float64 tensors without the layer prefix; c: the layer's sizes."""
+def exact(a):
+    return a
+
+
+def mlstm_mixer(h, W, c, eps, state=None, r=exact):
+    """W: dict of float64 tensors without the layer prefix; c: the layer's sizes; r: applied to what a 16-bit path rounds."""
     T = h.shape[0]
     H, D, V, cap = c["heads"], c["dim"], c["vdim"], c["gate_cap"]
-    q = (h @ W["q"].T).reshape(T, H, D) * D ** -0.5
-    k = (h @ W["k"].T).reshape(T, H, D)
-    v = (h @ W["v"].T).reshape(T, H, V)
+    h = r(h)
+    q = r(h @ W["q"].T).reshape(T, H, D) * D ** -0.5
+    k = r(h @ W["k"].T).reshape(T, H, D)
+    v = r(h @ W["v"].T).reshape(T, H, V)
     ig = cap * np.tanh((h @ W["i"].T + W["i.b"]) / cap)
     fg = log_sigmoid(cap * np.tanh((h @ W["f"].T + W["f.b"]) / cap))
     o, state = mlstm_recurrence(q, k, v, ig, fg, state)
-    o = rms_unit(o, eps).reshape(T, H * V) * W["norm"] * sigmoid(h @ W["g"].T)
-    return o @ W["o"].T, state
+    o = rms_unit(o, eps).reshape(T, H * V) * W["norm"] * sigmoid(r(h @ W["g"].T))
+    return r(o) @ W["o"].T, state
 
 
-def latent_rows(h, W, c, eps, pos):
+def latent_rows(h, W, c, eps, pos, r=exact):
     """The cached rows of a latent-attention layer: normed latent and rotated key part."""
-    y = h @ W["dkv"].T
-    r = c["kv_rank"]
-    return rms_norm(y[:, :r], W["dkv.norm"], eps), rotate_half(y[:, r:], pos, c["rot"]["base"])
+    y = r(h) @ W["dkv"].T
+    n = c["kv_rank"]
+    return r(rms_norm(y[:, :n], W["dkv.norm"], eps)), r(rotate_half(y[:, n:], pos, c["rot"]["base"]))
 
 
 def window_softmax(q, k, v, scale, size, pos0):
@@ -89,24 +94,25 @@ def window_softmax(q, k, v, scale, size, pos0):
     return np.einsum("htn,nhv->thv", p / p.sum(-1, keepdims=True), v)
 
 
-def latent_mixer(h, W, c, eps, lat, pos0):
+def latent_mixer(h, W, c, eps, lat, pos0, r=exact):
     """lat = (latents [N, rank], rotated key parts [N, R]) of positions 0 .. N-1, this call's own included."""
     T = h.shape[0]
     H, D, R, V = c["heads"], c["dim"], c["rot_dim"], c["vdim"]
     pos = pos0 + np.arange(T)
-    q = (h @ W["q"].T).reshape(T, H, D + R)
+    q = r(r(h) @ W["q"].T).reshape(T, H, D + R)
     q = np.concatenate([q[..., :D], rotate_half(q[..., D:], pos, c["rot"]["base"])], -1)
     lc, lr = lat
     N = lc.shape[0]
-    ku = (lc @ W["uk"].T).reshape(N, H, D)
-    vv = (lc @ W["uv"].T).reshape(N, H, V)
+    ku = r(lc @ W["uk"].T).reshape(N, H, D)
+    vv = r(lc @ W["uv"].T).reshape(N, H, V)
     k = np.concatenate([ku, np.broadcast_to(lr[:, None, :], (N, H, R))], -1)
     o = window_softmax(q, k, vv, c["scale"], c["mask"]["size"], pos0)
-    return o.reshape(T, H * V) @ W["o"].T
+    return r(o.reshape(T, H * V)) @ W["o"].T
 
 
-def dense_ff(h, W):
-    return (gelu_tanh(h @ W["gate"].T) * (h @ W["up"].T)) @ W["down"].T
+def dense_ff(h, W, r=exact):
+    h = r(h)
+    return r(gelu_tanh(r(h @ W["gate"].T)) * r(h @ W["up"].T)) @ W["down"].T
 
 
 class PlainModel:
@@ -122,27 +128,27 @@ class PlainModel:
     def start(self):
         return dict(pos=0, layers=[None] * len(self.c["layers"]))
 
-    def forward(self, seq, tokens, trace=None):
-        """Runs `tokens` behind what `seq` has seen; returns logits [T, vocab]."""
+    def forward(self, seq, tokens, trace=None, r=exact):
+        """Runs `tokens` behind what `seq` has seen; returns logits [T, vocab].  `r` may disturb what a 16-bit path rounds."""
         c, eps, p0 = self.c, self.c["norm"]["eps"], seq["pos"]
         x = self.t["embed"][np.asarray(tokens)] * c["embedding"]["scale"]
         pos = p0 + np.arange(len(tokens))
         for i, layer in enumerate(c["layers"]):
             W, mc = self._sub(f"l{i}.mix."), layer["mixer"]
             if layer["type"] == "mlstm":
-                y, seq["layers"][i] = mlstm_mixer(x, W, mc, eps, seq["layers"][i])
+                y, seq["layers"][i] = mlstm_mixer(x, W, mc, eps, seq["layers"][i], r)
             else:
                 src = mc.get("kv_from")
                 if src is None:
                     src = i
-                    new = latent_rows(x, W, mc, eps, pos)
+                    new = latent_rows(x, W, mc, eps, pos, r)
                     old = seq["layers"][i]
                     seq["layers"][i] = new if old is None else tuple(np.concatenate([a, b]) for a, b in zip(old, new))
-                y = latent_mixer(x, W, mc, eps, seq["layers"][src], p0)
+                y = latent_mixer(x, W, mc, eps, seq["layers"][src], p0, r)
             x = x + rms_norm(y, self.t[f"l{i}.norm1"], eps)
             if layer["mlp"] is not None:
-                x = x + rms_norm(dense_ff(x, self._sub(f"l{i}.mlp.")), self.t[f"l{i}.norm2"], eps)
+                x = x + rms_norm(dense_ff(x, self._sub(f"l{i}.mlp."), r), self.t[f"l{i}.norm2"], eps)
             if trace is not None:
                 trace.append(x.copy())
         seq["pos"] = p0 + len(tokens)
-        return rms_norm(x, self.t["final.norm"], eps) @ self.t["embed"].T * c["logit_scale"]
+        return r(rms_norm(x, self.t["final.norm"], eps)) @ self.t["embed"].T * c["logit_scale"]
