@@ -4,10 +4,12 @@
 // step needs the pages its window touches; the pages of all (row, head group) pairs form one list that is cut into equal
 // ranges, one per CTA (one CTA per SM), so every SM streams the same number of bytes whatever the lengths are.  A producer
 // lane brings whole pages (64 rows) into a ring of shared-memory stages with bulk TMA copies; eight consumer warps run
-//     S [16 heads x 64 keys] = Q' [16 x (rank + rot)] C^T     one 8-key tile per warp
+//     S [16 heads x 64 keys] = Q' [16 x (rank + rot)] C^T     a quarter of the contraction for half of the keys per warp
 //     O [16 x rank] += P C                                    rank / 8 columns per warp
 // on mma.sync m16n8k16 (bf16, fp32 accumulation): at 16 query rows per key byte the kernel is bound by HBM, not by the
-// tensor pipe.  A range that ends inside a pair leaves an (m, l, O) partial; the CTA that delivers a pair's last one joins
+// tensor pipe.  What counts on chip is shared-memory traffic: a warp keeps its part of the queries in registers for a whole
+// pair and every key and value byte is read once; the four partial scores meet in the softmax step, which 16 threads per
+// head do once for all warps.  A range that ends inside a pair leaves an (m, l, O) partial; the CTA that delivers a pair's last one joins
 // them.  The row pitch is an odd number of 16-byte units, which keeps ldmatrix free of bank conflicts.
 #include "block_model.cuh"
 #include "elem.cuh"
@@ -22,7 +24,8 @@ constexpr int kHG = 16;               // heads per group
 constexpr int kLdParts = 16;          // partial slots per pair
 constexpr int kLdMaxRows = 2048;
 constexpr int kLdThreads = 288;       // 8 consumer warps + producer
-constexpr int kSPitch = 68;           // floats per row of the score tile
+constexpr int kSPitch = 68;           // floats per row of a score tile
+constexpr int kPPitch = 72;           // bf16 per row of the weight tile
 
 __device__ __forceinline__ void ldm_x4(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
@@ -42,17 +45,17 @@ __device__ __forceinline__ float ex2l(float x) {
 }
 __device__ __forceinline__ void sync_consumers() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
-struct LdLayout { uint32_t q, s, mx, pre, bar, stage0, stage_bytes, total; int stages; };
+struct LdLayout { uint32_t q, q_bytes, s, p, pre, bar, stage0, stage_bytes, total; int stages; };
 __host__ __device__ inline LdLayout ld_layout(int pitch, int rows) {
     LdLayout L;
     L.q = 0;
-    L.s = L.q + kHG * pitch * 2;
-    L.s = (L.s + 127) / 128 * 128;
-    L.mx = L.s + 2 * kHG * kSPitch * 4;
-    L.pre = L.mx + 2 * 8 * kHG * 4;
-    L.bar = L.pre + (rows + 2 + 3) / 4 * 16;
+    L.q_bytes = (kHG * pitch * 2 + 127) / 128 * 128;         // two query buffers
+    L.s = L.q + 2 * L.q_bytes;
+    L.p = L.s + 4 * kHG * kSPitch * 4;                       // partial scores of the four quarters
+    L.pre = L.p + kHG * kPPitch * 2 + 3 * kHG * 4;           // weights (bf16), then factor, maximum and sum of every head
+    L.bar = L.pre + (2 * rows + 2 + 3) / 4 * 16;
     L.bar = (L.bar + 15) / 16 * 16;
-    L.stage0 = (L.bar + 96 + 127) / 128 * 128;
+    L.stage0 = (L.bar + 128 + 127) / 128 * 128;
     L.stage_bytes = kPageTokens * pitch * 2;
     const uint32_t room = 227 * 1024 - 256 - L.stage0;       // the last column tile of a warp may read a little past a row's end
     L.stages = (int)(room / L.stage_bytes);
@@ -60,11 +63,12 @@ __host__ __device__ inline LdLayout ld_layout(int pitch, int rows) {
     L.total = L.stage0 + L.stages * L.stage_bytes + 256;
     return L;
 }
+template <int NT> constexpr int kPartFloats = NT * 1024 + 32;      // O in register order, then (m, l) of the 16 heads
 struct Seg { int row, hg, p0, p1, np; };   // pages [p0, p1) of the np of one pair
 }  // namespace
 
-// NT = 8-column tiles of the latent per consumer warp
-template <int NT>
+// NT = 8-column tiles of the latent per consumer warp, KQ = 16-column steps of the contraction per warp
+template <int NT, int KQ>
 __global__ void __launch_bounds__(kLdThreads, 1)
 latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa, const LatentView cache, const int* __restrict__ row_slot,
                      const int* __restrict__ row_pos, int rows, float* __restrict__ part, int* __restrict__ counters,
@@ -74,16 +78,24 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
     const LdLayout L = ld_layout(pitch, rows);
     const uint32_t base = smem_u32(sm);
     int* s_pre = reinterpret_cast<int*>(sm + L.pre);              // pages before row r; [rows] = all; [rows + 1] = most of one row
-    uint64_t* bars = reinterpret_cast<uint64_t*>(sm + L.bar);     // full[4], empty[4]
-    volatile int* abort_flag = reinterpret_cast<volatile int*>(bars + 8);
-    int* s_last = reinterpret_cast<int*>(bars + 9);
+    int* s_pos = s_pre + rows + 2;
+    uint64_t* bars = reinterpret_cast<uint64_t*>(sm + L.bar);     // full[4], empty[4], q_full[2], q_empty[2]
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(bars + 12);
+    int* s_last = reinterpret_cast<int*>(bars + 13);
     auto full = [&](int s) { return base + L.bar + 8u * s; };
     auto empty = [&](int s) { return base + L.bar + 32u + 8u * s; };
+    auto q_full = [&](int b) { return base + L.bar + 64u + 8u * b; };
+    auto q_empty = [&](int b) { return base + L.bar + 80u + 8u * b; };
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     if (tid == 0) {
         for (int s = 0; s < 4; ++s) { mbar_init(full(s), 1); mbar_init(empty(s), 8); }
+        for (int b = 0; b < 2; ++b) { mbar_init(q_full(b), 1); mbar_init(q_empty(b), 8); }
         *abort_flag = 0;
         mbar_fence_init();
+    }
+    if (sh.heads % kHG) {             // query rows of absent heads are never copied: finite from the start
+        for (uint32_t e = tid; e < 2 * L.q_bytes / 16; e += kLdThreads) reinterpret_cast<uint4*>(sm + L.q)[e] = make_uint4(0u, 0u, 0u, 0u);
+        fence_proxy_async_smem();
     }
     pdl_wait();
     auto first_key = [&](int pos) { return sh.window > 0 ? max(0, pos - sh.window + 1) : 0; };
@@ -94,6 +106,7 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
             int n = 0;
             if (r < rows) {
                 const int slot = row_slot[r], pos = row_pos[r];
+                s_pos[r] = pos;
                 if (slot >= 0 && slot < cache.max_seqs && pos < cache.capacity[slot]) n = pos / kPageTokens - first_key(pos) / kPageTokens + 1;
             }
             most = max(most, n);
@@ -134,10 +147,14 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
 
     if (warp == 8) {
         if (lane == 0) {
-            int it = 0;
-            for (int u = u0; u < u1;) {
+            int it = 0, sg = 0;
+            for (int u = u0; u < u1; ++sg) {
                 const Seg g = segment(u);
-                const int slot = row_slot[g.row], first = first_key(row_pos[g.row]) / kPageTokens;
+                const int slot = row_slot[g.row], first = first_key(s_pos[g.row]) / kPageTokens;
+                const uint32_t qb = (uint32_t)min(kHG, sh.heads - g.hg * kHG) * pitch * 2;
+                if (sg >= 2 && !mbar_wait(q_empty(sg & 1), ((sg >> 1) - 1) & 1, abort_flag)) break;
+                mbar_arrive_expect_tx(q_full(sg & 1), qb);
+                bulk_g2s(base + L.q + (sg & 1) * L.q_bytes, qa + ((size_t)g.row * sh.heads + g.hg * kHG) * pitch, qb, q_full(sg & 1));
                 const int* table = cache.block_table + (size_t)slot * cache.max_pages_per_seq + first;
                 for (int p = g.p0; p < g.p1; ++p, ++it) {
                     const int s = it % L.stages;
@@ -151,89 +168,94 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
         }
     } else {
         const int g4 = lane >> 2, t4 = lane & 3;                  // fragment row and column pair
-        const int ksteps = (pitch - 8) / 16;
+        const int ksteps = (pitch - 8) / 16, k0 = (warp & 3) * KQ, keys = (warp >> 2) * 32;
+        const int srow = tid >> 4, skey = 4 * (tid & 15);         // softmax: head and four keys of this thread
         const float sc = sh.scale * 1.4426950408889634f;
-        const uint32_t a_addr = base + L.q + ((lane & 15) * pitch + (lane >> 4) * 8) * 2;
-        int it = 0;
-        for (int u = u0; u < u1;) {
+        float* SP = reinterpret_cast<float*>(sm + L.s);
+        __nv_bfloat16* PT = reinterpret_cast<__nv_bfloat16*>(sm + L.p);
+        float* s_al = reinterpret_cast<float*>(sm + L.p + kHG * kPPitch * 2);
+        float *s_m = s_al + kHG, *s_l = s_m + kHG;
+        const uint32_t p_addr = base + L.p + ((lane & 15) * kPPitch + (lane >> 4) * 8) * 2;
+        int it = 0, sg = 0;
+        for (int u = u0; u < u1; ++sg) {
             const Seg g = segment(u);
             u += g.p1 - g.p0;
-            const int pos = row_pos[g.row], first = first_key(pos), key0 = first / kPageTokens * kPageTokens;
+            const int pos = s_pos[g.row], first = first_key(pos), key0 = first / kPageTokens * kPageTokens;
             const int n_heads = min(kHG, sh.heads - g.hg * kHG);
-            sync_consumers();                                     // everyone has left the previous pair's queries
+            mbar_wait_warp(q_full(sg & 1), (sg >> 1) & 1, abort_flag);
+            uint32_t qf[KQ][4];
             {
-                const uint4* src = reinterpret_cast<const uint4*>(qa + ((size_t)g.row * sh.heads + g.hg * kHG) * pitch);
-                const int per_row = pitch / 8;
-                for (int e = tid; e < kHG * per_row; e += 256)
-                    reinterpret_cast<uint4*>(sm + L.q)[e] = e / per_row < n_heads ? src[e] : make_uint4(0u, 0u, 0u, 0u);
+                const uint32_t a_addr = base + L.q + (sg & 1) * L.q_bytes + ((lane & 15) * pitch + (lane >> 4) * 8) * 2;
+#pragma unroll
+                for (int k = 0; k < KQ; ++k)
+                    if (k0 + k < ksteps) ldm_x4(qf[k], a_addr + (k0 + k) * 32);
             }
-            sync_consumers();
-            float o[NT][4], m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+            __syncwarp();
+            if (lane == 0) mbar_arrive(q_empty(sg & 1));
+            float o[NT][4], m_run = -INFINITY, l_run = 0.f;
 #pragma unroll
             for (int n = 0; n < NT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
             for (int p = g.p0; p < g.p1; ++p, ++it) {
-                const int s = it % L.stages, b = it & 1;
+                const int s = it % L.stages;
                 const uint32_t st = base + L.stage0 + s * L.stage_bytes;
                 mbar_wait_warp(full(s), (it / L.stages) & 1, abort_flag);
-                // ---- scores of keys 8 warp .. 8 warp + 7 of the page ----
-                float d[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-                const uint32_t b_addr = st + ((8 * warp + (lane & 7)) * pitch + (lane >> 3) * 8) * 2;
-                int ks = 0;
-#pragma unroll 4
-                for (; ks + 1 < ksteps; ks += 2) {
-                    uint32_t a0[4], a1[4], bb[4];
-                    ldm_x4(bb, b_addr + ks * 32);
-                    ldm_x4(a0, a_addr + ks * 32);
-                    ldm_x4(a1, a_addr + ks * 32 + 32);
-                    mma_bf16(d[0], a0, bb[0], bb[1]);
-                    mma_bf16(d[1], a1, bb[2], bb[3]);
-                }
-                if (ks < ksteps) {                                // the last step reads 8 columns of the row's tail beside its own 16
-                    uint32_t a0[4], bb[4];
-                    ldm_x4(bb, st + ((8 * warp + (lane & 7)) * pitch + ((lane >> 3) & 1) * 8) * 2 + ks * 32);
-                    ldm_x4(a0, a_addr + ks * 32);
-                    mma_bf16(d[0], a0, bb[0], bb[1]);
-                }
-                float v[4];
-                const int kpos = key0 + p * kPageTokens + 8 * warp + 2 * t4;
+                // ---- partial scores of 32 keys over this warp's columns ----
+                {
+                    float d[4][4];
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int k = kpos + (e & 1);
-                    v[e] = (k >= first && k <= pos) ? (d[0][e] + d[1][e]) * sc : -INFINITY;
-                }
-                float* S = reinterpret_cast<float*>(sm + L.s) + b * kHG * kSPitch;
-                float* X = reinterpret_cast<float*>(sm + L.mx) + b * 8 * kHG;
-                *reinterpret_cast<float2*>(S + g4 * kSPitch + 8 * warp + 2 * t4) = make_float2(v[0], v[1]);
-                *reinterpret_cast<float2*>(S + (g4 + 8) * kSPitch + 8 * warp + 2 * t4) = make_float2(v[2], v[3]);
-                float x0 = fmaxf(v[0], v[1]), x1 = fmaxf(v[2], v[3]);
+                    for (int n = 0; n < 4; ++n) d[n][0] = d[n][1] = d[n][2] = d[n][3] = 0.f;
+                    const uint32_t b_addr = st + ((keys + (lane & 7) + ((lane >> 4) << 3)) * pitch + ((lane >> 3) & 1) * 8 + k0 * 16) * 2;
 #pragma unroll
-                for (int k = 1; k < 4; k <<= 1) {
-                    x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, k));
-                    x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, k));
+                    for (int k = 0; k < KQ; ++k)
+                        if (k0 + k < ksteps) {
+                            uint32_t b0[4], b1[4];
+                            ldm_x4(b0, b_addr + k * 32);
+                            ldm_x4(b1, b_addr + k * 32 + 32 * pitch);
+                            mma_bf16(d[0], qf[k], b0[0], b0[1]);
+                            mma_bf16(d[1], qf[k], b0[2], b0[3]);
+                            mma_bf16(d[2], qf[k], b1[0], b1[1]);
+                            mma_bf16(d[3], qf[k], b1[2], b1[3]);
+                        }
+                    float* S = SP + (warp & 3) * kHG * kSPitch + keys + 2 * t4;
+#pragma unroll
+                    for (int n = 0; n < 4; ++n) {
+                        *reinterpret_cast<float2*>(S + g4 * kSPitch + 8 * n) = make_float2(d[n][0], d[n][1]);
+                        *reinterpret_cast<float2*>(S + (g4 + 8) * kSPitch + 8 * n) = make_float2(d[n][2], d[n][3]);
+                    }
                 }
-                if (t4 == 0) { X[warp * kHG + g4] = x0; X[warp * kHG + g4 + 8] = x1; }
                 sync_consumers();
-                // ---- weights: every warp forms the whole 16 x 64 tile as its A operand ----
-                float n0 = m0, n1 = m1;
+                // ---- softmax: 16 threads per head ----
+                {
+                    const float* S = SP + srow * kSPitch + skey;
+                    const float4 a = *reinterpret_cast<const float4*>(S), b = *reinterpret_cast<const float4*>(S + kHG * kSPitch);
+                    const float4 c = *reinterpret_cast<const float4*>(S + 2 * kHG * kSPitch), d = *reinterpret_cast<const float4*>(S + 3 * kHG * kSPitch);
+                    float v[4] = {(a.x + b.x) + (c.x + d.x), (a.y + b.y) + (c.y + d.y), (a.z + b.z) + (c.z + d.z), (a.w + b.w) + (c.w + d.w)};
+                    const int kpos = key0 + p * kPageTokens + skey;
+                    float mx = -INFINITY;
 #pragma unroll
-                for (int w = 0; w < 8; ++w) { n0 = fmaxf(n0, X[w * kHG + g4]); n1 = fmaxf(n1, X[w * kHG + g4 + 8]); }
-                const float al0 = ex2l(m0 - n0), al1 = ex2l(m1 - n1);   // a page holds a visible key, so n0 and n1 are finite
-                m0 = n0; m1 = n1;
-                l0 *= al0; l1 *= al1;
+                    for (int e = 0; e < 4; ++e) {
+                        v[e] = (kpos + e >= first && kpos + e <= pos) ? v[e] * sc : -INFINITY;
+                        mx = fmaxf(mx, v[e]);
+                    }
+#pragma unroll
+                    for (int k = 8; k > 0; k >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, k));
+                    const float mn = fmaxf(m_run, mx), al = ex2l(m_run - mn);    // a page holds a visible key, so mn is finite
+                    m_run = mn;
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) v[e] = ex2l(v[e] - mn);
+                    l_run = l_run * al + ((v[0] + v[1]) + (v[2] + v[3]));
+                    *reinterpret_cast<uint2*>(PT + srow * kPPitch + skey) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+                    if (skey == 0) s_al[srow] = al;
+                }
+                sync_consumers();
+                // ---- O += P C over this warp's columns ----
+                const float al0 = s_al[g4], al1 = s_al[g4 + 8];
 #pragma unroll
                 for (int n = 0; n < NT; ++n) { o[n][0] *= al0; o[n][1] *= al0; o[n][2] *= al1; o[n][3] *= al1; }
 #pragma unroll
                 for (int k = 0; k < 4; ++k) {
                     uint32_t a[4];
-#pragma unroll
-                    for (int hh = 0; hh < 2; ++hh) {
-                        const float2 s0 = *reinterpret_cast<const float2*>(S + g4 * kSPitch + 16 * k + 8 * hh + 2 * t4);
-                        const float2 s1 = *reinterpret_cast<const float2*>(S + (g4 + 8) * kSPitch + 16 * k + 8 * hh + 2 * t4);
-                        const float p0 = ex2l(s0.x - n0), p1 = ex2l(s0.y - n0), p2 = ex2l(s1.x - n1), p3 = ex2l(s1.y - n1);
-                        l0 += p0 + p1; l1 += p2 + p3;
-                        a[2 * hh] = pack_bf16x2(p0, p1);
-                        a[2 * hh + 1] = pack_bf16x2(p2, p3);
-                    }
+                    ldm_x4(a, p_addr + k * 32);
                     // value tiles: 16 keys x 16 columns per transposed load
                     const uint32_t v_addr = st + ((16 * k + (lane & 15)) * pitch + warp * 8 * NT + (lane >> 4) * 8) * 2;
 #pragma unroll
@@ -249,37 +271,43 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
                 if (lane == 0) mbar_arrive(empty(s));
             }
 #pragma unroll
-            for (int k = 1; k < 4; k <<= 1) {
-                l0 += __shfl_xor_sync(0xffffffffu, l0, k);
-                l1 += __shfl_xor_sync(0xffffffffu, l1, k);
-            }
-            const int col = warp * 8 * NT + 2 * t4;
-            __nv_bfloat16* orow = out + ((size_t)g.row * sh.heads + g.hg * kHG) * sh.rank;
-            if (g.p0 == 0 && g.p1 == g.np) {
+            for (int k = 8; k > 0; k >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, k);
+            if (skey == 0) { s_m[srow] = m_run; s_l[srow] = l_run; }
+            sync_consumers();
+            float m0 = s_m[g4], m1 = s_m[g4 + 8], l0 = s_l[g4], l1 = s_l[g4 + 8];
+            auto store = [&] {
                 const float i0 = 1.f / l0, i1 = 1.f / l1;
+                const int col = warp * 8 * NT + 2 * t4;
+                __nv_bfloat16* orow = out + ((size_t)g.row * sh.heads + g.hg * kHG) * sh.rank;
 #pragma unroll
                 for (int n = 0; n < NT; ++n)
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) {
-                        const int hd = g4 + 8 * (e >> 1), c = col + 8 * n + (e & 1);
-                        if (hd < n_heads && c < sh.rank) orow[(size_t)hd * sh.rank + c] = __float2bfloat16_rn(o[n][e] * (e < 2 ? i0 : i1));
+                    for (int e = 0; e < 2; ++e) {
+                        const int hd = g4 + 8 * e, c = col + 8 * n;
+                        const float x = o[n][2 * e] * (e ? i1 : i0), y = o[n][2 * e + 1] * (e ? i1 : i0);
+                        if (hd >= n_heads) continue;
+                        __nv_bfloat16* dst = orow + (size_t)hd * sh.rank + c;
+                        if ((sh.rank & 1) == 0) {
+                            if (c < sh.rank) *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(x, y);
+                        } else {
+                            if (c < sh.rank) dst[0] = __float2bfloat16_rn(x);
+                            if (c + 1 < sh.rank) dst[1] = __float2bfloat16_rn(y);
+                        }
                     }
-                continue;
-            }
-            // ---- partial of a split pair: slot = this CTA's place among the CTAs that share it ----
+            };
+            if (g.p0 == 0 && g.p1 == g.np) { store(); continue; }
+            // ---- partial of a split pair: slot = this CTA's place among the CTAs that share it; accumulators in register order ----
             const int pair = g.row * hgs + g.hg, begin = s_pre[g.row] * hgs + g.hg * g.np, end = begin + g.np;
-            const int cta0 = begin / per, n_parts = (end - 1) / per - cta0 + 1, ld = sh.rank + 2;
-            float* dst = part + ((size_t)pair * kLdParts + (blockIdx.x - cta0)) * kHG * ld;
+            const int cta0 = begin / per, n_parts = (end - 1) / per - cta0 + 1, mine = blockIdx.x - cta0;
+            float* pp = part + (size_t)pair * kLdParts * kPartFloats<NT>;
+            {
+                float* dst = pp + (size_t)mine * kPartFloats<NT>;
 #pragma unroll
-            for (int n = 0; n < NT; ++n)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int hd = g4 + 8 * (e >> 1), c = col + 8 * n + (e & 1);
-                    if (c < sh.rank) dst[hd * ld + c] = o[n][e];
+                for (int n = 0; n < NT; ++n) __stcg(reinterpret_cast<float4*>(dst) + n * 256 + tid, make_float4(o[n][0], o[n][1], o[n][2], o[n][3]));
+                if (warp == 0 && t4 == 0) {
+                    __stcg(reinterpret_cast<float2*>(dst + NT * 1024) + g4, make_float2(m0, l0));
+                    __stcg(reinterpret_cast<float2*>(dst + NT * 1024) + g4 + 8, make_float2(m1, l1));
                 }
-            if (warp == 0 && t4 == 0) {
-                dst[g4 * ld + sh.rank] = m0; dst[g4 * ld + sh.rank + 1] = l0;
-                dst[(g4 + 8) * ld + sh.rank] = m1; dst[(g4 + 8) * ld + sh.rank + 1] = l1;
             }
             __threadfence();
             sync_consumers();
@@ -287,23 +315,29 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
                 const int seen = atomicAdd(counters + pair, 1);
                 *s_last = seen == n_parts - 1;
                 if (seen == n_parts - 1) counters[pair] = 0;      // ready for the next launch
+                __threadfence();
             }
             sync_consumers();
-            if (*s_last) {
-                __threadfence();
-                const float* src = part + (size_t)pair * kLdParts * kHG * ld;
-                for (int e = tid; e < n_heads * sh.rank; e += 256) {
-                    const int hd = e / sh.rank, c = e % sh.rank;
-                    float mx = -INFINITY, l = 0.f, acc = 0.f;
-                    for (int q = 0; q < n_parts; ++q) mx = fmaxf(mx, __ldcg(src + ((size_t)q * kHG + hd) * ld + sh.rank));
-                    for (int q = 0; q < n_parts; ++q) {
-                        const float* r = src + ((size_t)q * kHG + hd) * ld;
-                        const float w = ex2l(__ldcg(r + sh.rank) - mx);
-                        l += w * __ldcg(r + sh.rank + 1);
-                        acc += w * __ldcg(r + c);
+            if (*s_last) {                                        // join the others' partials with the one still in registers
+                for (int q = 0; q < n_parts; ++q) {
+                    if (q == mine) continue;
+                    const float* src = pp + (size_t)q * kPartFloats<NT>;
+                    const float2 a = __ldcg(reinterpret_cast<const float2*>(src + NT * 1024) + g4);
+                    const float2 c = __ldcg(reinterpret_cast<const float2*>(src + NT * 1024) + g4 + 8);
+                    float4 x[NT];
+#pragma unroll
+                    for (int n = 0; n < NT; ++n) x[n] = __ldcg(reinterpret_cast<const float4*>(src) + n * 256 + tid);
+                    const float n0 = fmaxf(m0, a.x), n1 = fmaxf(m1, c.x);
+                    const float s0 = ex2l(m0 - n0), s1 = ex2l(m1 - n1), t0 = ex2l(a.x - n0), t1 = ex2l(c.x - n1);
+                    m0 = n0; m1 = n1;
+                    l0 = l0 * s0 + a.y * t0; l1 = l1 * s1 + c.y * t1;
+#pragma unroll
+                    for (int n = 0; n < NT; ++n) {
+                        o[n][0] = o[n][0] * s0 + x[n].x * t0; o[n][1] = o[n][1] * s0 + x[n].y * t0;
+                        o[n][2] = o[n][2] * s1 + x[n].z * t1; o[n][3] = o[n][3] * s1 + x[n].w * t1;
                     }
-                    orow[(size_t)hd * sh.rank + c] = __float2bfloat16_rn(acc / l);
                 }
+                store();
             }
         }
     }
@@ -312,12 +346,15 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
     if (tid == 0 && *abort_flag) atomicExch(cache.error, 3);
 }
 
+static int ld_tiles(int rank) { return rank <= 64 ? 1 : rank <= 128 ? 2 : rank <= 256 ? 4 : 8; }
+static int ld_steps(const LatentShape& sh) { return ceil_div(sh.row_pitch() - 8, 64); }       // contraction steps per warp
+
 bool latent_decode_fits(const LatentShape& sh, int max_rows) {
-    return sh.rank <= 512 && max_rows <= kLdMaxRows && ld_layout(sh.row_pitch(), max_rows).stages >= 2;
+    return sh.rank <= 512 && ld_steps(sh) <= 12 && max_rows <= kLdMaxRows && ld_layout(sh.row_pitch(), max_rows).stages >= 2;
 }
 
 size_t latent_decode_scratch_floats(const LatentShape& sh, int max_rows) {
-    return (size_t)max_rows * ceil_div(sh.heads, kHG) * kLdParts * kHG * (sh.rank + 2);
+    return (size_t)max_rows * ceil_div(sh.heads, kHG) * kLdParts * (ld_tiles(sh.rank) * 1024 + 32);
 }
 
 int launch_latent_decode(const LatentShape& sh, const void* qa, const LatentView& cache, const int* row_slot, const int* row_pos, int rows,
@@ -325,21 +362,29 @@ int launch_latent_decode(const LatentShape& sh, const void* qa, const LatentView
     int n_sm = 0;
     B2_TRY(device_sm_count(&n_sm));
     const uint32_t smem = ld_layout(sh.row_pitch(), rows).total;
-    static PerDeviceOnce once;
-    B2_PER_DEVICE_ONCE(once,
-        B2_CUDA(cudaFuncSetAttribute(latent_decode_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
-        B2_CUDA(cudaFuncSetAttribute(latent_decode_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
-        B2_CUDA(cudaFuncSetAttribute(latent_decode_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
-        B2_CUDA(cudaFuncSetAttribute(latent_decode_kernel<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024)));
     unsigned long long* stamp = prof_stamp_slot(PROF_FA_DECODE);
     auto go = [&](auto kernel) {
         launch_pdl(kernel, dim3(n_sm), dim3(kLdThreads), smem, s, sh, (const __nv_bfloat16*)qa, cache, row_slot, row_pos, rows, part, counters,
                    (__nv_bfloat16*)out, stamp);
     };
-    if (sh.rank <= 64) go(latent_decode_kernel<1>);
-    else if (sh.rank <= 128) go(latent_decode_kernel<2>);
-    else if (sh.rank <= 256) go(latent_decode_kernel<4>);
-    else go(latent_decode_kernel<8>);
+    auto pick = [&](auto nt) -> int {
+        constexpr int NT = decltype(nt)::value;
+        static PerDeviceOnce once;
+        B2_PER_DEVICE_ONCE(once,
+            B2_CUDA(cudaFuncSetAttribute(latent_decode_kernel<NT, 3>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+            B2_CUDA(cudaFuncSetAttribute(latent_decode_kernel<NT, 9>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+            B2_CUDA(cudaFuncSetAttribute(latent_decode_kernel<NT, 12>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024)));
+        if (ld_steps(sh) <= 3) go(latent_decode_kernel<NT, 3>);
+        else if (ld_steps(sh) <= 9) go(latent_decode_kernel<NT, 9>);
+        else go(latent_decode_kernel<NT, 12>);
+        return 0;
+    };
+    switch (ld_tiles(sh.rank)) {
+        case 1: B2_TRY(pick(std::integral_constant<int, 1>{})); break;
+        case 2: B2_TRY(pick(std::integral_constant<int, 2>{})); break;
+        case 4: B2_TRY(pick(std::integral_constant<int, 4>{})); break;
+        default: B2_TRY(pick(std::integral_constant<int, 8>{})); break;
+    }
     B2_LAUNCH_CHECK();
     return 0;
 }
