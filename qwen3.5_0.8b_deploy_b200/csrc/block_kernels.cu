@@ -21,6 +21,25 @@ int launch_row_map(const LaSeqMeta* d_seqs, int n_seqs, int max_count, const int
     return 0;
 }
 
+// One block of 64 threads per row: cos and sin of position times frequency, the product in double and reduced to one turn.
+__global__ void __launch_bounds__(64)
+rot_table_kernel(const int* __restrict__ row_pos, const double* __restrict__ freq, int half, float2* __restrict__ table) {
+    pdl_enter();
+    const double pos = row_pos[blockIdx.x];
+    for (int i = threadIdx.x; i < half; i += 64) {
+        const double turns = pos * freq[i] * 0.15915494309189535;
+        float2 cs;
+        sincosf((float)((turns - rint(turns)) * 6.283185307179586), &cs.y, &cs.x);
+        table[(size_t)blockIdx.x * half + i] = cs;
+    }
+}
+
+int launch_rot_table(const int* row_pos, const double* freq, int half, int rows, float2* table, cudaStream_t s) {
+    launch_pdl(rot_table_kernel, dim3(rows), dim3(64), 0, s, row_pos, freq, half, table);
+    B2_LAUNCH_CHECK();
+    return 0;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128)
 embed_scaled_kernel(const int* __restrict__ tokens, const T* __restrict__ embed, int vocab, int width, float scale,
@@ -35,6 +54,14 @@ embed_scaled_kernel(const int* __restrict__ tokens, const T* __restrict__ embed,
     }
     const int tok = min(max(tokens[row], 0), vocab - 1);
     const T* e = embed + (size_t)tok * width;
+    if ((width & 3) == 0) {
+        for (int c = 4 * threadIdx.x; c < width; c += 512) {
+            const float4 v = load4(e + c), r = make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale);
+            store4(x + (size_t)row * width + c, r);
+            store4(xt + (size_t)row * width + c, r);
+        }
+        return;
+    }
     for (int c = threadIdx.x; c < width; c += 128) {
         const float v = to_f32(e[c]) * scale;
         x[(size_t)row * width + c] = v;
@@ -123,26 +150,31 @@ int launch_rms_norm_rows(ElemType t, const float* x, const int* row_index, const
     return 0;
 }
 
+// 0.5 z (1 + tanh y) = z / (1 + e^{-2y}), y = sqrt(2 / pi) (z + 0.044715 z^3)
 __device__ __forceinline__ float gelu_tanh(float z) {
-    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }
 
 template <typename T>
 __global__ void __launch_bounds__(256)
 gelu_mul_kernel(const T* __restrict__ gu, int ff, size_t n, T* __restrict__ act) {
     pdl_enter();
-    if ((ff & 3) == 0) {
-        const size_t i = 4 * ((size_t)blockIdx.x * 256 + threadIdx.x);
-        if (i >= n) return;
-        const size_t row = i / ff, c = i % ff;
-        const float4 g = load4(gu + row * 2 * ff + c), u = load4(gu + row * 2 * ff + ff + c);
-        store4(act + i, make_float4(gelu_tanh(g.x) * u.x, gelu_tanh(g.y) * u.y, gelu_tanh(g.z) * u.z, gelu_tanh(g.w) * u.w));
+    const size_t i0 = 8 * ((size_t)blockIdx.x * 256 + threadIdx.x);
+    if (i0 >= n) return;
+    if ((ff & 7) == 0) {
+        const size_t row = i0 / ff, c = i0 - row * ff;
+        const T* p = gu + row * 2 * ff + c;
+        float4 g[2], u[2];
+#pragma unroll
+        for (int k = 0; k < 2; ++k) { g[k] = load4(p + 4 * k); u[k] = load4(p + ff + 4 * k); }
+#pragma unroll
+        for (int k = 0; k < 2; ++k)
+            store4(act + i0 + 4 * k, make_float4(gelu_tanh(g[k].x) * u[k].x, gelu_tanh(g[k].y) * u[k].y, gelu_tanh(g[k].z) * u[k].z,
+                                                 gelu_tanh(g[k].w) * u[k].w));
         return;
     }
-    for (int e = 0; e < 4; ++e) {
-        const size_t i = 4 * ((size_t)blockIdx.x * 256 + threadIdx.x) + e;
-        if (i >= n) return;
-        const size_t row = i / ff, c = i % ff;
+    for (size_t i = i0; i < i0 + 8 && i < n; ++i) {
+        const size_t row = i / ff, c = i - row * ff;
         act[i] = from_f32<T>(gelu_tanh(to_f32(gu[row * 2 * ff + c])) * to_f32(gu[row * 2 * ff + ff + c]));
     }
 }
@@ -151,7 +183,7 @@ int launch_gelu_mul(ElemType t, const void* gu, int rows, int ff, void* act, cud
     const size_t n = (size_t)rows * ff;
     dispatch_elem(t, [&](auto tag) {
         using T = decltype(tag);
-        launch_pdl(gelu_mul_kernel<T>, dim3((unsigned)((n + 1023) / 1024)), dim3(256), 0, s, (const T*)gu, ff, n, (T*)act);
+        launch_pdl(gelu_mul_kernel<T>, dim3((unsigned)((n + 2047) / 2048)), dim3(256), 0, s, (const T*)gu, ff, n, (T*)act);
     });
     B2_LAUNCH_CHECK();
     return 0;

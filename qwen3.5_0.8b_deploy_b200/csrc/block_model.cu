@@ -48,10 +48,6 @@ static int make_latent(const b200attn_layer_desc& d, const b200attn_model_config
     B2_TRY(op.w_uv.alloc((size_t)sh.heads * sh.vp * sh.rank * e));
     B2_TRY(op.w_out.alloc((size_t)c.width * sh.heads * sh.vp * e));
     B2_TRY(op.c_norm.alloc((size_t)sh.rank * 4));
-    std::vector<double> f(std::max(1, sh.rot / 2));
-    for (int i = 0; i < sh.rot / 2; ++i) f[i] = std::pow(d.rot_base, -2.0 * i / sh.rot);
-    B2_TRY(op.freq.alloc(f.size() * 8));
-    B2_CUDA(cudaMemcpy(op.freq.p, f.data(), f.size() * 8, cudaMemcpyHostToDevice));
     return 0;
 }
 
@@ -106,6 +102,15 @@ int block_model_create(const b200attn_model_config* cfg, const b200attn_layer_de
                 op.pool_layer = m.layers[d.kv_from].latent->pool_layer;
             }
             for (const char* n : {"mix.q", "mix.uk", "mix.uv", "mix.o"}) need(n);
+            op.rot_table = -1;
+            for (size_t k = 0; k < m.rot.size(); ++k)
+                if (m.rot[k].base == d.rot_base && m.rot[k].half == sh.rot / 2) op.rot_table = (int)k;
+            if (op.rot_table < 0) {
+                op.rot_table = (int)m.rot.size();
+                m.rot.emplace_back();
+                m.rot.back().base = d.rot_base;
+                m.rot.back().half = sh.rot / 2;
+            }
             proj = std::max(proj, (size_t)sh.pitch());
             mixed = std::max(mixed, (size_t)sh.heads * sh.vp);
             q = std::max(q, (size_t)sh.q_cols());
@@ -152,6 +157,13 @@ int block_model_create(const b200attn_model_config* cfg, const b200attn_layer_de
     m.abs_rows = (int)std::min<size_t>(R, std::max(4096, cfg->max_seqs));
     m.ctx_rows = (int)R + max_window;
     m.max_spans = (int)std::max<size_t>(cfg->max_seqs, 1);
+    for (RotTable& t : m.rot) {
+        std::vector<double> f(std::max(1, t.half));
+        for (int i = 0; i < t.half; ++i) f[i] = std::pow(t.base, -(double)i / t.half);
+        B2_TRY(t.freq.alloc(f.size() * 8));
+        B2_CUDA(cudaMemcpy(t.freq.p, f.data(), f.size() * 8, cudaMemcpyHostToDevice));
+        B2_TRY(t.cs.alloc(R * f.size() * sizeof(float2)));
+    }
     B2_TRY(m.x.alloc(R * W * 4));
     B2_TRY(m.xt.alloc(R * W * e));
     B2_TRY(m.y.alloc(R * W * 4));
@@ -370,7 +382,7 @@ static int latent_absorbed(BlockModel& m, LatentOp& op, const PassRows& p, const
         const int n = std::min(m.abs_rows, p.rows - r0);
         void* q = (char*)m.q.p + (size_t)r0 * sh.q_cols() * e;
         const int *slot = p.row_slot + r0, *pos = p.row_pos + r0;
-        LatentPreArgs a{sh, m.proj.f() + (size_t)r0 * sh.pitch(), (const double*)op.freq.p, op.c_norm.f(), slot, pos, cache, q, m.qa.p};
+        LatentPreArgs a{sh, m.proj.f() + (size_t)r0 * sh.pitch(), (const float2*)m.rot[op.rot_table].cs.p + (size_t)r0 * (sh.rot / 2), op.c_norm.f(), slot, pos, cache, q, m.qa.p};
         B2_TRY(launch_latent_pre(op.elem, a, n, s));
         B2_TRY(gemm_heads(s, q, sh.q_cols(), hw, op.w_uk.p, true, m.qa.p, sh.heads * sh.row_pitch(), sh.row_pitch(), op.elem, op.elem, n, sh.rank, sh.dp,
                           sh.heads));
@@ -394,7 +406,7 @@ static LatentSpan context_span(const LatentShape& sh, int slot, int base, int co
 // Prefill on the tensor cores: the context's latents are staged and up-projected to keys and values once per pass.
 static int latent_expanded(BlockModel& m, LatentOp& op, const PassRows& p, const LatentView& cache, cudaStream_t s) {
     const LatentShape& sh = op.sh;
-    LatentPreArgs a{sh, m.proj.f(), (const double*)op.freq.p, op.c_norm.f(), p.row_slot, p.row_pos, cache, m.q.p, nullptr};
+    LatentPreArgs a{sh, m.proj.f(), (const float2*)m.rot[op.rot_table].cs.p, op.c_norm.f(), p.row_slot, p.row_pos, cache, m.q.p, nullptr};
     B2_TRY(launch_latent_pre(op.elem, a, p.rows, s));
     std::vector<LatentSpan> spans;
     std::vector<LatentTile> tiles;
@@ -446,6 +458,8 @@ static int run_layers(BlockModel& m, const PassRows& p, cudaStream_t s) {
     const int W = m.cfg.width;
     const float eps = (float)m.cfg.norm_eps;
     m.staged_layer = -1;
+    for (RotTable& t : m.rot)
+        if (t.half > 0) B2_TRY(launch_rot_table(p.row_pos, (const double*)t.freq.p, t.half, p.rows, (float2*)t.cs.p, s));
     for (size_t i = 0; i < m.layers.size(); ++i) {
         if (m.stop_after >= 0 && (int)i >= m.stop_after) break;
         BlockLayer& L = m.layers[i];

@@ -52,6 +52,8 @@ struct PassRows {
 
 // ---- block_kernels.cu: element-wise steps around the mixers -----------------------------------------------------------
 int launch_row_map(const LaSeqMeta* d_seqs, int n_seqs, int max_count, const int* lens, int* row_slot, int* row_pos, cudaStream_t s);
+// table[row][i] = (cos, sin) of row_pos[row] * freq[i].
+int launch_rot_table(const int* row_pos, const double* freq, int half, int rows, float2* table, cudaStream_t s);
 // x = embed[token] * scale, with a copy in the element type; decode also fills row_slot / row_pos from d_slots and lens.
 int launch_embed_scaled(ElemType t, const int* tokens, const void* embed, int vocab, int width, float scale, int rows, const int* d_slots,
                         const int* lens, int max_seqs, int* row_slot, int* row_pos, float* x, void* xt, cudaStream_t s);
@@ -125,7 +127,7 @@ struct LatentShape {
 struct LatentPreArgs {                 // behind the input projection: rotate q, norm and rotate the new latents, append them
     LatentShape sh;
     const float* proj;
-    const double* freq;                // [rot / 2]
+    const float2* cs;                  // [rows][rot / 2] cos and sin of the rows' angles
     const float* c_norm;               // [rank]
     const int* row_slot;
     const int* row_pos;
@@ -159,7 +161,14 @@ struct LatentOp {
     ElemType elem = ELEM_BF16;
     int width = 0, pool_layer = 0;     // the pool layer it reads (its own or its source's)
     bool tc_prefill = false, tc_decode = false;
-    DevBuf w_in, w_uk, w_uv, w_out, c_norm, freq;
+    int rot_table = 0;                 // index of its rotation's table
+    DevBuf w_in, w_uk, w_uv, w_out, c_norm;
+};
+
+struct RotTable {                      // one rotation (base and size) of a model: filled once per pass, shared by the layers that use it
+    double base = 0;
+    int half = 0;
+    DevBuf freq, cs;
 };
 
 // ---- block_model.cu ---------------------------------------------------------------------------------------------------------
@@ -175,6 +184,7 @@ struct BlockModel {
     b200attn_model_config cfg{};
     ElemType elem = ELEM_BF16;
     std::vector<BlockLayer> layers;
+    std::vector<RotTable> rot;
     std::vector<std::string> missing;
     DevBuf embed, final_norm;
     int stop_after = -1;               // >= 0: passes end behind that many layers

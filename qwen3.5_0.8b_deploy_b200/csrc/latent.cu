@@ -11,87 +11,96 @@
 
 namespace b200 {
 
-// One block of 128 threads per row.  Angles: position times the frequency in double, reduced to one turn before sin and cos.
+// One block of 256 threads per row.  The new latents' values are requested before the queries are worked on.
 template <typename T>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 latent_pre_kernel(const LatentPreArgs a) {
-    extern __shared__ float s_cs[];            // cos[half], sin[half], partial sums[4]
+    constexpr int kOwn = 4;                    // latent values a thread keeps (ranks of up to 1024)
+    __shared__ float s_part[8];
+    extern __shared__ float2 s_cs[];
     pdl_enter();
     const LatentShape& sh = a.sh;
     const int row = blockIdx.x, tid = threadIdx.x, half = sh.rot / 2;
     const int slot = a.row_slot[row], pos = a.row_pos[row];
     if (slot < 0 || slot >= a.cache.max_seqs) return;
-    float *s_c = s_cs, *s_s = s_cs + half, *s_part = s_cs + 2 * half;
-    for (int i = tid; i < half; i += 128) {
-        const double turns = (double)pos * a.freq[i] * 0.15915494309189535;
-        sincosf((float)((turns - rint(turns)) * 6.283185307179586), &s_s[i], &s_c[i]);
-    }
     const float* pr = a.proj + (size_t)row * sh.pitch();
-    __syncthreads();
-    const int hw = sh.dp + sh.rp;
-    T* q = static_cast<T*>(a.q) + (size_t)row * sh.heads * hw;
-    for (int e = tid; e < sh.heads * (hw / 4); e += 128) {          // four columns at a time; hw and dp are multiples of 8
-        const int h = e / (hw / 4), c = 4 * (e % (hw / 4));
-        const float* src = pr + h * hw;
-        float4 v = load4(src + c);
-        if (c >= sh.dp) {
-            float r[4];
+    const float* y = pr + sh.q_cols();
+    float own[kOwn], ss = 0.f;
+    if (sh.own) {
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
-                const int i = c - sh.dp + j, p = i < half ? i : i - half;
-                r[j] = 0.f;
-                if (i < sh.rot) {
-                    const float x = src[sh.dp + i], y = i < half ? src[sh.dp + i + half] : src[sh.dp + i - half];
-                    r[j] = i < half ? x * s_c[p] - y * s_s[p] : x * s_c[p] + y * s_s[p];
-                }
-            }
-            v = make_float4(r[0], r[1], r[2], r[3]);
-            if (a.qa) {
-                T* qa = static_cast<T*>(a.qa) + ((size_t)row * sh.heads + h) * sh.row_pitch() + sh.rank;
-#pragma unroll
-                for (int j = 0; j < 4; ++j)
-                    if (c - sh.dp + j < sh.rot) qa[c - sh.dp + j] = from_f32<T>(r[j]);
-            }
+        for (int k = 0; k < kOwn; ++k) {
+            const int c = tid + 256 * k;
+            own[k] = c < sh.rank ? y[c] : 0.f;
+            ss += own[k] * own[k];
         }
-        store4(q + h * hw + c, v);
+    }
+    for (int i = tid; i < half; i += 256) s_cs[i] = a.cs[(size_t)row * half + i];
+    const int hw = sh.dp + sh.rp, per = hw / 4;
+    T* q = static_cast<T*>(a.q) + (size_t)row * sh.heads * hw;
+    // unrotated parts: four columns at a time (hw and dp are multiples of 8)
+    const int n4 = sh.heads * per;
+#pragma unroll 4
+    for (int e = tid; e < n4; e += 256) {
+        const int h = e / per, c = 4 * (e - h * per);
+        if (c < sh.dp) store4(q + 4 * (size_t)e, load4(pr + 4 * (size_t)e));
+    }
+    __syncthreads();
+    // rotated parts, a pair (i, i + half) at a time; the padded columns behind are zero
+    for (int e = tid; e < sh.heads * half; e += 256) {
+        const int h = e / half, i = e - h * half;
+        const float* src = pr + h * hw + sh.dp;
+        const float u = src[i], v = src[i + half];
+        const float2 cs = s_cs[i];
+        const T ru = from_f32<T>(u * cs.x - v * cs.y), rv = from_f32<T>(v * cs.x + u * cs.y);
+        T* dst = q + h * hw + sh.dp;
+        dst[i] = ru;
+        dst[i + half] = rv;
+        if (a.qa) {
+            T* qa = static_cast<T*>(a.qa) + ((size_t)row * sh.heads + h) * sh.row_pitch() + sh.rank;
+            qa[i] = ru;
+            qa[i + half] = rv;
+        }
+    }
+    if (sh.rp > sh.rot) {
+        const int pad = sh.rp - sh.rot;
+        for (int e = tid; e < sh.heads * pad; e += 256) q[(e / pad) * hw + sh.dp + sh.rot + e % pad] = from_f32<T>(0.f);
     }
     if (a.qa) {                                                    // zero tail behind the rotated part
         const int tail0 = sh.rank + sh.rot, tail = sh.row_pitch() - tail0;
-        T* qa = static_cast<T*>(a.qa) + (size_t)row * sh.heads * sh.row_pitch();
-        for (int e = tid; e < sh.heads * tail; e += 128) qa[(e / tail) * sh.row_pitch() + tail0 + e % tail] = from_f32<T>(0.f);
+        T* qa = static_cast<T*>(a.qa) + (size_t)row * sh.heads * sh.row_pitch() + tail0;
+        for (int e = tid; e < sh.heads * tail; e += 256) qa[(e / tail) * sh.row_pitch() + e % tail] = from_f32<T>(0.f);
     }
     if (!sh.own) return;
-    const float* y = pr + sh.q_cols();
-    float ss = 0.f;
-    for (int c = tid; c < sh.rank; c += 128) ss += y[c] * y[c];
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     if ((tid & 31) == 0) s_part[tid >> 5] = ss;
     __syncthreads();
-    const float rms = sqrtf(((s_part[0] + s_part[1]) + (s_part[2] + s_part[3])) / (float)sh.rank + sh.eps);
+    ss = ((s_part[0] + s_part[1]) + (s_part[2] + s_part[3])) + ((s_part[4] + s_part[5]) + (s_part[6] + s_part[7]));
+    const float rms = sqrtf(ss / (float)sh.rank + sh.eps);
     if (pos >= a.cache.capacity[slot]) {
         if (tid == 0) atomicExch(a.cache.error, 2);                // page not reserved: skip the write
         return;
     }
     const int page = a.cache.block_table[slot * a.cache.max_pages_per_seq + pos / kPageTokens];
     T* dst = static_cast<T*>(a.cache.rows) + ((size_t)page * kPageTokens + pos % kPageTokens) * a.cache.pitch;
-    for (int c = tid; c < a.cache.pitch; c += 128) {
-        float v = 0.f;
-        if (c < sh.rank) {
-            v = y[c] / rms * a.c_norm[c];
-        } else if (c < sh.rank + sh.rot) {
-            const int i = c - sh.rank, p = i < half ? i : i - half;
-            const float x = y[c], z = i < half ? y[c + half] : y[c - half];
-            v = i < half ? x * s_c[p] - z * s_s[p] : x * s_c[p] + z * s_s[p];
-        }
-        dst[c] = from_f32<T>(v);
+#pragma unroll
+    for (int k = 0; k < kOwn; ++k) {
+        const int c = tid + 256 * k;
+        if (c < sh.rank) dst[c] = from_f32<T>(own[k] / rms * a.c_norm[c]);
     }
+    for (int i = tid; i < half; i += 256) {
+        const float u = y[sh.rank + i], v = y[sh.rank + half + i];
+        const float2 cs = s_cs[i];
+        dst[sh.rank + i] = from_f32<T>(u * cs.x - v * cs.y);
+        dst[sh.rank + half + i] = from_f32<T>(v * cs.x + u * cs.y);
+    }
+    for (int c = sh.rank + sh.rot + tid; c < a.cache.pitch; c += 256) dst[c] = from_f32<T>(0.f);
 }
 
 int launch_latent_pre(ElemType t, const LatentPreArgs& a, int rows, cudaStream_t s) {
     dispatch_elem(t, [&](auto tag) {
         using T = decltype(tag);
-        launch_pdl(latent_pre_kernel<T>, dim3(rows), dim3(128), (size_t)(round_up(a.sh.rot, 4) + 4) * 4, s, a);
+        launch_pdl(latent_pre_kernel<T>, dim3(rows), dim3(256), (size_t)(a.sh.rot / 2 + 1) * sizeof(float2), s, a);
     });
     B2_LAUNCH_CHECK();
     return 0;

@@ -319,14 +319,7 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
             }
             sync_consumers();
             if (*s_last) {                                        // join the others' partials with the one still in registers
-                for (int q = 0; q < n_parts; ++q) {
-                    if (q == mine) continue;
-                    const float* src = pp + (size_t)q * kPartFloats<NT>;
-                    const float2 a = __ldcg(reinterpret_cast<const float2*>(src + NT * 1024) + g4);
-                    const float2 c = __ldcg(reinterpret_cast<const float2*>(src + NT * 1024) + g4 + 8);
-                    float4 x[NT];
-#pragma unroll
-                    for (int n = 0; n < NT; ++n) x[n] = __ldcg(reinterpret_cast<const float4*>(src) + n * 256 + tid);
+                auto join = [&](float2 a, float2 c, const float4 (&x)[NT]) {
                     const float n0 = fmaxf(m0, a.x), n1 = fmaxf(m1, c.x);
                     const float s0 = ex2l(m0 - n0), s1 = ex2l(m1 - n1), t0 = ex2l(a.x - n0), t1 = ex2l(c.x - n1);
                     m0 = n0; m1 = n1;
@@ -336,6 +329,22 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
                         o[n][0] = o[n][0] * s0 + x[n].x * t0; o[n][1] = o[n][1] * s0 + x[n].y * t0;
                         o[n][2] = o[n][2] * s1 + x[n].z * t1; o[n][3] = o[n][3] * s1 + x[n].w * t1;
                     }
+                };
+                auto fetch = [&](int q, float2& a, float2& c, float4 (&x)[NT]) {
+                    const float* src = pp + (size_t)q * kPartFloats<NT>;
+                    a = __ldcg(reinterpret_cast<const float2*>(src + NT * 1024) + g4);
+                    c = __ldcg(reinterpret_cast<const float2*>(src + NT * 1024) + g4 + 8);
+#pragma unroll
+                    for (int n = 0; n < NT; ++n) x[n] = __ldcg(reinterpret_cast<const float4*>(src) + n * 256 + tid);
+                };
+                for (int i = 0; i < n_parts - 1; i += 2) {        // two parts' loads under way together
+                    const int qa2 = i + (i >= mine), qb2 = i + 1 + (i + 1 >= mine);
+                    float2 a, c, b = make_float2(0.f, 0.f), d = b;
+                    float4 x[NT], z[NT];
+                    fetch(qa2, a, c, x);
+                    if (i + 1 < n_parts - 1) fetch(qb2, b, d, z);
+                    join(a, c, x);
+                    if (i + 1 < n_parts - 1) join(b, d, z);
                 }
                 store();
             }

@@ -74,3 +74,33 @@ def ffn_weights(seed: int, tag: str) -> dict:
 
 def hidden_states(seed: int, name: str, rows: int) -> np.ndarray:
     return normal(seed, name, (rows, HIDDEN), 1.0)
+
+
+def nuzopel_tensors(config: dict, seed: int, std: float = 0.02) -> dict:
+    """Random weights of a Nuzopel configuration under the names a model file has: matrices ~ N(0, std), norms 1, gate biases
+    0 (input) and 3 (forget)."""
+    out = {"embed": normal(seed, "embed", (config["vocab"], config["width"]), std), "final.norm": np.ones(config["width"], np.float32)}
+    w = config["width"]
+    for i, layer in enumerate(config["layers"]):
+        m, p = layer["mixer"], f"l{i}."
+        heads, dim, vdim = m["heads"], m["dim"], m["vdim"]
+        if layer["type"] == "mlstm":
+            shapes = {"q": (heads * dim, w), "k": (heads * dim, w), "v": (heads * vdim, w), "g": (heads * vdim, w), "o": (w, heads * vdim), "i": (heads, w),
+                      "f": (heads, w)}
+            out.update({p + "mix.norm": np.ones(heads * vdim, np.float32), p + "mix.i.b": np.zeros(heads, np.float32),
+                        p + "mix.f.b": np.full(heads, 3.0, np.float32)})
+        else:
+            rot, rank = m["rot_dim"], m["kv_rank"]
+            shapes = {"q": (heads * (dim + rot), w), "uk": (heads * dim, rank), "uv": (heads * vdim, rank), "o": (w, heads * vdim)}
+            if m.get("kv_from") is None:
+                shapes["dkv"] = (rank + rot, w)
+                out[p + "mix.dkv.norm"] = np.ones(rank, np.float32)
+        for n, shape in shapes.items():
+            out[p + "mix." + n] = normal(seed, p + "mix." + n, shape, std)
+        out[p + "norm1"] = np.ones(w, np.float32)
+        if layer["mlp"] is not None:
+            ff = layer["mlp"]["ff"]
+            out[p + "norm2"] = np.ones(w, np.float32)
+            for n, shape in (("gate", (ff, w)), ("up", (ff, w)), ("down", (w, ff))):
+                out[p + "mlp." + n] = normal(seed, p + "mlp." + n, shape, std)
+    return out
