@@ -151,39 +151,33 @@ int launch_rms_norm_rows(ElemType t, const float* x, const int* row_index, const
 }
 
 // 0.5 z (1 + tanh y) = z / (1 + e^{-2y}), y = sqrt(2 / pi) (z + 0.044715 z^3)
+template <typename T>
 __device__ __forceinline__ float gelu_tanh(float z) {
-    return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+    return times_sigmoid<T>(z, 1.5957691216057308f * (z + 0.044715f * z * z * z));
 }
 
+// Blocks of 128 threads: one per row, or (few rows) several along it.
 template <typename T>
-__global__ void __launch_bounds__(256)
-gelu_mul_kernel(const T* __restrict__ gu, int ff, size_t n, T* __restrict__ act) {
+__global__ void __launch_bounds__(128)
+gelu_mul_kernel(const T* __restrict__ gu, int ff, T* __restrict__ act) {
     pdl_enter();
-    const size_t i0 = 8 * ((size_t)blockIdx.x * 256 + threadIdx.x);
-    if (i0 >= n) return;
-    if ((ff & 7) == 0) {
-        const size_t row = i0 / ff, c = i0 - row * ff;
-        const T* p = gu + row * 2 * ff + c;
-        float4 g[2], u[2];
-#pragma unroll
-        for (int k = 0; k < 2; ++k) { g[k] = load4(p + 4 * k); u[k] = load4(p + ff + 4 * k); }
-#pragma unroll
-        for (int k = 0; k < 2; ++k)
-            store4(act + i0 + 4 * k, make_float4(gelu_tanh(g[k].x) * u[k].x, gelu_tanh(g[k].y) * u[k].y, gelu_tanh(g[k].z) * u[k].z,
-                                                 gelu_tanh(g[k].w) * u[k].w));
+    const T* g = gu + (size_t)blockIdx.x * 2 * ff;
+    T* o = act + (size_t)blockIdx.x * ff;
+    if ((ff & 3) == 0) {
+#pragma unroll 4
+        for (int c = 4 * (threadIdx.x + 128 * blockIdx.y); c < ff; c += 512 * gridDim.y) {
+            const float4 a = load4(g + c), u = load4(g + ff + c);
+            store4(o + c, make_float4(gelu_tanh<T>(a.x) * u.x, gelu_tanh<T>(a.y) * u.y, gelu_tanh<T>(a.z) * u.z, gelu_tanh<T>(a.w) * u.w));
+        }
         return;
     }
-    for (size_t i = i0; i < i0 + 8 && i < n; ++i) {
-        const size_t row = i / ff, c = i - row * ff;
-        act[i] = from_f32<T>(gelu_tanh(to_f32(gu[row * 2 * ff + c])) * to_f32(gu[row * 2 * ff + ff + c]));
-    }
+    for (int c = threadIdx.x + 128 * blockIdx.y; c < ff; c += 128 * gridDim.y) o[c] = from_f32<T>(gelu_tanh<T>(to_f32(g[c])) * to_f32(g[ff + c]));
 }
 
 int launch_gelu_mul(ElemType t, const void* gu, int rows, int ff, void* act, cudaStream_t s) {
-    const size_t n = (size_t)rows * ff;
     dispatch_elem(t, [&](auto tag) {
         using T = decltype(tag);
-        launch_pdl(gelu_mul_kernel<T>, dim3((unsigned)((n + 2047) / 2048)), dim3(256), 0, s, (const T*)gu, ff, n, (T*)act);
+        launch_pdl(gelu_mul_kernel<T>, dim3(rows, rows < 1024 ? ceil_div(ff, 512) : 1), dim3(128), 0, s, (const T*)gu, ff, (T*)act);
     });
     B2_LAUNCH_CHECK();
     return 0;

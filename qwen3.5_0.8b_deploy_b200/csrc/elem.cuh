@@ -40,6 +40,11 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
     *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
 }
 
+// x * sigmoid(z): library functions for fp32 outputs, the fast exponential and divide where the result is rounded to bf16.
+template <typename T> __device__ __forceinline__ float times_sigmoid(float x, float z);
+template <> __device__ __forceinline__ float times_sigmoid<float>(float x, float z) { return x / (1.0f + expf(-z)); }
+template <> __device__ __forceinline__ float times_sigmoid<__nv_bfloat16>(float x, float z) { return __fdividef(x, 1.0f + __expf(-z)); }
+
 template <typename F>
 inline void dispatch_elem(ElemType t, F&& f) {
     if (t == ELEM_F32) f(float{});

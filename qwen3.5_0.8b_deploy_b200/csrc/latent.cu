@@ -11,96 +11,110 @@
 
 namespace b200 {
 
-// One block of 256 threads per row.  The new latents' values are requested before the queries are worked on.
-template <typename T>
-__global__ void __launch_bounds__(256)
-latent_pre_kernel(const LatentPreArgs a) {
-    constexpr int kOwn = 4;                    // latent values a thread keeps (ranks of up to 1024)
-    __shared__ float s_part[8];
-    extern __shared__ float2 s_cs[];
-    pdl_enter();
-    const LatentShape& sh = a.sh;
-    const int row = blockIdx.x, tid = threadIdx.x, half = sh.rot / 2;
-    const int slot = a.row_slot[row], pos = a.row_pos[row];
-    if (slot < 0 || slot >= a.cache.max_seqs) return;
-    const float* pr = a.proj + (size_t)row * sh.pitch();
-    const float* y = pr + sh.q_cols();
-    float own[kOwn], ss = 0.f;
-    if (sh.own) {
+// The queries of a row: unrotated parts converted, rotated parts turned.  A warp per head.  With heads of up to 128 + 64
+// columns (kSmallHead) two whole heads are requested before the first value is used; the others go piece by piece.
+template <typename T, bool kSmallHead>
+__device__ __forceinline__ void latent_queries(const LatentPreArgs& a, int row, const float* __restrict__ pr) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int half = a.sh.rot / 2, heads = a.sh.heads, dp = a.sh.dp, hw = a.sh.dp + a.sh.rp, ap = a.sh.row_pitch();
+    const float2* __restrict__ cs = a.cs + (size_t)row * half;
+    T* __restrict__ q = static_cast<T*>(a.q) + (size_t)row * heads * hw;
+    T* __restrict__ qa = a.qa ? static_cast<T*>(a.qa) + (size_t)row * heads * ap + a.sh.rank : nullptr;
+    auto rotated = [&](int h, int i, float u, float v, float2 t) {           // pair (i, i + half)
+        const T x = from_f32<T>(u * t.x - v * t.y), z = from_f32<T>(v * t.x + u * t.y);
+        T* dst = q + h * hw + dp + i;
+        dst[0] = x;
+        dst[half] = z;
+        if (qa) {
+            qa[h * ap + i] = x;
+            qa[h * ap + i + half] = z;
+        }
+    };
+    auto pads = [&](int h) {                                                 // columns behind the rotated part are zero
+        for (int i = a.sh.rot + lane; i < a.sh.rp; i += 32) q[h * hw + dp + i] = from_f32<T>(0.f);
+        if (qa)
+            for (int i = a.sh.rot + lane; i < ap - a.sh.rank; i += 32) qa[h * ap + i] = from_f32<T>(0.f);
+    };
+    if constexpr (kSmallHead) {
+        const float2 t = lane < half ? cs[lane] : make_float2(1.f, 0.f);
+        for (int h0 = warp; h0 < heads; h0 += 16) {
+            float4 x[2];
+            float u[2], v[2];
 #pragma unroll
-        for (int k = 0; k < kOwn; ++k) {
-            const int c = tid + 256 * k;
-            own[k] = c < sh.rank ? y[c] : 0.f;
-            ss += own[k] * own[k];
+            for (int k = 0; k < 2; ++k) {
+                const float* src = pr + (h0 + 8 * k) * hw;
+                const bool in = h0 + 8 * k < heads;
+                x[k] = in && 4 * lane < dp ? load4(src + 4 * lane) : make_float4(0.f, 0.f, 0.f, 0.f);
+                u[k] = in && lane < half ? src[dp + lane] : 0.f;
+                v[k] = in && lane < half ? src[dp + half + lane] : 0.f;
+            }
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                const int h = h0 + 8 * k;
+                if (h >= heads) break;
+                if (4 * lane < dp) store4(q + h * hw + 4 * lane, x[k]);
+                if (lane < half) rotated(h, lane, u[k], v[k], t);
+                pads(h);
+            }
+        }
+    } else {
+        for (int h = warp; h < heads; h += 8) {
+            const float* src = pr + h * hw;
+            for (int c = 4 * lane; c < dp; c += 128) store4(q + h * hw + c, load4(src + c));
+            for (int i = lane; i < half; i += 32) rotated(h, i, src[dp + i], src[dp + i + half], cs[i]);
+            pads(h);
         }
     }
-    for (int i = tid; i < half; i += 256) s_cs[i] = a.cs[(size_t)row * half + i];
-    const int hw = sh.dp + sh.rp, per = hw / 4;
-    T* q = static_cast<T*>(a.q) + (size_t)row * sh.heads * hw;
-    // unrotated parts: four columns at a time (hw and dp are multiples of 8)
-    const int n4 = sh.heads * per;
-#pragma unroll 4
-    for (int e = tid; e < n4; e += 256) {
-        const int h = e / per, c = 4 * (e - h * per);
-        if (c < sh.dp) store4(q + 4 * (size_t)e, load4(pr + 4 * (size_t)e));
+}
+
+// The cache row of a token: normed latent, rotated key part, zeros.
+template <typename T>
+__device__ __forceinline__ void latent_append(const LatentPreArgs& a, int row, int slot, int pos, const float* __restrict__ y, float* s_part) {
+    const int tid = threadIdx.x, rank = a.sh.rank, half = a.sh.rot / 2;
+    const int cap = a.cache.capacity[slot];
+    if (pos >= cap) {
+        if (tid == 0) atomicExch(a.cache.error, 2);                          // page not reserved: skip the write
+        return;
     }
-    __syncthreads();
-    // rotated parts, a pair (i, i + half) at a time; the padded columns behind are zero
-    for (int e = tid; e < sh.heads * half; e += 256) {
-        const int h = e / half, i = e - h * half;
-        const float* src = pr + h * hw + sh.dp;
-        const float u = src[i], v = src[i + half];
-        const float2 cs = s_cs[i];
-        const T ru = from_f32<T>(u * cs.x - v * cs.y), rv = from_f32<T>(v * cs.x + u * cs.y);
-        T* dst = q + h * hw + sh.dp;
-        dst[i] = ru;
-        dst[i + half] = rv;
-        if (a.qa) {
-            T* qa = static_cast<T*>(a.qa) + ((size_t)row * sh.heads + h) * sh.row_pitch() + sh.rank;
-            qa[i] = ru;
-            qa[i + half] = rv;
-        }
-    }
-    if (sh.rp > sh.rot) {
-        const int pad = sh.rp - sh.rot;
-        for (int e = tid; e < sh.heads * pad; e += 256) q[(e / pad) * hw + sh.dp + sh.rot + e % pad] = from_f32<T>(0.f);
-    }
-    if (a.qa) {                                                    // zero tail behind the rotated part
-        const int tail0 = sh.rank + sh.rot, tail = sh.row_pitch() - tail0;
-        T* qa = static_cast<T*>(a.qa) + (size_t)row * sh.heads * sh.row_pitch() + tail0;
-        for (int e = tid; e < sh.heads * tail; e += 256) qa[(e / tail) * sh.row_pitch() + e % tail] = from_f32<T>(0.f);
-    }
-    if (!sh.own) return;
+    const int page = a.cache.block_table[slot * a.cache.max_pages_per_seq + pos / kPageTokens];
+    float ss = 0.f;
+    for (int c = tid; c < rank; c += 256) ss += y[c] * y[c];
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     if ((tid & 31) == 0) s_part[tid >> 5] = ss;
     __syncthreads();
     ss = ((s_part[0] + s_part[1]) + (s_part[2] + s_part[3])) + ((s_part[4] + s_part[5]) + (s_part[6] + s_part[7]));
-    const float rms = sqrtf(ss / (float)sh.rank + sh.eps);
-    if (pos >= a.cache.capacity[slot]) {
-        if (tid == 0) atomicExch(a.cache.error, 2);                // page not reserved: skip the write
-        return;
-    }
-    const int page = a.cache.block_table[slot * a.cache.max_pages_per_seq + pos / kPageTokens];
-    T* dst = static_cast<T*>(a.cache.rows) + ((size_t)page * kPageTokens + pos % kPageTokens) * a.cache.pitch;
-#pragma unroll
-    for (int k = 0; k < kOwn; ++k) {
-        const int c = tid + 256 * k;
-        if (c < sh.rank) dst[c] = from_f32<T>(own[k] / rms * a.c_norm[c]);
-    }
+    const float rms = sqrtf(ss / (float)rank + a.sh.eps);
+    T* __restrict__ dst = static_cast<T*>(a.cache.rows) + ((size_t)page * kPageTokens + pos % kPageTokens) * a.cache.pitch;
+    for (int c = tid; c < rank; c += 256) dst[c] = from_f32<T>(y[c] / rms * a.c_norm[c]);
     for (int i = tid; i < half; i += 256) {
-        const float u = y[sh.rank + i], v = y[sh.rank + half + i];
-        const float2 cs = s_cs[i];
-        dst[sh.rank + i] = from_f32<T>(u * cs.x - v * cs.y);
-        dst[sh.rank + half + i] = from_f32<T>(v * cs.x + u * cs.y);
+        const float u = y[rank + i], v = y[rank + half + i];
+        const float2 t = a.cs[(size_t)row * half + i];
+        dst[rank + i] = from_f32<T>(u * t.x - v * t.y);
+        dst[rank + half + i] = from_f32<T>(v * t.x + u * t.y);
     }
-    for (int c = sh.rank + sh.rot + tid; c < a.cache.pitch; c += 256) dst[c] = from_f32<T>(0.f);
+    for (int c = rank + a.sh.rot + tid; c < a.cache.pitch; c += 256) dst[c] = from_f32<T>(0.f);
+}
+
+// grid (rows, 2 with latents of its own, else 1), block 256: queries, append.  A stream with little arithmetic: what counts
+// is how many loads are under way, hence the register bound.
+template <typename T, bool kSmallHead>
+__global__ void __launch_bounds__(256, 6)
+latent_pre_kernel(const LatentPreArgs a) {
+    __shared__ float s_part[8];
+    pdl_enter();
+    const int row = blockIdx.x, slot = a.row_slot[row];
+    if (slot < 0 || slot >= a.cache.max_seqs) return;
+    const float* pr = a.proj + (size_t)row * a.sh.pitch();
+    if (blockIdx.y == 0) latent_queries<T, kSmallHead>(a, row, pr);
+    else latent_append<T>(a, row, slot, a.row_pos[row], pr + a.sh.q_cols(), s_part);
 }
 
 int launch_latent_pre(ElemType t, const LatentPreArgs& a, int rows, cudaStream_t s) {
     dispatch_elem(t, [&](auto tag) {
         using T = decltype(tag);
-        launch_pdl(latent_pre_kernel<T>, dim3(rows), dim3(256), (size_t)(a.sh.rot / 2 + 1) * sizeof(float2), s, a);
+const bool small = a.sh.dp <= 128 && a.sh.rot <= 64;
+        launch_pdl(small ? latent_pre_kernel<T, true> : latent_pre_kernel<T, false>, dim3(rows, a.sh.own ? 2 : 1), dim3(256), 0, s, a);
     });
     B2_LAUNCH_CHECK();
     return 0;

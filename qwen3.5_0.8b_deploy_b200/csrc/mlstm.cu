@@ -170,72 +170,72 @@ int launch_mlstm_step(ElemType t, const MlstmStepArgs& a, int n, cudaStream_t s)
     return 0;
 }
 
-// The head's outputs over their root mean square, times the norm weight, times sigmoid(g).  A warp takes kUnits consecutive
-// (row, head) pairs and has all their loads under way before the first use (heads of up to 128 values; longer ones one by one).
+// The head's outputs over their root mean square, times the norm weight, times sigmoid(g).  One block per row, a warp takes
+// heads w, w + 8, ..; for heads of up to 128 values the loads of kUnits of them are under way before the first use.
 template <typename T, typename G>
 __global__ void __launch_bounds__(256)
 mlstm_head_norm_kernel(const float* __restrict__ core, const G* __restrict__ g, int g_pitch, int off_g, const float* __restrict__ norm_w,
-                       float eps, int heads, int vdim, int vp, int units, T* __restrict__ out) {
-    constexpr int kUnits = 4;
+                       float eps, int heads, int vdim, int vp, T* __restrict__ out) {
+    constexpr int kUnits = 2;
     pdl_enter();
-    const int u0 = ((blockIdx.x * 256 + threadIdx.x) >> 5) * kUnits, lane = threadIdx.x & 31;
-    auto gated = [](float x, float w, float z) { return x * w / (1.0f + expf(-z)); };
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const float* c = core + (size_t)blockIdx.x * heads * vp;
+    const G* gr = g + (size_t)blockIdx.x * g_pitch + off_g;
+    T* o = out + (size_t)blockIdx.x * heads * vp;
+    auto gated = [](float4 x, float inv, float4 w, float4 z) {
+        return make_float4(times_sigmoid<T>(x.x * inv * w.x, z.x), times_sigmoid<T>(x.y * inv * w.y, z.y), times_sigmoid<T>(x.z * inv * w.z, z.z),
+                           times_sigmoid<T>(x.w * inv * w.w, z.w));
+    };
     if (vp <= 128) {
         const int v = 4 * lane;
-        float4 x[kUnits], z[kUnits], w[kUnits];
-        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int h0 = warp; h0 < heads; h0 += 8 * kUnits) {
+            float4 x[kUnits], z[kUnits], w[kUnits];
+            const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-        for (int i = 0; i < kUnits; ++i) {
-            const int u = u0 + i, row = u / heads, h = u % heads;
-            const bool in = u < units && v < vp;                 // columns from vdim on are zero
-            x[i] = in ? __ldcs(reinterpret_cast<const float4*>(core + (size_t)u * vp + v)) : zero;
-            z[i] = in ? load4(g + (size_t)row * g_pitch + off_g + h * vp + v) : zero;
-            w[i] = in ? load4(norm_w + h * vp + v) : zero;
-        }
+            for (int i = 0; i < kUnits; ++i) {
+                const int h = h0 + 8 * i;
+                const bool in = h < heads && v < vp;              // columns from vdim on are zero
+                x[i] = in ? __ldcs(reinterpret_cast<const float4*>(c + h * vp + v)) : zero;
+                z[i] = in ? load4(gr + h * vp + v) : zero;
+                w[i] = in ? load4(norm_w + h * vp + v) : zero;
+            }
 #pragma unroll
-        for (int i = 0; i < kUnits; ++i) {
-            float ss = x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
+            for (int i = 0; i < kUnits; ++i) {
+                const int h = h0 + 8 * i;
+                float ss = x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
 #pragma unroll
-            for (int k = 16; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
-            const float inv = 1.0f / sqrtf(ss / (float)vdim + eps);
-            if (u0 + i < units && v < vp)
-                store4(out + (size_t)(u0 + i) * vp + v, make_float4(gated(x[i].x * inv, w[i].x, z[i].x), gated(x[i].y * inv, w[i].y, z[i].y),
-                                                                    gated(x[i].z * inv, w[i].z, z[i].z), gated(x[i].w * inv, w[i].w, z[i].w)));
+                for (int k = 16; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
+                const float inv = 1.0f / sqrtf(ss / (float)vdim + eps);
+                if (h < heads && v < vp) store4(o + h * vp + v, gated(x[i], inv, w[i], z[i]));
+            }
         }
         return;
     }
-    for (int u = u0; u < min(u0 + kUnits, units); ++u) {
-        const int row = u / heads, h = u % heads;
-        const float* c = core + (size_t)u * vp;
-        const G* gr = g + (size_t)row * g_pitch + off_g + h * vp;
+    for (int h = warp; h < heads; h += 8) {
         float ss = 0.f;
         for (int v = 4 * lane; v < vp; v += 128) {
-            const float4 x = load4(c + v);
+            const float4 x = load4(c + h * vp + v);
             ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
         }
 #pragma unroll
         for (int k = 16; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
         const float inv = 1.0f / sqrtf(ss / (float)vdim + eps);
-        for (int v = 4 * lane; v < vp; v += 128) {
-            const float4 x = load4(c + v), w = load4(norm_w + h * vp + v), z = load4(gr + v);
-            store4(out + (size_t)u * vp + v, make_float4(gated(x.x * inv, w.x, z.x), gated(x.y * inv, w.y, z.y), gated(x.z * inv, w.z, z.z),
-                                                         gated(x.w * inv, w.w, z.w)));
-        }
+        for (int v = 4 * lane; v < vp; v += 128)
+            store4(o + h * vp + v, gated(load4(c + h * vp + v), inv, load4(norm_w + h * vp + v), load4(gr + h * vp + v)));
     }
 }
 
 int launch_mlstm_head_norm(ElemType t, const MlstmShape& sh, const float* core, const void* g, bool g_f32, int g_pitch, const float* norm_w,
                            int rows, void* gated, cudaStream_t s) {
-    const int units = rows * sh.heads;
-    const dim3 grid(ceil_div(units, 32));
+    const dim3 grid(rows);
     dispatch_elem(t, [&](auto tag) {
         using T = decltype(tag);
         if (g_f32)
             launch_pdl(mlstm_head_norm_kernel<T, float>, grid, dim3(256), 0, s, core, (const float*)g, g_pitch, sh.off_g(), norm_w, sh.eps, sh.heads,
-                       sh.vdim, sh.vp, units, (T*)gated);
+                       sh.vdim, sh.vp, (T*)gated);
         else
             launch_pdl(mlstm_head_norm_kernel<T, T>, grid, dim3(256), 0, s, core, (const T*)g, g_pitch, sh.off_g(), norm_w, sh.eps, sh.heads, sh.vdim,
-                       sh.vp, units, (T*)gated);
+                       sh.vp, (T*)gated);
     });
     B2_LAUNCH_CHECK();
     return 0;

@@ -142,7 +142,7 @@ DTYPES = ["float32", "bfloat16"]
 MLSTM_SIZES = [(2, 64, 64), (2, 128, 128), (3, 40, 72), (1, 96, 160), (4, 16, 8), (1, 1, 1), (5, 24, 132), (2, 130, 20), (1, 300, 36), (1, 64, 256)]
 # heads, dim, rot, vdim, rank, window
 LATENT_SIZES = [(2, 64, 64, 64, 128, 70), (4, 128, 64, 128, 512, 130), (3, 40, 24, 56, 48, 17), (1, 16, 2, 8, 20, 1), (18, 32, 16, 24, 64, 64),
-                (2, 8, 40, 72, 30, 65), (2, 144, 32, 136, 96, 33), (1, 1, 2, 1, 1, 5), (2, 96, 32, 100, 256, 1000), (1, 64, 64, 192, 64, 40)]
+                (2, 8, 40, 72, 30, 65), (2, 144, 32, 136, 96, 33), (1, 1, 2, 1, 1, 5), (2, 96, 32, 100, 256, 1000), (1, 64, 64, 192, 64, 40), (2, 64, 32, 64, 64, 0), (33, 16, 16, 16, 300, 150)]
 
 
 # ---- each mechanism alone: a one-layer model without feed-forward -----------------------------------------------------------
