@@ -5,6 +5,7 @@ and prints its roofline line.  Sized by flags so the same command serves as a sm
     python kernel_bench.py --kernel fa_decode  --seqs 128 --ctx 1280 --kv fp16
     python kernel_bench.py --kernel fa_prefill --seqs 16  --ctx 1024
     python kernel_bench.py --kernel la_prefill --seqs 10  --ctx 1024
+    python kernel_bench.py --kernel mlstm_prefill  --seqs 16 --ctx 1024      # also mlstm_decode, latent_prefill, latent_decode
 
 Inputs are synthetic (unit-RMS q/k, N(0, 0.6) v, decays as in the model) and stay larger than L2 for the
 decode kernels by rotating over `--layers` independent caches.
@@ -45,9 +46,51 @@ def time_ms(fn, iters, warmup):
     return a.elapsed_time(b) / iters
 
 
+def measure_in_stack(kernel: str, seqs: int, ctx: int, iters: int, warmup: int) -> dict:
+    """mLSTM and latent-attention kernels inside a small stack (width 1024, 16 heads; one layer of each kind, layer sizes of
+    model_bench.py), timed by the library's own stamps and event pairs: prefill passes of all sequences, or eager decode steps
+    behind a prompt of `ctx` tokens."""
+    import importlib
+    import model_bench
+    ops = entry.load_ops()
+    models = importlib.import_module(entry.PKG_NAME + ".models")
+    case = dict(width=1024, ff=1024, vocab=1024, layers=4, batch=seqs, prompt=ctx, gen=0)
+    cfg = model_bench.nuzopel_config(case)
+    cfg["layers"] = cfg["layers"][2:4]
+    prefill = kernel.endswith("prefill")
+    st = models.build_model(cfg, models.Limits(seqs, ctx + iters + warmup + 1, 0, seqs * ctx if prefill else 8192, "bfloat16"))
+    models.load_tensors(st, entry.load_package().synth.nuzopel_tensors(cfg, 3))
+    cls = ("la_" if kernel.startswith("mlstm") else "fa_") + ("prefill" if prefill else "decode")
+    toks = torch.randint(0, 1024, (seqs, ctx), dtype=torch.int32, device="cuda")
+    with torch.cuda.stream(torch.cuda.Stream()):
+        nxt = None if prefill else st.forward_batch_prefill(toks)
+        for i in range(warmup + iters):
+            if i == warmup:
+                torch.cuda.synchronize()
+                ops.profile_reset(); ops.profile_enable(True)
+            if prefill:
+                st.reset_cache()
+                st.forward_batch_prefill(toks)
+            else:
+                nxt = st.forward_batch_decode(nxt)
+        torch.cuda.synchronize()
+        ms, n = ops.profile_read(cls)
+        ops.profile_enable(False); ops.profile_reset()
+    assert st.device_status() == 0
+    bound, work = model_bench.kernel_work("nuzopel", case)[cls]
+    hbm, tfl, src = peaks()
+    scale = 1e9 if bound == "hbm" else 1e12
+    out = dict(kernel=kernel, seqs=seqs, ctx=ctx, ms=ms / n, bound=bound, unit="GB/s" if bound == "hbm" else "TFLOP/s", peak=hbm if bound == "hbm" else tfl,
+               achieved=work / (ms / n * 1e-3) / scale, peak_source=src)
+    out["frac"] = out["achieved"] / out["peak"]
+    return out
+
+
 def measure(kernel: str, seqs: int = 128, ctx: int = 1024, kv: str = "fp16", layers: int = 4, iters: int = 20, warmup: int = 3,
             serial: bool = False) -> dict:
     """Times `iters` back-to-back launches of one kernel class on the current device and returns its roofline record."""
+    if kernel.startswith(("mlstm", "latent")):
+        return measure_in_stack(kernel, seqs, ctx, iters, warmup)
     args = argparse.Namespace(kernel=kernel, seqs=seqs, ctx=ctx, kv=kv, layers=layers, iters=iters, warmup=warmup, serial=serial)
     ops = entry.load_ops()
     g = torch.Generator(device="cuda").manual_seed(1)
@@ -127,7 +170,8 @@ def measure(kernel: str, seqs: int = 128, ctx: int = 1024, kv: str = "fp16", lay
 
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("--kernel", required=True, choices=["la_decode", "fa_decode", "fa_prefill", "la_prefill"])
+    ap.add_argument("--kernel", required=True, choices=["la_decode", "fa_decode", "fa_prefill", "la_prefill", "mlstm_prefill", "mlstm_decode",
+                                                        "latent_prefill", "latent_decode"])
     ap.add_argument("--seqs", type=int, default=128)
     ap.add_argument("--ctx", type=int, default=1024)
     ap.add_argument("--kv", default="fp16", choices=["fp16", "int8"])
