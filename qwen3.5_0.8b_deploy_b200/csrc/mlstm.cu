@@ -133,7 +133,8 @@ mlstm_step_kernel(const MlstmStepArgs a, unsigned long long* stamp) {
                 static_cast<T*>(a.gated)[row * (sh.heads * sh.vp) + h * sh.vp + vc] = from_f32<T>(r);
             }
         } else {
-            if (mine) a.core[row * (sh.heads * sh.vp) + h * sh.vp + vc] = o;
+            // padded columns too: the head norm reads whole rows, and the buffer holds what other layers left
+            if (tid < kMlstmTile && vc < sh.vp) a.core[row * (sh.heads * sh.vp) + h * sh.vp + vc] = o;
         }
         if (t + 1 < count) __syncthreads();       // s_q, s_k and the partial sums are free again
     }

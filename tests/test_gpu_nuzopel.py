@@ -311,6 +311,23 @@ def test_whole_model_portions(cuda, models, wts, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+def test_layers_of_different_sizes_share_the_working_buffers(cuda, models, wts, dtype):
+    """Layers whose padded sizes differ leave values where another layer's padding lies, and portions of one token use other
+    layouts than longer ones: neither may show."""
+    mixed = [mlstm(7, 8, 200, ff=40), latent(5, 40, 8, 72, 40, 50), mlstm(2, 128, 96), mlstm(3, 20, 130), latent(9, 8, 48, 24, 72, 33, ff=90), mlstm(1, 140, 300),
+             mlstm(4, 64, 40)]
+    c = Case(models, wts, *make(mixed, width=72, seed=31), dtype)
+    toks = c.tokens(180)
+    want = c.expect(toks)
+    with on_stream(cuda):
+        c.stack.begin_batching()
+        for cuts in ([180], [1], [60, 1, 1, 30, 2, 1], [180], [17, 1]):
+            row = c.stack.open()
+            c.judge(c.run(cuda, row, toks, cuts), want, f"cuts {cuts}")
+            c.stack.retire(row)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 def test_first_tokens_and_single_token(cuda, models, wts, dtype):
     c = Case(models, wts, *make(whole_layers(), seed=22), dtype)
     with on_stream(cuda):
