@@ -401,17 +401,28 @@ int b200attn_stack_step(b200attn_stack st, int n_rows, b200attn_stream stream);
 /* ------------------------------------------------------------------------------------------------
  * Stacks built from layer descriptions.
  * The same handle, caches, continuous batching and captured decode step as above, for models whose layers are given as a
- * list: every layer is x += norm1(mixer(x)), then (with a feed-forward) x += norm2(ff(x)), RMS norms with plain weights on
- * the sublayers' outputs; logits = embedding . norm(x) * logit_scale.  None of this has a counterpart in the reference.
+ * list: every layer is a mixer and (with ff > 0) a feed-forward, with RMS norms (plain weights) on the sublayers' outputs,
+ * x += norm1(mixer(x)), x += norm2(ff(x)), or on their inputs, x += mixer(norm1(x)), x += ff(norm2(x)).  A range of layers
+ * may run several times in a row with the same weights and caches of its own in every pass; the embedding output is added
+ * to x ahead of each pass but the first.  Logits: table . norm(x) * logit_scale, the table being the embedding or one of its
+ * own, then cap * tanh(. / cap) with a soft cap.  None of this has a counterpart in the reference.
  *
- * Mixers: B200ATTN_MIXER_MLSTM, a matrix memory with exponential gates (state per sequence and head: [dim][vdim], [dim],
- * one running maximum, fp32); B200ATTN_MIXER_LATENT, attention with keys and values up-projected from a cached latent of
- * kv_rank values and one rotated key part shared by all heads, over a sliding window.  A latent layer with kv_from >= 0
- * reads the cache of that earlier layer.
- * Feed-forward: down(gelu_tanh(gate x) * up x).
+ * Mixers
+ *   MLSTM          matrix memory with exponential gates (state per sequence and head: [dim][vdim], [dim], one running maximum, fp32)
+ *   LATENT         attention with keys and values up-projected from a cached latent of kv_rank values and one rotated key part
+ *                  shared by all heads, over a sliding window; with kv_from >= 0 it reads the cache of that earlier layer
+ *   LIGHTNING      matrix memory with one constant decay per head, silu on q, k and v (state [dim][vdim] per head, fp32); the
+ *                  concatenated heads are normed together and gated
+ *   CHANNEL_DELTA  gated delta rule with a decay per key channel: short convolutions on q, k and v, unit q and k, low-rank decay
+ *                  and output gates (state per head: [dim][vdim] and the convolutions' last inputs, fp32)
+ *   DIFF           differential attention: two softmax maps per head over the same values, combined as a1 - lambda a2, with
+ *                  normed and rotated q and k, over a sliding window plus the first keep_first positions
+ * Feed-forward: down(act(gate x) * up x).
  * ---------------------------------------------------------------------------------------------- */
 typedef enum { B200ATTN_DTYPE_BF16 = 0, B200ATTN_DTYPE_F32 = 1 } b200attn_dtype;
-typedef enum { B200ATTN_MIXER_MLSTM = 1, B200ATTN_MIXER_LATENT = 2 } b200attn_mixer;
+typedef enum { B200ATTN_MIXER_MLSTM = 1, B200ATTN_MIXER_LATENT = 2, B200ATTN_MIXER_LIGHTNING = 3, B200ATTN_MIXER_CHANNEL_DELTA = 4,
+               B200ATTN_MIXER_DIFF = 5 } b200attn_mixer;
+typedef enum { B200ATTN_ACT_GELU_TANH = 0, B200ATTN_ACT_SILU = 1 } b200attn_act;
 
 typedef struct {
     int width, vocab_size;
@@ -422,6 +433,10 @@ typedef struct {
     int max_pass_rows;     /* tokens per prefill pass (bounds the working buffers); longer prompts run in several passes */
     int dtype;             /* b200attn_dtype of weights, activations and cached latents                   */
     double norm_eps, embed_scale, logit_scale;
+    double logit_softcap;  /* 0 = none                                                                    */
+    int pre_norm;          /* 0: norms on the sublayers' outputs, 1: on their inputs                      */
+    int own_head;          /* 0: the embedding is the output table, 1: tensor "head"                      */
+    int loop_start, loop_stop, loop_times;   /* layers [start, stop) run `times` times; times <= 1: once  */
 } b200attn_model_config;
 
 typedef struct {
@@ -433,13 +448,22 @@ typedef struct {
     int kv_from;           /* index of the layer whose latents this one reads, -1 = its own                */
     double rot_base, scale;/* rotation base, score factor                                                  */
     int ff;                /* feed-forward size, 0 = no feed-forward                                       */
+    int act;               /* b200attn_act of the feed-forward                                            */
+    int kv_heads;          /* channel delta: q / k heads, diff: key / value heads; a divisor of heads      */
+    int conv_taps;         /* channel delta: taps of the short convolutions                                */
+    int a_rank, g_rank;    /* channel delta: inner sizes of the decay and output gates' projections        */
+    int keep_first;        /* diff: positions below it stay visible behind the window                      */
+    double diff;           /* diff: the constant of lambda and of the output factor                       */
+    const double* decay;   /* lightning: host array, one decay per head, read during creation              */
 } b200attn_layer_desc;
 
 /* Builds the stack: caches, state, working buffers, zeroed weights.  No reference counterpart. */
 int b200attn_stack_create_layers(const b200attn_model_config* cfg, const b200attn_layer_desc* layers, int num_layers, b200attn_stack* out);
 /* Gives one weight by name, host data in bf16 or fp32, row-major [rows, cols] (vectors: rows values, cols = 1).  Names:
- * "embed", "final.norm", and per layer i "l<i>.norm1", ".norm2", ".mlp.{gate,up,down}", ".mix.{q,k,v,g,o,norm,i,i.b,f,f.b}"
- * (mLSTM) or ".mix.{q,dkv,dkv.norm,uk,uv,o}" (latent).  A wrong name or shape is refused.  No reference counterpart. */
+ * "embed", "final.norm", "head", and per layer i "l<i>.norm1", ".norm2", ".mlp.{gate,up,down}", ".mix.{q,k,v,g,o,norm,i,i.b,f,f.b}"
+ * (mLSTM), ".mix.{q,dkv,dkv.norm,uk,uv,o}" (latent), ".mix.{q,k,v,g,o,norm}" (lightning), ".mix.{q,k,v}", ".mix.{q,k,v}.conv",
+ * ".mix.{b,a1,a2,dt_bias,A_log,g1,g2,norm,o}" (channel delta), ".mix.{q,k,v,q.norm,k.norm,lq1,lk1,lq2,lk2,o}" (diff).  A wrong
+ * name or shape is refused.  No reference counterpart. */
 int b200attn_stack_set_tensor(b200attn_stack st, const char* name, const void* h_data, int dtype, long long rows, long long cols);
 /* Admits a sequence without running a prompt (continuous batching): takes a slot and a row, reserves pages for
  * reserve_tokens (may be 0: they are reserved as the sequence grows), clears its state.  No reference counterpart. */
@@ -450,7 +474,7 @@ int b200attn_stack_open(b200attn_stack st, int reserve_tokens, int* row_out, b20
 int b200attn_stack_extend(b200attn_stack st, int row, const int* d_tokens, int n_tokens, const int* h_want, int n_want, float* d_logits,
                           int* d_next, b200attn_stream stream);
 /* The residual stream of the last pass's rows (fp32 [rows, width]; rows = 0: none), for checks of single layers:
- * stop_after >= 0 makes the following passes end behind that many layers, -1 runs all again, -2 changes nothing.
+ * stop_after >= 0 makes the following passes end behind that many layer runs, -1 runs all again, -2 changes nothing.
  * No reference counterpart. */
 int b200attn_stack_residual(b200attn_stack st, int rows, float* d_out, int stop_after, b200attn_stream stream);
 

@@ -1,8 +1,10 @@
 // Element-wise kernels of layer-described models: scaled embedding, RMS norm on a sublayer's output with the residual add,
-// gelu-gated products, and the row bookkeeping of a pass.  Any width; four values per thread and access where it divides.
+// gated products, soft caps, and the row bookkeeping of a pass.  Any width; four values per thread and access where it divides.
 #include "block_model.cuh"
 #include "elem.cuh"
 #include "ptx_utils.cuh"
+
+#include <algorithm>
 
 namespace b200 {
 
@@ -150,16 +152,84 @@ int launch_rms_norm_rows(ElemType t, const float* x, const int* row_index, const
     return 0;
 }
 
+// x += add (a repeated pass starts so), out = x / rms * w.  One block per row.
+template <typename T, bool kAdd>
+__global__ void __launch_bounds__(128)
+pre_norm_kernel(float* __restrict__ x, const float* __restrict__ add, const float* __restrict__ w, float eps, int width, T* __restrict__ out) {
+    __shared__ float s_part[4];
+    pdl_enter();
+    const size_t at = (size_t)blockIdx.x * width;
+    if ((width & 3) == 0 && width <= 2048) {
+        float4 v[4];
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int c = 4 * (threadIdx.x + 128 * i);
+            v[i] = c < width ? *reinterpret_cast<const float4*>(x + at + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            if (kAdd && c < width) {
+                const float4 e = *reinterpret_cast<const float4*>(add + at + c);
+                v[i] = make_float4(v[i].x + e.x, v[i].y + e.y, v[i].z + e.z, v[i].w + e.w);
+                *reinterpret_cast<float4*>(x + at + c) = v[i];
+            }
+            ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+        }
+        const float rms = sqrtf(block_sum128(ss, s_part) / (float)width + eps);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int c = 4 * (threadIdx.x + 128 * i);
+            if (c >= width) break;
+            const float4 ww = *reinterpret_cast<const float4*>(w + c);
+            store4(out + at + c, make_float4(v[i].x / rms * ww.x, v[i].y / rms * ww.y, v[i].z / rms * ww.z, v[i].w / rms * ww.w));
+        }
+        return;
+    }
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < width; c += 128) {
+        float v = x[at + c];
+        if (kAdd) { v += add[at + c]; x[at + c] = v; }
+        ss += v * v;
+    }
+    const float rms = sqrtf(block_sum128(ss, s_part) / (float)width + eps);
+    for (int c = threadIdx.x; c < width; c += 128) out[at + c] = from_f32<T>(x[at + c] / rms * w[c]);
+}
+
+int launch_pre_norm(ElemType t, float* x, const float* add, const float* w, float eps, int rows, int width, void* out, cudaStream_t s) {
+    dispatch_elem(t, [&](auto tag) {
+        using T = decltype(tag);
+        launch_pdl(add ? pre_norm_kernel<T, true> : pre_norm_kernel<T, false>, dim3(rows), dim3(128), 0, s, x, add, w, eps, width, (T*)out);
+    });
+    B2_LAUNCH_CHECK();
+    return 0;
+}
+
+__global__ void __launch_bounds__(256)
+softcap_kernel(float* __restrict__ p, size_t n, float cap) {
+    pdl_enter();
+    for (size_t i = (size_t)blockIdx.x * 256 + threadIdx.x; i < n; i += (size_t)gridDim.x * 256) p[i] = cap * tanhf(p[i] / cap);
+}
+
+int launch_softcap(float* logits, size_t n, float cap, cudaStream_t s) {
+    launch_pdl(softcap_kernel, dim3((unsigned)std::min<size_t>((n + 255) / 256, 148 * 16)), dim3(256), 0, s, logits, n, cap);
+    B2_LAUNCH_CHECK();
+    return 0;
+}
+
 // 0.5 z (1 + tanh y) = z / (1 + e^{-2y}), y = sqrt(2 / pi) (z + 0.044715 z^3)
 template <typename T>
 __device__ __forceinline__ float gelu_tanh(float z) {
     return times_sigmoid<T>(z, 1.5957691216057308f * (z + 0.044715f * z * z * z));
 }
 
+template <typename T, int kAct>
+__device__ __forceinline__ float activated(float z) {
+    if constexpr (kAct == B200ATTN_ACT_SILU) return times_sigmoid<T>(z, z);
+    else return gelu_tanh<T>(z);
+}
+
 // Blocks of 128 threads: one per row, or (few rows) several along it.
-template <typename T>
+template <typename T, int kAct>
 __global__ void __launch_bounds__(128)
-gelu_mul_kernel(const T* __restrict__ gu, int ff, T* __restrict__ act) {
+act_mul_kernel(const T* __restrict__ gu, int ff, T* __restrict__ act) {
     pdl_enter();
     const T* g = gu + (size_t)blockIdx.x * 2 * ff;
     T* o = act + (size_t)blockIdx.x * ff;
@@ -167,17 +237,17 @@ gelu_mul_kernel(const T* __restrict__ gu, int ff, T* __restrict__ act) {
 #pragma unroll 4
         for (int c = 4 * (threadIdx.x + 128 * blockIdx.y); c < ff; c += 512 * gridDim.y) {
             const float4 a = load4(g + c), u = load4(g + ff + c);
-            store4(o + c, make_float4(gelu_tanh<T>(a.x) * u.x, gelu_tanh<T>(a.y) * u.y, gelu_tanh<T>(a.z) * u.z, gelu_tanh<T>(a.w) * u.w));
+            store4(o + c, make_float4(activated<T, kAct>(a.x) * u.x, activated<T, kAct>(a.y) * u.y, activated<T, kAct>(a.z) * u.z, activated<T, kAct>(a.w) * u.w));
         }
         return;
     }
-    for (int c = threadIdx.x + 128 * blockIdx.y; c < ff; c += 128 * gridDim.y) o[c] = from_f32<T>(gelu_tanh<T>(to_f32(g[c])) * to_f32(g[ff + c]));
+    for (int c = threadIdx.x + 128 * blockIdx.y; c < ff; c += 128 * gridDim.y) o[c] = from_f32<T>(activated<T, kAct>(to_f32(g[c])) * to_f32(g[ff + c]));
 }
 
-int launch_gelu_mul(ElemType t, const void* gu, int rows, int ff, void* act, cudaStream_t s) {
+int launch_act_mul(ElemType t, int f, const void* gu, int rows, int ff, void* act, cudaStream_t s) {
     dispatch_elem(t, [&](auto tag) {
         using T = decltype(tag);
-        launch_pdl(gelu_mul_kernel<T>, dim3(rows, rows < 1024 ? ceil_div(ff, 512) : 1), dim3(128), 0, s, (const T*)gu, ff, (T*)act);
+        launch_pdl(f == B200ATTN_ACT_SILU ? act_mul_kernel<T, B200ATTN_ACT_SILU> : act_mul_kernel<T, B200ATTN_ACT_GELU_TANH>, dim3(rows, rows < 1024 ? ceil_div(ff, 512) : 1), dim3(128), 0, s, (const T*)gu, ff, (T*)act);
     });
     B2_LAUNCH_CHECK();
     return 0;

@@ -1,4 +1,4 @@
-// Layer-described models: construction from descriptions, weights by name, and the layer loop over the mixers.
+// Layer-described models: construction from descriptions, weights by name, the layer loop, and the mixers with norms on their outputs.
 #include "stack.cuh"
 #include "elem.cuh"
 
@@ -51,6 +51,16 @@ static int make_latent(const b200attn_layer_desc& d, const b200attn_model_config
     return 0;
 }
 
+// Index of a rotation's table, added where no layer before has it.
+static int rot_table(BlockModel& m, double base, int half) {
+    for (size_t k = 0; k < m.rot.size(); ++k)
+        if (m.rot[k].base == base && m.rot[k].half == half) return (int)k;
+    m.rot.emplace_back();
+    m.rot.back().base = base;
+    m.rot.back().half = half;
+    return (int)m.rot.size() - 1;
+}
+
 int block_model_create(const b200attn_model_config* cfg, const b200attn_layer_desc* layers, int num_layers, b200attn_stack st) {
     B2_CHECK_ARG(cfg->dtype == B200ATTN_DTYPE_BF16 || cfg->dtype == B200ATTN_DTYPE_F32, "model: bad dtype");
     st->blocks.reset(new (std::nothrow) BlockModel());
@@ -63,12 +73,10 @@ int block_model_create(const b200attn_model_config* cfg, const b200attn_layer_de
     m.max_rows = std::max(cfg->max_seqs, cfg->max_pass_rows > 0 ? cfg->max_pass_rows : (int)std::min(all, 8192ll));
     st->max_rows = m.max_rows;
 
-    std::vector<size_t> state_floats;
-    std::vector<int> row_pitch;
     m.layers.resize(num_layers);
     m.missing = {"embed", "final.norm"};
-    size_t proj = 0, mixed = 0, core = 0, gates = 0, ff = 0, q = 0, qa = 0, olat = 0, cst = 0, rst = 0, kup = 0, vup = 0, part = 0, counters = 0;
-    int max_window = 0;
+    if (cfg->own_head) m.missing.push_back("head");
+    BlockSizes z;
     for (int i = 0; i < num_layers; ++i) {
         const b200attn_layer_desc& d = layers[i];
         BlockLayer& L = m.layers[i];
@@ -78,68 +86,95 @@ int block_model_create(const b200attn_model_config* cfg, const b200attn_layer_de
             L.mlstm.reset(new MlstmOp());
             B2_TRY(make_mlstm(d, *cfg, m.elem, *L.mlstm));
             const MlstmShape& sh = L.mlstm->sh;
-            L.mlstm->state_layer = (int)state_floats.size();
-            state_floats.push_back(sh.state_floats());
-            proj = std::max(proj, (size_t)sh.pitch());
-            mixed = std::max(mixed, (size_t)sh.heads * sh.vp);
-            if (L.mlstm->chunk || sh.n_vt > 1) core = std::max(core, (size_t)sh.heads * sh.vp);
-            if (L.mlstm->chunk) gates = std::max(gates, (size_t)2 * sh.heads);
+            z.proj = std::max(z.proj, (size_t)sh.pitch());
+            z.mixed = std::max(z.mixed, (size_t)sh.heads * sh.vp);
+            if (L.mlstm->chunk || sh.n_vt > 1) z.core = std::max(z.core, (size_t)sh.heads * sh.vp);
+            if (L.mlstm->chunk) z.gates = std::max(z.gates, (size_t)2 * sh.heads);
             for (const char* n : {"mix.q", "mix.k", "mix.v", "mix.g", "mix.o", "mix.norm", "mix.i", "mix.i.b", "mix.f", "mix.f.b"}) need(n);
         } else if (d.mixer == B200ATTN_MIXER_LATENT) {
             L.latent.reset(new LatentOp());
             LatentOp& op = *L.latent;
             B2_TRY(make_latent(d, *cfg, m.elem, op));
             const LatentShape& sh = op.sh;
+            op.kv_from = d.kv_from;
             if (sh.own) {
-                op.pool_layer = (int)row_pitch.size();
-                row_pitch.push_back(sh.row_pitch());
                 for (const char* n : {"mix.dkv", "mix.dkv.norm"}) need(n);
             } else {
                 B2_CHECK_ARG(d.kv_from < i && m.layers[d.kv_from].latent && m.layers[d.kv_from].latent->sh.own,
                              "layer %d: kv_from %d is not an earlier layer with latents of its own", i, d.kv_from);
                 const LatentShape& src = m.layers[d.kv_from].latent->sh;
                 B2_CHECK_ARG(src.rank == sh.rank && src.rot == sh.rot, "layer %d: kv_rank and rot_dim differ from those of layer %d", i, d.kv_from);
-                op.pool_layer = m.layers[d.kv_from].latent->pool_layer;
             }
             for (const char* n : {"mix.q", "mix.uk", "mix.uv", "mix.o"}) need(n);
-            op.rot_table = -1;
-            for (size_t k = 0; k < m.rot.size(); ++k)
-                if (m.rot[k].base == d.rot_base && m.rot[k].half == sh.rot / 2) op.rot_table = (int)k;
-            if (op.rot_table < 0) {
-                op.rot_table = (int)m.rot.size();
-                m.rot.emplace_back();
-                m.rot.back().base = d.rot_base;
-                m.rot.back().half = sh.rot / 2;
-            }
-            proj = std::max(proj, (size_t)sh.pitch());
-            mixed = std::max(mixed, (size_t)sh.heads * sh.vp);
-            q = std::max(q, (size_t)sh.q_cols());
-            qa = std::max(qa, (size_t)sh.heads * sh.row_pitch());
-            olat = std::max(olat, (size_t)sh.heads * sh.rank);
+            op.rot_table = rot_table(m, d.rot_base, sh.rot / 2);
+            z.proj = std::max(z.proj, (size_t)sh.pitch());
+            z.mixed = std::max(z.mixed, (size_t)sh.heads * sh.vp);
+            z.q = std::max(z.q, (size_t)sh.q_cols());
+            z.qa = std::max(z.qa, (size_t)sh.heads * sh.row_pitch());
+            z.olat = std::max(z.olat, (size_t)sh.heads * sh.rank);
             if (op.tc_prefill) {
-                cst = std::max(cst, (size_t)sh.rank); rst = std::max(rst, (size_t)sh.rp);
-                kup = std::max(kup, (size_t)sh.heads * sh.dp); vup = std::max(vup, (size_t)sh.heads * sh.vp);
-                max_window = std::max(max_window, sh.window > 0 ? std::min(sh.window, cfg->max_seq_len) : cfg->max_seq_len);
+                z.cst = std::max(z.cst, (size_t)sh.rank); z.rst = std::max(z.rst, (size_t)sh.rp);
+                z.kup = std::max(z.kup, (size_t)sh.heads * sh.dp); z.vup = std::max(z.vup, (size_t)sh.heads * sh.vp);
+                z.max_window = std::max(z.max_window, sh.window > 0 ? std::min(sh.window, cfg->max_seq_len) : cfg->max_seq_len);
             }
             if (op.tc_decode) {
-                part = std::max(part, latent_decode_scratch_floats(sh, cfg->max_seqs));
-                counters = std::max(counters, (size_t)cfg->max_seqs * ceil_div(sh.heads, 16));
+                z.part = std::max(z.part, latent_decode_scratch_floats(sh, cfg->max_seqs));
+                z.counters = std::max(z.counters, (size_t)cfg->max_seqs * ceil_div(sh.heads, 16));
             }
+        } else if (d.mixer == B200ATTN_MIXER_LIGHTNING) {
+            L.mlstm.reset(new MlstmOp());
+            B2_TRY(make_lightning(d, *cfg, m.elem, *L.mlstm, z));
+            for (const char* n : {"mix.q", "mix.k", "mix.v", "mix.g", "mix.o", "mix.norm"}) need(n);
+        } else if (d.mixer == B200ATTN_MIXER_CHANNEL_DELTA) {
+            L.delta.reset(new DeltaOp());
+            B2_TRY(make_delta(d, *cfg, m.elem, *L.delta, z));
+            for (const char* n : {"mix.q", "mix.q.conv", "mix.k", "mix.k.conv", "mix.v", "mix.v.conv", "mix.b", "mix.A_log", "mix.norm", "mix.a1", "mix.a2",
+                                  "mix.dt_bias", "mix.g1", "mix.g2", "mix.o"}) need(n);
+        } else if (d.mixer == B200ATTN_MIXER_DIFF) {
+            L.diff.reset(new DiffOp());
+            B2_TRY(make_diff(d, *cfg, m.elem, *L.diff, z));
+            L.diff->rot_table = rot_table(m, d.rot_base, d.rot_dim / 2);
+            for (const char* n : {"mix.q", "mix.k", "mix.v", "mix.q.norm", "mix.k.norm", "mix.lq1", "mix.lk1", "mix.lq2", "mix.lk2", "mix.o"}) need(n);
         } else {
             B2_FAIL(B200ATTN_ERR_INVALID, "layer %d: unknown mixer %d", i, d.mixer);
         }
         B2_TRY(L.norm1.alloc(W * 4));
+        B2_CHECK_ARG(d.act == B200ATTN_ACT_GELU_TANH || d.act == B200ATTN_ACT_SILU, "layer %d: unknown activation %d", i, d.act);
         L.ff = d.ff;
+        L.act = d.act;
         if (d.ff > 0) {
             B2_TRY(L.norm2.alloc(W * 4));
             B2_TRY(L.w_gu.alloc((size_t)2 * d.ff * W * e));
             B2_TRY(L.w_down.alloc((size_t)d.ff * W * e));
-            ff = std::max(ff, (size_t)d.ff);
+            z.ff = std::max(z.ff, (size_t)d.ff);
             for (const char* n : {"norm2", "mlp.gate", "mlp.up", "mlp.down"}) need(n);
         }
     }
+
+    // The layers in the order they run; every run has its own state and cache.
+    const int times = std::max(1, cfg->loop_times), start = times > 1 ? cfg->loop_start : 0, stop = times > 1 ? cfg->loop_stop : 0;
+    B2_CHECK_ARG(times == 1 || (0 <= start && start < stop && stop <= num_layers), "model: loop over layers [%d, %d) of %d", start, stop, num_layers);
+    if (times > 1 && !cfg->pre_norm) B2_FAIL(B200ATTN_ERR_UNSUPPORTED, "model: loops need norms on the sublayers' inputs");
+    auto run = [&](int i, bool again) { m.runs.emplace_back(); m.runs.back().layer = i; m.runs.back().add_embedding = again; };
+    for (int i = 0; i < start; ++i) run(i, false);
+    for (int t = 0; t < times; ++t)
+        for (int i = start; i < stop; ++i) run(i, t > 0 && i == start);
+    for (int i = stop; i < num_layers; ++i) run(i, false);
+    std::vector<size_t> state_floats;
+    std::vector<int> row_pitch, last_pool_layer(num_layers, -1);
+    for (LayerRun& r : m.runs) {
+        BlockLayer& L = m.layers[r.layer];
+        auto state = [&](size_t n) { r.state_layer = (int)state_floats.size(); state_floats.push_back(n); };
+        auto cache = [&](int pitch) { r.pool_layer = last_pool_layer[r.layer] = (int)row_pitch.size(); row_pitch.push_back(pitch); };
+        if (L.mlstm) state(L.mlstm->sh.state_floats());
+        if (L.delta) state(L.delta->sh.state_floats());
+        if (L.diff) cache(L.diff->sh.row_pitch());
+        if (L.latent && L.latent->sh.own) cache(L.latent->sh.row_pitch());
+        if (L.latent && !L.latent->sh.own) r.pool_layer = last_pool_layer[L.latent->kv_from];     // its source's latest run
+    }
     B2_TRY(m.embed.alloc((size_t)cfg->vocab_size * W * e));
     B2_TRY(m.final_norm.alloc(W * 4));
+    if (cfg->own_head) B2_TRY(m.head.alloc((size_t)cfg->vocab_size * W * e));
 
     if (!state_floats.empty()) B2_TRY(state_pool_create_blocks(state_floats, cfg->max_seqs, &st->state));
     if (!row_pitch.empty()) {
@@ -155,7 +190,7 @@ int block_model_create(const b200attn_model_config* cfg, const b200attn_layer_de
 
     const size_t R = m.max_rows;
     m.abs_rows = (int)std::min<size_t>(R, std::max(4096, cfg->max_seqs));
-    m.ctx_rows = (int)R + max_window;
+    m.ctx_rows = (int)R + z.max_window;
     m.max_spans = (int)std::max<size_t>(cfg->max_seqs, 1);
     for (RotTable& t : m.rot) {
         std::vector<double> f(std::max(1, t.half));
@@ -165,23 +200,25 @@ int block_model_create(const b200attn_model_config* cfg, const b200attn_layer_de
         B2_TRY(t.cs.alloc(R * f.size() * sizeof(float2)));
     }
     B2_TRY(m.x.alloc(R * W * 4));
+    if (times > 1) B2_TRY(m.x0.alloc(R * W * 4));
     B2_TRY(m.xt.alloc(R * W * e));
-    B2_TRY(m.y.alloc(R * W * 4));
-    B2_TRY(m.proj.alloc(R * proj * 4));
-    B2_TRY(m.gates.alloc(R * gates * 4));
-    B2_TRY(m.core.alloc(R * core * 4));
-    B2_TRY(m.mixed.alloc(R * mixed * e));
-    B2_TRY(m.gu.alloc(R * 2 * ff * e));
-    B2_TRY(m.act.alloc(R * ff * e));
-    B2_TRY(m.q.alloc(R * q * e));
-    B2_TRY(m.qa.alloc((size_t)m.abs_rows * qa * e));
-    B2_TRY(m.olat.alloc((size_t)m.abs_rows * olat * e));
-    B2_TRY(m.c_stage.alloc((size_t)m.ctx_rows * cst * e));
-    B2_TRY(m.r_stage.alloc((size_t)m.ctx_rows * rst * e));
-    B2_TRY(m.k_up.alloc((size_t)m.ctx_rows * kup * e));
-    B2_TRY(m.v_up.alloc((size_t)m.ctx_rows * vup * e));
-    B2_TRY(m.part.alloc(part * 4));
-    B2_TRY(m.counters.alloc(counters * 4));
+    if (!cfg->pre_norm) B2_TRY(m.y.alloc(R * W * 4));
+    B2_TRY(m.proj.alloc(R * z.proj * 4));
+    B2_TRY(m.gates.alloc(R * z.gates * 4));
+    B2_TRY(m.low.alloc(R * z.low * e));
+    B2_TRY(m.core.alloc(R * z.core * 4));
+    B2_TRY(m.mixed.alloc(R * z.mixed * e));
+    B2_TRY(m.gu.alloc(R * 2 * z.ff * e));
+    B2_TRY(m.act.alloc(R * z.ff * e));
+    B2_TRY(m.q.alloc(R * z.q * e));
+    B2_TRY(m.qa.alloc((size_t)m.abs_rows * z.qa * e));
+    B2_TRY(m.olat.alloc((size_t)m.abs_rows * z.olat * e));
+    B2_TRY(m.c_stage.alloc((size_t)m.ctx_rows * z.cst * e));
+    B2_TRY(m.r_stage.alloc((size_t)m.ctx_rows * z.rst * e));
+    B2_TRY(m.k_up.alloc((size_t)m.ctx_rows * z.kup * e));
+    B2_TRY(m.v_up.alloc((size_t)m.ctx_rows * z.vup * e));
+    B2_TRY(m.part.alloc(z.part * 4));
+    B2_TRY(m.counters.alloc(z.counters * 4));
     const size_t tiles = R / 128 + m.max_spans + 1;
     B2_TRY(m.meta.alloc((2 * R + 7 * (size_t)m.max_spans + 5 * tiles) * 4));
     return m.error.alloc(4);
@@ -202,26 +239,11 @@ int block_model_status(BlockModel& m, int* code) {
 }
 
 // ---- weights by name ---------------------------------------------------------------------------------------------------------
-namespace {
-struct Source {
-    const void* data;
-    bool f32;
-    long long rows, cols;
-    float at(size_t i) const {
-        if (f32) return static_cast<const float*>(data)[i];
-        const uint32_t u = (uint32_t)static_cast<const uint16_t*>(data)[i] << 16;
-        float v;
-        std::memcpy(&v, &u, 4);
-        return v;
-    }
-};
-
 int check_shape(const Source& t, const char* name, long long rows, long long cols) {
     B2_CHECK_ARG(t.rows == rows && t.cols == cols, "tensor '%s': shape [%lld, %lld], expected [%lld, %lld]", name, t.rows, t.cols, rows, cols);
     return 0;
 }
 
-// Copies a [rows, cols] block of the source to (row0, col0) of a device matrix with row pitch ld.
 int put(DevBuf& dst, ElemType elem, size_t ld, size_t row0, size_t col0, const Source& t, size_t src_row, size_t src_col, size_t rows, size_t cols) {
     const size_t e = elem_bytes(elem);
     std::vector<char> h(rows * cols * e);
@@ -245,9 +267,7 @@ int put_vector(DevBuf& dst, const char* name, const Source& t, size_t at, long l
     return put(dst, ELEM_F32, 1, at, 0, t, 0, 0, n, 1);
 }
 
-// [heads * size, in] rows into rows of padded heads.
-int put_heads(DevBuf& dst, ElemType elem, size_t row0, int stride, const char* name, const Source& t, int heads, int size, int in, int src_stride,
-              int src_off) {
+int put_heads(DevBuf& dst, ElemType elem, size_t row0, int stride, const Source& t, int heads, int size, int in, int src_stride, int src_off) {
     for (int h = 0; h < heads; ++h) B2_TRY(put(dst, elem, in, row0 + (size_t)h * stride, 0, t, (size_t)h * src_stride + src_off, 0, size, in));
     return 0;
 }
@@ -258,12 +278,13 @@ int put_out(DevBuf& dst, ElemType elem, const char* name, const Source& t, int w
     return 0;
 }
 
+namespace {
 int set_mlstm(MlstmOp& op, const std::string& n, const char* name, const Source& t) {
     const MlstmShape& sh = op.sh;
     const int W = op.width, H = sh.heads;
     auto heads = [&](int row0, int stride, int size) -> int {
         B2_TRY(check_shape(t, name, (long long)H * size, W));
-        return put_heads(op.w_in, op.elem, row0, stride, name, t, H, size, W, size, 0);
+        return put_heads(op.w_in, op.elem, row0, stride, t, H, size, W, size, 0);
     };
     if (n == "q") return heads(sh.off_q(), sh.dp, sh.dim);
     if (n == "k") return heads(sh.off_k(), sh.dp, sh.dim);
@@ -287,8 +308,8 @@ int set_latent(LatentOp& op, const std::string& n, const char* name, const Sourc
     const int W = op.width, H = sh.heads;
     if (n == "q") {
         B2_TRY(check_shape(t, name, (long long)H * (sh.dim + sh.rot), W));
-        B2_TRY(put_heads(op.w_in, op.elem, 0, sh.dp + sh.rp, name, t, H, sh.dim, W, sh.dim + sh.rot, 0));
-        return put_heads(op.w_in, op.elem, sh.dp, sh.dp + sh.rp, name, t, H, sh.rot, W, sh.dim + sh.rot, sh.dim);
+        B2_TRY(put_heads(op.w_in, op.elem, 0, sh.dp + sh.rp, t, H, sh.dim, W, sh.dim + sh.rot, 0));
+        return put_heads(op.w_in, op.elem, sh.dp, sh.dp + sh.rp, t, H, sh.rot, W, sh.dim + sh.rot, sh.dim);
     }
     if (n == "dkv" && sh.own) {
         B2_TRY(check_shape(t, name, sh.rank + sh.rot, W));
@@ -297,11 +318,11 @@ int set_latent(LatentOp& op, const std::string& n, const char* name, const Sourc
     if (n == "dkv.norm" && sh.own) return put_vector(op.c_norm, name, t, 0, sh.rank);
     if (n == "uk") {
         B2_TRY(check_shape(t, name, (long long)H * sh.dim, sh.rank));
-        return put_heads(op.w_uk, op.elem, 0, sh.dp, name, t, H, sh.dim, sh.rank, sh.dim, 0);
+        return put_heads(op.w_uk, op.elem, 0, sh.dp, t, H, sh.dim, sh.rank, sh.dim, 0);
     }
     if (n == "uv") {
         B2_TRY(check_shape(t, name, (long long)H * sh.vdim, sh.rank));
-        return put_heads(op.w_uv, op.elem, 0, sh.vp, name, t, H, sh.vdim, sh.rank, sh.vdim, 0);
+        return put_heads(op.w_uv, op.elem, 0, sh.vp, t, H, sh.vdim, sh.rank, sh.vdim, 0);
     }
     if (n == "o") return put_out(op.w_out, op.elem, name, t, W, H, sh.vdim, sh.vp);
     B2_FAIL(B200ATTN_ERR_INVALID, "tensor '%s': this latent-attention layer has no such tensor", name);
@@ -311,9 +332,9 @@ int set_tensor(BlockModel& m, const char* name, const Source& t) {
     const int W = m.cfg.width;
     auto given = [](std::vector<std::string>& missing, const std::string& n) { missing.erase(std::remove(missing.begin(), missing.end(), n), missing.end()); };
     const std::string full = name;
-    if (full == "embed") {
+    if (full == "embed" || (full == "head" && m.cfg.own_head)) {
         B2_TRY(check_shape(t, name, m.cfg.vocab_size, W));
-        B2_TRY(put(m.embed, m.elem, W, 0, 0, t, 0, 0, t.rows, W));
+        B2_TRY(put(full == "head" ? m.head : m.embed, m.elem, W, 0, 0, t, 0, 0, t.rows, W));
         given(m.missing, full);
         return 0;
     }
@@ -336,7 +357,11 @@ int set_tensor(BlockModel& m, const char* name, const Source& t) {
         B2_TRY(check_shape(t, name, W, L.ff));
         B2_TRY(put(L.w_down, m.elem, L.ff, 0, 0, t, 0, 0, W, L.ff));
     } else if (n.rfind("mix.", 0) == 0) {
-        B2_TRY(L.mlstm ? set_mlstm(*L.mlstm, n.substr(4), name, t) : set_latent(*L.latent, n.substr(4), name, t));
+        const std::string w = n.substr(4);
+        if (L.mlstm) B2_TRY(L.mlstm->sh.gated ? set_mlstm(*L.mlstm, w, name, t) : set_lightning(*L.mlstm, w, name, t));
+        else if (L.delta) B2_TRY(set_delta(*L.delta, w, name, t));
+        else if (L.diff) B2_TRY(set_diff(*L.diff, w, name, t));
+        else B2_TRY(set_latent(*L.latent, w, name, t));
     } else {
         B2_FAIL(B200ATTN_ERR_INVALID, "tensor '%s': unknown name", name);
     }
@@ -346,11 +371,10 @@ int set_tensor(BlockModel& m, const char* name, const Source& t) {
 }  // namespace
 
 // ---- layer loop ---------------------------------------------------------------------------------------------------------------
-static int mlstm_forward(BlockModel& m, MlstmOp& op, const PassRows& p, cudaStream_t s) {
+static int mlstm_forward(BlockModel& m, MlstmOp& op, const LayerRun& run, const PassRows& p, cudaStream_t s) {
     const MlstmShape& sh = op.sh;
     const int W = m.cfg.width;
-    float* state = m.state->d_recurrent + m.state->block_offset[op.state_layer];
-    const int vcols = sh.heads * sh.vp;
+    float* state = m.state->d_recurrent + m.state->block_offset[run.state_layer];
     if (!p.decode && op.chunk && p.max_count >= 16) {
         // q | k | v | g in bf16 for the tensor cores, the gate pre-activations in fp32
         B2_TRY(gemm_typed(s, m.xt.p, W, op.w_in.p, m.proj.p, sh.cols(), op.elem, ELEM_BF16, p.rows, sh.cols(), W));
@@ -370,7 +394,7 @@ static int mlstm_forward(BlockModel& m, MlstmOp& op, const PassRows& p, cudaStre
         if (sh.n_vt > 1)
             B2_TRY(launch_mlstm_head_norm(op.elem, sh, m.core.f(), m.proj.p, true, sh.pitch(), op.norm_w.f(), p.rows, m.mixed.p, s));
     }
-    return gemm_typed(s, m.mixed.p, vcols, op.w_out.p, m.y.p, W, op.elem, ELEM_F32, p.rows, W, vcols);
+    return 0;
 }
 
 // Attention with the up-projections absorbed into the queries and outputs: decode, and prefill in blocks of rows.
@@ -404,7 +428,7 @@ static LatentSpan context_span(const LatentShape& sh, int slot, int base, int co
 }
 
 // Prefill on the tensor cores: the context's latents are staged and up-projected to keys and values once per pass.
-static int latent_expanded(BlockModel& m, LatentOp& op, const PassRows& p, const LatentView& cache, cudaStream_t s) {
+static int latent_expanded(BlockModel& m, LatentOp& op, const LayerRun& run, const PassRows& p, const LatentView& cache, cudaStream_t s) {
     const LatentShape& sh = op.sh;
     LatentPreArgs a{sh, m.proj.f(), (const float2*)m.rot[op.rot_table].cs.p, op.c_norm.f(), p.row_slot, p.row_pos, cache, m.q.p, nullptr};
     B2_TRY(launch_latent_pre(op.elem, a, p.rows, s));
@@ -426,7 +450,7 @@ static int latent_expanded(BlockModel& m, LatentOp& op, const PassRows& p, const
         return std::min(x.q_pos0 + 1, W) + x.n_rows > std::min(y.q_pos0 + 1, W) + y.n_rows;
     });
     auto same = [&] {
-        if (m.staged_layer != op.pool_layer || m.staged.size() != spans.size()) return false;
+        if (m.staged_layer != run.pool_layer || m.staged.size() != spans.size()) return false;
         for (size_t i = 0; i < spans.size(); ++i)
             if (std::memcmp(&m.staged[i], &spans[i], sizeof(LatentSpan)) != 0) return false;
         return true;
@@ -434,7 +458,7 @@ static int latent_expanded(BlockModel& m, LatentOp& op, const PassRows& p, const
     if (!same()) {
         B2_CUDA(cudaMemcpyAsync(m.spans(), spans.data(), spans.size() * sizeof(LatentSpan), cudaMemcpyHostToDevice, s));
         B2_TRY(launch_latent_stage(sh, cache, m.spans(), (int)spans.size(), longest, m.c_stage.p, m.r_stage.p, s));
-        m.staged_layer = op.pool_layer;
+        m.staged_layer = run.pool_layer;
         m.staged = spans;
     }
     B2_CUDA(cudaMemcpyAsync(m.tiles(), tiles.data(), tiles.size() * sizeof(LatentTile), cudaMemcpyHostToDevice, s));
@@ -445,31 +469,52 @@ static int latent_expanded(BlockModel& m, LatentOp& op, const PassRows& p, const
     return launch_latent_prefill(sh, m.q.p, p.rows, m.k_up.p, m.r_stage.p, m.v_up.p, ctx, m.tiles(), (int)tiles.size(), m.mixed.p, m.error.i(), s);
 }
 
-static int latent_forward(BlockModel& m, LatentOp& op, const PassRows& p, cudaStream_t s) {
+static int latent_forward(BlockModel& m, LatentOp& op, const LayerRun& run, const PassRows& p, cudaStream_t s) {
     const LatentShape& sh = op.sh;
-    const int W = m.cfg.width, vcols = sh.heads * sh.vp;
-    const LatentView cache = m.pool->latent_view(op.pool_layer);
+    const int W = m.cfg.width;
+    const LatentView cache = m.pool->latent_view(run.pool_layer);
     B2_TRY(gemm_typed(s, m.xt.p, W, op.w_in.p, m.proj.p, sh.pitch(), op.elem, ELEM_F32, p.rows, sh.pitch(), W));
-    B2_TRY(!p.decode && op.tc_prefill ? latent_expanded(m, op, p, cache, s) : latent_absorbed(m, op, p, cache, s));
-    return gemm_typed(s, m.mixed.p, vcols, op.w_out.p, m.y.p, W, op.elem, ELEM_F32, p.rows, W, vcols);
+    return !p.decode && op.tc_prefill ? latent_expanded(m, op, run, p, cache, s) : latent_absorbed(m, op, p, cache, s);
 }
 
 static int run_layers(BlockModel& m, const PassRows& p, cudaStream_t s) {
-    const int W = m.cfg.width;
+    const int W = m.cfg.width, R = p.rows;
     const float eps = (float)m.cfg.norm_eps;
+    const bool pre = m.cfg.pre_norm != 0;
     m.staged_layer = -1;
     for (RotTable& t : m.rot)
-        if (t.half > 0) B2_TRY(launch_rot_table(p.row_pos, (const double*)t.freq.p, t.half, p.rows, (float2*)t.cs.p, s));
-    for (size_t i = 0; i < m.layers.size(); ++i) {
+        if (t.half > 0) B2_TRY(launch_rot_table(p.row_pos, (const double*)t.freq.p, t.half, R, (float2*)t.cs.p, s));
+    if (m.x0.bytes) B2_CUDA(cudaMemcpyAsync(m.x0.p, m.x.p, (size_t)R * W * 4, cudaMemcpyDeviceToDevice, s));
+    // A sublayer's last product: into y, whose norm is added to x, or straight onto x.
+    auto out = [&](const void* in, int cols, const DevBuf& w, const DevBuf& norm) -> int {
+        if (pre) return gemm_typed(s, in, cols, w.p, m.x.p, W, m.elem, ELEM_F32, R, W, cols, 1.0f);
+        B2_TRY(gemm_typed(s, in, cols, w.p, m.y.p, W, m.elem, ELEM_F32, R, W, cols));
+        return launch_post_norm_residual(m.elem, m.y.f(), norm.f(), eps, R, W, m.x.f(), m.xt.p, s);
+    };
+    for (size_t i = 0; i < m.runs.size(); ++i) {
         if (m.stop_after >= 0 && (int)i >= m.stop_after) break;
-        BlockLayer& L = m.layers[i];
-        B2_TRY(L.mlstm ? mlstm_forward(m, *L.mlstm, p, s) : latent_forward(m, *L.latent, p, s));
-        B2_TRY(launch_post_norm_residual(m.elem, m.y.f(), L.norm1.f(), eps, p.rows, W, m.x.f(), m.xt.p, s));
+        const LayerRun& run = m.runs[i];
+        BlockLayer& L = m.layers[run.layer];
+        if (pre) B2_TRY(launch_pre_norm(m.elem, m.x.f(), run.add_embedding ? m.x0.f() : nullptr, L.norm1.f(), eps, R, W, m.xt.p, s));
+        if (L.mlstm) {
+            const MlstmShape& sh = L.mlstm->sh;
+            B2_TRY(sh.gated ? mlstm_forward(m, *L.mlstm, run, p, s) : lightning_forward(m, *L.mlstm, run, p, s));
+            B2_TRY(out(m.mixed.p, sh.heads * sh.vp, L.mlstm->w_out, L.norm1));
+        } else if (L.latent) {
+            B2_TRY(latent_forward(m, *L.latent, run, p, s));
+            B2_TRY(out(m.mixed.p, L.latent->sh.heads * L.latent->sh.vp, L.latent->w_out, L.norm1));
+        } else if (L.delta) {
+            B2_TRY(delta_forward(m, *L.delta, run, p, s));
+            B2_TRY(out(m.mixed.p, L.delta->sh.heads * L.delta->sh.vp, L.delta->w_out, L.norm1));
+        } else {
+            B2_TRY(diff_forward(m, *L.diff, run, p, s));
+            B2_TRY(out(m.mixed.p, L.diff->sh.heads * L.diff->sh.vp, L.diff->w_out, L.norm1));
+        }
         if (L.ff == 0) continue;
-        B2_TRY(gemm_typed(s, m.xt.p, W, L.w_gu.p, m.gu.p, 2 * L.ff, m.elem, m.elem, p.rows, 2 * L.ff, W));
-        B2_TRY(launch_gelu_mul(m.elem, m.gu.p, p.rows, L.ff, m.act.p, s));
-        B2_TRY(gemm_typed(s, m.act.p, L.ff, L.w_down.p, m.y.p, W, m.elem, ELEM_F32, p.rows, W, L.ff));
-        B2_TRY(launch_post_norm_residual(m.elem, m.y.f(), L.norm2.f(), eps, p.rows, W, m.x.f(), m.xt.p, s));
+        if (pre) B2_TRY(launch_pre_norm(m.elem, m.x.f(), nullptr, L.norm2.f(), eps, R, W, m.xt.p, s));
+        B2_TRY(gemm_typed(s, m.xt.p, W, L.w_gu.p, m.gu.p, 2 * L.ff, m.elem, m.elem, R, 2 * L.ff, W));
+        B2_TRY(launch_act_mul(m.elem, L.act, m.gu.p, R, L.ff, m.act.p, s));
+        B2_TRY(out(m.act.p, L.ff, L.w_down, L.norm2));
     }
     if (m.pool)
         B2_TRY(launch_lens_advance(m.pool->d_lens, m.pool->cfg.num_layers, m.cfg.max_seqs, p.d_slots, p.decode ? nullptr : p.d_seqs, p.n_seqs, s));
@@ -552,7 +597,9 @@ int block_prefill_rows(BlockModel& m, int n_seqs, const int* h_slots, const int*
 int block_logits(BlockModel& m, int n, const int* d_row_index, float* d_logits, cudaStream_t s) {
     const int W = m.cfg.width;
     B2_TRY(launch_rms_norm_rows(m.elem, m.x.f(), d_row_index, m.final_norm.f(), (float)m.cfg.norm_eps, n, W, m.xt.p, s));
-    return gemm_typed(s, m.xt.p, W, m.embed.p, d_logits, m.cfg.vocab_size, m.elem, ELEM_F32, n, m.cfg.vocab_size, W, 0.f, (float)m.cfg.logit_scale);
+    B2_TRY(gemm_typed(s, m.xt.p, W, m.cfg.own_head ? m.head.p : m.embed.p, d_logits, m.cfg.vocab_size, m.elem, ELEM_F32, n, m.cfg.vocab_size, W, 0.f,
+                      (float)m.cfg.logit_scale));
+    return m.cfg.logit_softcap > 0 ? launch_softcap(d_logits, (size_t)n * m.cfg.vocab_size, (float)m.cfg.logit_softcap, s) : 0;
 }
 
 }  // namespace b200

@@ -1,6 +1,8 @@
-// Matrix memory with exponential gating (mLSTM): the token-serial recurrence and the head norm.
+// Matrix memory: the token-serial recurrence and the norms behind it, with exponential gating (mLSTM) or with one constant
+// decay per head (lightning attention: S_t = decay S_{t-1} + k_t v_t^T, o_t = S_t^T q_t, with silu on q, k and v; the
+// concatenated heads are normed together).
 //
-// Per head, with log input gate i = cap tanh(. / cap) and log forget gate f = logsigmoid(cap tanh(. / cap)):
+// mLSTM: per head, with log input gate i = cap tanh(. / cap) and log forget gate f = logsigmoid(cap tanh(. / cap)):
 //     m_t = max(f_t + m_{t-1}, i_t),   S_t = e^{f_t + m_{t-1} - m_t} S_{t-1} + e^{i_t - m_t} k_t v_t^T,   n_t likewise with k_t
 //     o_t = S_t^T q_t / (max(|n_t . q_t|, e^{-m_t}) + 1e-6)
 // and all of S, n, m start at zero.  The state of a head lies in tiles of up to 128 value columns, each with a copy of n
@@ -18,7 +20,7 @@ namespace b200 {
 // key rows w, w + 8, ...; with dim <= 8 NR a thread's part of the state stays in registers over the whole run of tokens
 // (decode: one token), else it is streamed through for every token.  Decode loads its state ahead of the wait on the
 // preceding kernel: the state was last written one step earlier.
-template <int NR, typename T, bool kFuseNorm>
+template <int NR, typename T, bool kGated, bool kFuseNorm>
 __global__ void __launch_bounds__(256)
 mlstm_step_kernel(const MlstmStepArgs a, unsigned long long* stamp) {
     extern __shared__ float sm[];
@@ -53,26 +55,37 @@ mlstm_step_kernel(const MlstmStepArgs a, unsigned long long* stamp) {
             if (d < D) st[i] = __ldcs(reinterpret_cast<const float4*>(S + (size_t)d * sh.vt + c0));
         }
     }
-    float m = *gm;
-    for (int d = tid; d < D; d += 256) s_n[d] = gn[d];
+    float m = 0.f;
+    if constexpr (kGated) {
+        m = *gm;
+        for (int d = tid; d < D; d += 256) s_n[d] = gn[d];
+    }
     pdl_enter();
     stamp_begin(stamp);
-    const float q_scale = 1.0f / sqrtf((float)D);
+    const float q_scale = kGated ? 1.0f / sqrtf((float)D) : 1.0f;
+    auto taken = [](float x) { return kGated ? x : times_sigmoid<float>(x, x); };
     const int V = sh.vdim;
     for (int t = 0; t < count; ++t) {
         const size_t row = row0 + t;
         const float* pr = a.proj + row * sh.pitch();
         for (int d = tid; d < D; d += 256) {
-            s_q[d] = pr[sh.off_q() + h * sh.dp + d] * q_scale;
-            s_k[d] = pr[sh.off_k() + h * sh.dp + d];
+            s_q[d] = taken(pr[sh.off_q() + h * sh.dp + d]) * q_scale;
+            s_k[d] = taken(pr[sh.off_k() + h * sh.dp + d]);
         }
         float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
         if (act && vcol < sh.vp) v = *reinterpret_cast<const float4*>(pr + sh.off_v() + h * sh.vp + vcol);
-        const float ig = mlstm_log_input(pr[sh.off_i() + h] + a.bias[h], sh.gate_cap);
-        const float fg = mlstm_log_forget(pr[sh.off_f() + h] + a.bias[sh.heads + h], sh.gate_cap);
-        const float m_new = fmaxf(fg + m, ig);
-        const float keep = expf(fg + m - m_new), add = expf(ig - m_new);
-        m = m_new;
+        v = make_float4(taken(v.x), taken(v.y), taken(v.z), taken(v.w));
+        float keep, add = 1.f;
+        if constexpr (kGated) {
+            const float ig = mlstm_log_input(pr[sh.off_i() + h] + a.bias[h], sh.gate_cap);
+            const float fg = mlstm_log_forget(pr[sh.off_f() + h] + a.bias[sh.heads + h], sh.gate_cap);
+            const float m_new = fmaxf(fg + m, ig);
+            keep = expf(fg + m - m_new);
+            add = expf(ig - m_new);
+            m = m_new;
+        } else {
+            keep = a.bias[h];
+        }
         __syncthreads();
         float4 num = make_float4(0.f, 0.f, 0.f, 0.f);
         auto row_step = [&](float4 x, int d) -> float4 {
@@ -97,7 +110,7 @@ mlstm_step_kernel(const MlstmStepArgs a, unsigned long long* stamp) {
             }
         }
         float nq = 0.f;
-        for (int d = tid; d < D; d += 256) {
+        if constexpr (kGated) for (int d = tid; d < D; d += 256) {
             const float nn = keep * s_n[d] + add * s_k[d];
             s_n[d] = nn;
             nq += nn * s_q[d];
@@ -115,7 +128,7 @@ mlstm_step_kernel(const MlstmStepArgs a, unsigned long long* stamp) {
             if (mine) {
 #pragma unroll
                 for (int w = 0; w < 8; ++w) o += s_red[w * kMlstmTile + tid];
-                o /= fmaxf(fabsf(nq), expf(-m)) + 1e-6f;
+                if constexpr (kGated) o /= fmaxf(fabsf(nq), expf(-m)) + 1e-6f;
             }
         }
         if constexpr (kFuseNorm) {
@@ -145,8 +158,10 @@ mlstm_step_kernel(const MlstmStepArgs a, unsigned long long* stamp) {
             if (d < D) __stcs(reinterpret_cast<float4*>(S + (size_t)d * sh.vt + c0), st[i]);
         }
     }
-    for (int d = tid; d < D; d += 256) gn[d] = s_n[d];
-    if (tid == 0) *gm = m;
+    if constexpr (kGated) {
+        for (int d = tid; d < D; d += 256) gn[d] = s_n[d];
+        if (tid == 0) *gm = m;
+    }
     if (stamp) { __syncthreads(); stamp_end(stamp); }
 }
 
@@ -158,14 +173,16 @@ int launch_mlstm_step(ElemType t, const MlstmStepArgs& a, int n, cudaStream_t s)
     dispatch_elem(t, [&](auto tag) {
         using T = decltype(tag);
         auto go = [&](auto kernel) { launch_pdl(kernel, grid, dim3(256), smem, s, a, stamp); };
-        auto pick = [&](auto fuse) {
-            constexpr bool kFuse = decltype(fuse)::value;
-            if (sh.dim <= 32) go(mlstm_step_kernel<4, T, kFuse>);
-            else if (sh.dim <= 64) go(mlstm_step_kernel<8, T, kFuse>);
-            else if (sh.dim <= 128) go(mlstm_step_kernel<16, T, kFuse>);
-            else go(mlstm_step_kernel<32, T, kFuse>);
+        auto pick = [&](auto gated, auto fuse) {
+            constexpr bool kGated = decltype(gated)::value, kFuse = decltype(fuse)::value;
+            if (sh.dim <= 32) go(mlstm_step_kernel<4, T, kGated, kFuse>);
+            else if (sh.dim <= 64) go(mlstm_step_kernel<8, T, kGated, kFuse>);
+            else if (sh.dim <= 128) go(mlstm_step_kernel<16, T, kGated, kFuse>);
+            else go(mlstm_step_kernel<32, T, kGated, kFuse>);
         };
-        if (sh.n_vt == 1) pick(std::true_type{}); else pick(std::false_type{});
+        if (!sh.gated) pick(std::false_type{}, std::false_type{});
+        else if (sh.n_vt == 1) pick(std::true_type{}, std::true_type{});
+        else pick(std::true_type{}, std::false_type{});
     });
     B2_LAUNCH_CHECK();
     return 0;
@@ -237,6 +254,92 @@ int launch_mlstm_head_norm(ElemType t, const MlstmShape& sh, const float* core, 
         else
             launch_pdl(mlstm_head_norm_kernel<T, T>, grid, dim3(256), 0, s, core, (const T*)g, g_pitch, sh.off_g(), norm_w, sh.eps, sh.heads, sh.vdim,
                        sh.vp, (T*)gated);
+    });
+    B2_LAUNCH_CHECK();
+    return 0;
+}
+
+// All heads of a row over their common root mean square, times the weight, times sigmoid(g).  One block per row; rows of up
+// to 4096 values stay in registers between the two passes.  Columns from vdim on in every head are zero.
+template <typename T, typename G>
+__global__ void __launch_bounds__(256)
+row_norm_gate_kernel(const float* __restrict__ core, const G* __restrict__ g, int g_pitch, int off_g, const float* __restrict__ norm_w, float eps,
+                     int cols, int n, T* __restrict__ out) {
+    __shared__ float s_part[8];
+    pdl_enter();
+    const float* c = core + (size_t)blockIdx.x * cols;
+    const G* gr = g + (size_t)blockIdx.x * g_pitch + off_g;
+    T* o = out + (size_t)blockIdx.x * cols;
+    auto gated = [](float4 x, float inv, float4 w, float4 z) {
+        return make_float4(times_sigmoid<T>(x.x * inv * w.x, z.x), times_sigmoid<T>(x.y * inv * w.y, z.y), times_sigmoid<T>(x.z * inv * w.z, z.z),
+                           times_sigmoid<T>(x.w * inv * w.w, z.w));
+    };
+    auto block_sum = [&](float v) {
+#pragma unroll
+        for (int k = 16; k > 0; k >>= 1) v += __shfl_xor_sync(0xffffffffu, v, k);
+        if ((threadIdx.x & 31) == 0) s_part[threadIdx.x >> 5] = v;
+        __syncthreads();
+        return ((s_part[0] + s_part[1]) + (s_part[2] + s_part[3])) + ((s_part[4] + s_part[5]) + (s_part[6] + s_part[7]));
+    };
+    float ss = 0.f;
+    if (cols <= 4096) {
+        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+        float4 x[4], z[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int v = 4 * (threadIdx.x + 256 * i);
+            x[i] = v < cols ? __ldcs(reinterpret_cast<const float4*>(c + v)) : zero;
+            z[i] = v < cols ? load4(gr + v) : zero;
+            ss += x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
+        }
+        const float inv = 1.0f / sqrtf(block_sum(ss) / (float)n + eps);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int v = 4 * (threadIdx.x + 256 * i);
+            if (v < cols) store4(o + v, gated(x[i], inv, load4(norm_w + v), z[i]));
+        }
+        return;
+    }
+    for (int v = 4 * threadIdx.x; v < cols; v += 1024) {
+        const float4 x = load4(c + v);
+        ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss) / (float)n + eps);
+    for (int v = 4 * threadIdx.x; v < cols; v += 1024) store4(o + v, gated(load4(c + v), inv, load4(norm_w + v), load4(gr + v)));
+}
+
+int launch_row_norm_gate(ElemType t, const MlstmShape& sh, const float* core, const void* g, bool g_f32, int g_pitch, const float* norm_w, int rows,
+                         void* gated, cudaStream_t s) {
+    const int cols = sh.heads * sh.vp, n = sh.heads * sh.vdim;
+    dispatch_elem(t, [&](auto tag) {
+        using T = decltype(tag);
+        if (g_f32)
+            launch_pdl(row_norm_gate_kernel<T, float>, dim3(rows), dim3(256), 0, s, core, (const float*)g, g_pitch, sh.off_g(), norm_w, sh.eps, cols, n,
+                       (T*)gated);
+        else
+            launch_pdl(row_norm_gate_kernel<T, T>, dim3(rows), dim3(256), 0, s, core, (const T*)g, g_pitch, sh.off_g(), norm_w, sh.eps, cols, n, (T*)gated);
+    });
+    B2_LAUNCH_CHECK();
+    return 0;
+}
+
+// One block of 256 threads per row.
+template <typename T>
+__global__ void __launch_bounds__(256)
+silu_cols_kernel(T* __restrict__ p, int cols, int pitch) {
+    pdl_enter();
+    T* r = p + (size_t)blockIdx.x * pitch;
+#pragma unroll 4
+    for (int c = 4 * threadIdx.x; c < cols; c += 1024) {
+        const float4 v = load4(r + c);
+        store4(r + c, make_float4(times_sigmoid<T>(v.x, v.x), times_sigmoid<T>(v.y, v.y), times_sigmoid<T>(v.z, v.z), times_sigmoid<T>(v.w, v.w)));
+    }
+}
+
+int launch_silu_cols(ElemType t, void* p, int rows, int cols, int pitch, cudaStream_t s) {
+    dispatch_elem(t, [&](auto tag) {
+        using T = decltype(tag);
+        launch_pdl(silu_cols_kernel<T>, dim3(rows), dim3(256), 0, s, (T*)p, cols, pitch);
     });
     B2_LAUNCH_CHECK();
     return 0;

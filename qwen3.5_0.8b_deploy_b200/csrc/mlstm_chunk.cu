@@ -12,6 +12,9 @@
 //     issuer    S1                O1            O2, S^T += V^T Kw
 //     threads        Kw, n, decay     P, n . q                     outputs, S^T -> tile
 // The keys are scaled in their TMA tile (hi; lo beside it); the P tiles overwrite the state tile, which is dead by then.
+//
+// A constant decay (kGated false; lightning attention) is the same with f = log decay, i = 0 and M_t = -F_t, so that m stays
+// zero and the state is not rescaled: e^{a_s - M_t} = decay^{t - s}.  There is no normaliser and no q factor then.
 #include "block_model.cuh"
 #include "elem.cuh"
 #include "mlstm.cuh"
@@ -44,7 +47,7 @@ __device__ __forceinline__ uint32_t sw128(int r, int p) { return (uint32_t)(r * 
 }  // namespace
 
 // grid (heads * value tiles, sequences); ND = dp / 64 key blocks, NV = value blocks of a tile
-template <int ND, int NV>
+template <int ND, int NV, bool kGated>
 __global__ void __launch_bounds__(kMThreads, 1)
 mlstm_chunk_kernel(const __grid_constant__ CUtensorMap map, const MlstmShape sh, const float* __restrict__ gates, int gate_pitch,
                    const float* __restrict__ bias, const LaSeqMeta* __restrict__ seqs, int max_seqs, float* __restrict__ state,
@@ -149,8 +152,27 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap map, const MlstmShape sh,
     } else if (warp == 9) {
         // ------------------------------ gates: four tokens per lane ------------------------------
         const float bi = bias[h], bf = bias[sh.heads + h], q_scale = 1.0f / sqrtf((float)sh.dim);
-        float m0 = *gm;
-        for (int c = 0; c < n_chunks; ++c) {
+        float m0 = kGated ? *gm : 0.f;
+        if constexpr (!kGated) {
+            const float ld = bf;
+            for (int c = 0; c < n_chunks; ++c) {
+                const int b = c & 1, left = min(kMC, sq.count - c * kMC);
+                if (c >= 2 && !mbar_wait_warp(bar(M_GE + b), ((c >> 1) - 1) & 1, abort_flag)) break;
+                float* ga = g_arr(b);
+                const float F_all = ld * (float)left;
+                for (int t = lane; t < kMC; t += 32) {
+                    const float F = ld * (float)min(t + 1, left);
+                    ga[t] = t < left ? -F * kL2e : -INFINITY;
+                    ga[kMC + t] = -F * kL2e;
+                    ga[2 * kMC + t] = expf(F);
+                    ga[4 * kMC + t] = t < left ? expf(ld * (float)(left - 1 - t)) : 0.f;
+                }
+                if (lane == 0) ga[5 * kMC] = expf(F_all);
+                __syncwarp();
+                if (lane == 0) mbar_arrive(bar(M_GF + b));
+            }
+        }
+        if constexpr (kGated) for (int c = 0; c < n_chunks; ++c) {
             const int b = c & 1;
             float ig[4], F[4];
             float run = 0.f;
@@ -209,13 +231,13 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap map, const MlstmShape sh,
             __syncwarp();
             if (lane == 0) mbar_arrive(bar(M_GF + b));
         }
-        if (lane == 0 && !*abort_flag) *gm = m0;
+        if (kGated && lane == 0 && !*abort_flag) *gm = m0;
     } else {
         // ------------------------------ compute warps ------------------------------
         const int r = tid & 127;     // TMEM lane: token of S1 / O1 / O2, value column of S^T
         const int hf = tid >> 7;     // which half of the columns
         const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
-        const float q_scale = 1.0f / sqrtf((float)sh.dim);
+        const float q_scale = kGated ? 1.0f / sqrtf((float)sh.dim) : 1.0f;
         float* s_rs = reinterpret_cast<float*>(sm + kMOffR);
         auto s_n = [&](int b) { return reinterpret_cast<float*>(sm + kMOffN) + b * kMC; };
         bool ok = true;
@@ -246,7 +268,7 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap map, const MlstmShape sh,
             tmem_st32(tm_st + lane_base + ch * 32, sv);
             state_cols(ch, sv);
         }
-        if (tid < kMC) s_n(0)[tid] = tid < sh.dim ? gn[tid] : 0.f;
+        if (kGated && tid < kMC) s_n(0)[tid] = tid < sh.dim ? gn[tid] : 0.f;
         tmem_wait_st();
         fence_proxy_async_smem();
         tc_fence_before();
@@ -260,7 +282,7 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap map, const MlstmShape sh,
             const float keep = ga[5 * kMC];
             // n_0 . q of this thread's row, its half of the key columns
             float nq = 0.f;
-            {
+            if constexpr (kGated) {
                 const float* n0 = s_n(par);
 #pragma unroll
                 for (int p = 0; p < 4 * ND; ++p) {
@@ -298,6 +320,7 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap map, const MlstmShape sh,
                     *p = make_uint4(hi[0], hi[1], hi[2], hi[3]);
                     *reinterpret_cast<uint4*>(reinterpret_cast<unsigned char*>(p) + (kMOffKlo - kMOffK)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
                 }
+                if constexpr (!kGated) continue;
                 // eight sums over 32 lanes: halve the values while halving the lanes, lane groups of four end with one column each
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
@@ -375,10 +398,13 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap map, const MlstmShape sh,
             fence_proxy_async_smem();
             tc_fence_before();
             mbar_arrive(bar(M_P));
-            s_rs[hf * kMC + r] = nq;
+            if constexpr (kGated) s_rs[hf * kMC + r] = nq;
             sync_compute();
-            nq += s_rs[(hf ^ 1) * kMC + r];
-            const float inv = 1.0f / (fmaxf(fabsf(nq), ga[3 * kMC + r]) + 1e-6f);
+            float inv = 1.0f;
+            if constexpr (kGated) {
+                nq += s_rs[(hf ^ 1) * kMC + r];
+                inv = 1.0f / (fmaxf(fabsf(nq), ga[3 * kMC + r]) + 1e-6f);
+            }
             const float em = ga[2 * kMC + r];
             mbar_arrive(bar(M_GE + par));
             // ---- outputs and the next state tile ----
@@ -431,7 +457,7 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap map, const MlstmShape sh,
                     if (d < sh.dim && r < sh.vt) Sg[(size_t)d * sh.vt + r] = __uint_as_float(sv[e]);
                 }
             }
-            if (tid < sh.dim) gn[tid] = s_n(n_chunks & 1)[tid];
+            if (kGated && tid < sh.dim) gn[tid] = s_n(n_chunks & 1)[tid];
         }
     }
     tc_fence_before();
@@ -445,7 +471,7 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap map, const MlstmShape sh,
 
 bool mlstm_chunk_fits(const MlstmShape& sh) { return sh.dp <= 128; }
 
-// qkvg: bf16 [rows][cols]; gates: fp32 [rows][gate_pitch], input then forget pre-activations.
+// qkvg: bf16 [rows][cols]; gates: fp32 [rows][gate_pitch], input then forget pre-activations (not gated: unused, bias holds decays and log decays).
 int launch_mlstm_chunk(const MlstmShape& sh, const void* qkvg, int rows, const float* gates, int gate_pitch, const float* bias,
                        const LaSeqMeta* d_seqs, int n_seqs, int max_seqs, float* state, float* core, int* d_error, cudaStream_t s) {
     CUtensorMap map;
@@ -455,17 +481,20 @@ int launch_mlstm_chunk(const MlstmShape& sh, const void* qkvg, int rows, const f
     B2_TRY(make_tensor_map(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, qkvg, dims, str, box));
     static PerDeviceOnce once;
     B2_PER_DEVICE_ONCE(once,
-        B2_CUDA(cudaFuncSetAttribute(mlstm_chunk_kernel<1, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMSmem));
-        B2_CUDA(cudaFuncSetAttribute(mlstm_chunk_kernel<1, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMSmem));
-        B2_CUDA(cudaFuncSetAttribute(mlstm_chunk_kernel<2, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMSmem));
-        B2_CUDA(cudaFuncSetAttribute(mlstm_chunk_kernel<2, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMSmem)));
+        for (auto k : {mlstm_chunk_kernel<1, 1, true>, mlstm_chunk_kernel<1, 2, true>, mlstm_chunk_kernel<2, 1, true>, mlstm_chunk_kernel<2, 2, true>,
+                       mlstm_chunk_kernel<1, 1, false>, mlstm_chunk_kernel<1, 2, false>, mlstm_chunk_kernel<2, 1, false>, mlstm_chunk_kernel<2, 2, false>})
+            B2_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, kMSmem)));
     const dim3 grid(sh.heads * sh.n_vt, n_seqs);
     auto go = [&](auto kernel) { kernel<<<grid, kMThreads, kMSmem, s>>>(map, sh, gates, gate_pitch, bias, d_seqs, max_seqs, state, core, d_error); };
     const bool d2 = sh.dp > 64, v2 = sh.vp > 64;
-    if (d2 && v2) go(mlstm_chunk_kernel<2, 2>);
-    else if (d2) go(mlstm_chunk_kernel<2, 1>);
-    else if (v2) go(mlstm_chunk_kernel<1, 2>);
-    else go(mlstm_chunk_kernel<1, 1>);
+    auto pick = [&](auto gated) {
+        constexpr bool kGated = decltype(gated)::value;
+        if (d2 && v2) go(mlstm_chunk_kernel<2, 2, kGated>);
+        else if (d2) go(mlstm_chunk_kernel<2, 1, kGated>);
+        else if (v2) go(mlstm_chunk_kernel<1, 2, kGated>);
+        else go(mlstm_chunk_kernel<1, 1, kGated>);
+    };
+    if (sh.gated) pick(std::true_type{}); else pick(std::false_type{});
     B2_LAUNCH_CHECK();
     return 0;
 }

@@ -1,11 +1,17 @@
-// Split decode attention over cached latents, up to 16 heads at a time (bf16).
+// Split decode attention over pages of cache rows, 16 query rows at a time (bf16).
 //
-// With absorbed queries all heads of a row share one key and value stream: the cache rows themselves.  A row of a decode
-// step needs the pages its window touches; the pages of all (row, head group) pairs form one list that is cut into equal
-// ranges, one per CTA (one CTA per SM), so every SM streams the same number of bytes whatever the lengths are.  A producer
-// lane brings whole pages (64 rows) into a ring of shared-memory stages with bulk TMA copies; eight consumer warps run
-//     S [16 heads x 64 keys] = Q' [16 x (rank + rot)] C^T     a quarter of the contraction for half of the keys per warp
-//     O [16 x rank] += P C                                    rank / 8 columns per warp
+// Latents: with absorbed queries all heads of a row share one key and value stream, the cache rows themselves, whose first
+// `rank` columns are the values; 16 heads form a group.  Differential attention: a group is one key / value head with up to 8
+// query heads; its cache rows are [k of map 1 | k of map 2 | v], and its query rows 0 .. 7 hold the heads' map-1 queries over
+// the columns of map 1 (zeros elsewhere), rows 8 .. 15 the map-2 queries over those of map 2, so that one product gives the
+// scores of both maps and one product both maps' outputs, which meet in the same thread.
+//
+// A row of a decode step needs the pages its kept positions and its window touch; the pages of all (row, group) pairs form one
+// list that is cut into equal ranges, one per CTA (one CTA per SM), so every SM streams the same number of bytes whatever the
+// lengths are.  A producer lane brings whole pages (64 rows) into a ring of shared-memory stages with bulk TMA copies; eight
+// consumer warps run
+//     S [16 x 64 keys] = Q [16 x key columns] K^T     a quarter of the contraction for half of the keys per warp
+//     O [16 x value columns] += P V                   an eighth of the columns per warp
 // on mma.sync m16n8k16 (bf16, fp32 accumulation): at 16 query rows per key byte the kernel is bound by HBM, not by the
 // tensor pipe.  What counts on chip is shared-memory traffic: a warp keeps its part of the queries in registers for a whole
 // pair and every key and value byte is read once; the four partial scores meet in the softmax step, which 16 threads per
@@ -45,14 +51,25 @@ __device__ __forceinline__ float ex2l(float x) {
 }
 __device__ __forceinline__ void sync_consumers() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
+// What the kernel is told about the rows it reads.
+struct LdShape {
+    int pitch, qpitch;                    // elements per cache row of a group / per query row
+    int groups;                           // groups per row
+    int ksteps, vcol0, vcols;             // 16-column steps of the contraction; value columns
+    int window, keep;
+    float sc;                             // score factor times log2 e
+    int heads, per;                       // heads of a row, of a group
+    int vdim;                             // differential attention: real value columns, and the constants of the combination
+    float lambda, out_scale, eps;
+};
 struct LdLayout { uint32_t q, q_bytes, s, p, pre, bar, stage0, stage_bytes, total; int stages; };
-__host__ __device__ inline LdLayout ld_layout(int pitch, int rows) {
+__host__ __device__ inline LdLayout ld_layout(int pitch, int qpitch, int rows) {
     LdLayout L;
     L.q = 0;
-    L.q_bytes = (kHG * pitch * 2 + 127) / 128 * 128;         // two query buffers
+    L.q_bytes = (kHG * qpitch * 2 + 127) / 128 * 128;        // two query buffers
     L.s = L.q + 2 * L.q_bytes;
     L.p = L.s + 4 * kHG * kSPitch * 4;                       // partial scores of the four quarters
-    L.pre = L.p + kHG * kPPitch * 2 + 3 * kHG * 4;           // weights (bf16), then factor, maximum and sum of every head
+    L.pre = L.p + kHG * kPPitch * 2 + 3 * kHG * 4 + 64 * 4;  // weights (bf16), then factor, maximum and sum of every query row, sums of squares
     L.bar = L.pre + (2 * rows + 2 + 3) / 4 * 16;
     L.bar = (L.bar + 15) / 16 * 16;
     L.stage0 = (L.bar + 128 + 127) / 128 * 128;
@@ -65,17 +82,28 @@ __host__ __device__ inline LdLayout ld_layout(int pitch, int rows) {
 }
 template <int NT> constexpr int kPartFloats = NT * 1024 + 32;      // O in register order, then (m, l) of the 16 heads
 struct Seg { int row, hg, p0, p1, np; };   // pages [p0, p1) of the np of one pair
+// The pages of a row: those with kept positions, then those its window touches behind them.
+struct Pages {
+    int first, kept, w0, n;               // first position of the window, pages of kept positions, first page behind them, pages in all
+    __device__ Pages(const LdShape& sh, int pos) {
+        first = sh.window > 0 ? max(0, pos - sh.window + 1) : 0;
+        kept = (min(sh.keep, pos + 1) + kPageTokens - 1) / kPageTokens;
+        w0 = max(kept, first / kPageTokens);
+        n = kept + max(0, pos / kPageTokens - w0 + 1);
+    }
+    __device__ int at(int j) const { return j < kept ? j : w0 + j - kept; }
+};
 }  // namespace
 
 // NT = 8-column tiles of the latent per consumer warp, KQ = 16-column steps of the contraction per warp
-template <int NT, int KQ>
+template <int NT, int KQ, bool kDiff>
 __global__ void __launch_bounds__(kLdThreads, 1)
-latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa, const LatentView cache, const int* __restrict__ row_slot,
+page_decode_kernel(const LdShape sh, const __nv_bfloat16* __restrict__ qa, const LatentView cache, const int* __restrict__ row_slot,
                      const int* __restrict__ row_pos, int rows, float* __restrict__ part, int* __restrict__ counters,
                      __nv_bfloat16* __restrict__ out, unsigned long long* stamp) {
     extern __shared__ __align__(128) unsigned char sm[];
-    const int pitch = sh.row_pitch(), hgs = (sh.heads + kHG - 1) / kHG;
-    const LdLayout L = ld_layout(pitch, rows);
+    const int pitch = sh.pitch, qpitch = sh.qpitch, hgs = sh.groups;
+    const LdLayout L = ld_layout(pitch, qpitch, rows);
     const uint32_t base = smem_u32(sm);
     int* s_pre = reinterpret_cast<int*>(sm + L.pre);              // pages before row r; [rows] = all; [rows + 1] = most of one row
     int* s_pos = s_pre + rows + 2;
@@ -93,12 +121,11 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
         *abort_flag = 0;
         mbar_fence_init();
     }
-    if (sh.heads % kHG) {             // query rows of absent heads are never copied: finite from the start
+    if (!kDiff && sh.heads % kHG) {   // query rows of absent heads are never copied: finite from the start
         for (uint32_t e = tid; e < 2 * L.q_bytes / 16; e += kLdThreads) reinterpret_cast<uint4*>(sm + L.q)[e] = make_uint4(0u, 0u, 0u, 0u);
         fence_proxy_async_smem();
     }
     pdl_wait();
-    auto first_key = [&](int pos) { return sh.window > 0 ? max(0, pos - sh.window + 1) : 0; };
     if (warp == 0) {                                              // page counts and their running sum
         int sum = 0, most = 0;
         for (int r0 = 0; r0 < rows; r0 += 32) {
@@ -107,7 +134,7 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
             if (r < rows) {
                 const int slot = row_slot[r], pos = row_pos[r];
                 s_pos[r] = pos;
-                if (slot >= 0 && slot < cache.max_seqs && pos < cache.capacity[slot]) n = pos / kPageTokens - first_key(pos) / kPageTokens + 1;
+                if (slot >= 0 && slot < cache.max_seqs && pos < cache.capacity[slot]) n = Pages(sh, pos).n;
             }
             most = max(most, n);
             int inc = n;
@@ -150,42 +177,45 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
             int it = 0, sg = 0;
             for (int u = u0; u < u1; ++sg) {
                 const Seg g = segment(u);
-                const int slot = row_slot[g.row], first = first_key(s_pos[g.row]) / kPageTokens;
-                const uint32_t qb = (uint32_t)min(kHG, sh.heads - g.hg * kHG) * pitch * 2;
+                const int slot = row_slot[g.row];
+                const Pages pg(sh, s_pos[g.row]);
+                const uint32_t qb = (uint32_t)(kDiff ? kHG : min(kHG, sh.heads - g.hg * kHG)) * qpitch * 2;
                 if (sg >= 2 && !mbar_wait(q_empty(sg & 1), ((sg >> 1) - 1) & 1, abort_flag)) break;
                 mbar_arrive_expect_tx(q_full(sg & 1), qb);
-                bulk_g2s(base + L.q + (sg & 1) * L.q_bytes, qa + ((size_t)g.row * sh.heads + g.hg * kHG) * pitch, qb, q_full(sg & 1));
-                const int* table = cache.block_table + (size_t)slot * cache.max_pages_per_seq + first;
+                bulk_g2s(base + L.q + (sg & 1) * L.q_bytes, qa + (kDiff ? ((size_t)g.row * hgs + g.hg) * kHG : (size_t)g.row * sh.heads + g.hg * kHG) * qpitch, qb, q_full(sg & 1));
+                const int* table = cache.block_table + (size_t)slot * cache.max_pages_per_seq;
                 for (int p = g.p0; p < g.p1; ++p, ++it) {
                     const int s = it % L.stages;
                     if (it >= L.stages && !mbar_wait(empty(s), (it / L.stages - 1) & 1, abort_flag)) { u = u1; break; }
                     mbar_arrive_expect_tx(full(s), L.stage_bytes);
                     bulk_g2s(base + L.stage0 + s * L.stage_bytes,
-                             static_cast<const __nv_bfloat16*>(cache.rows) + (size_t)table[p] * kPageTokens * pitch, L.stage_bytes, full(s));
+                             static_cast<const __nv_bfloat16*>(cache.rows) + (kDiff ? (size_t)table[pg.at(p)] * hgs + g.hg : (size_t)table[pg.at(p)]) * kPageTokens * pitch,
+                             L.stage_bytes, full(s));
                 }
                 u += g.p1 - g.p0;
             }
         }
     } else {
         const int g4 = lane >> 2, t4 = lane & 3;                  // fragment row and column pair
-        const int ksteps = (pitch - 8) / 16, k0 = (warp & 3) * KQ, keys = (warp >> 2) * 32;
+        const int ksteps = sh.ksteps, k0 = (warp & 3) * KQ, keys = (warp >> 2) * 32;
         const int srow = tid >> 4, skey = 4 * (tid & 15);         // softmax: head and four keys of this thread
-        const float sc = sh.scale * 1.4426950408889634f;
+        const float sc = sh.sc;
         float* SP = reinterpret_cast<float*>(sm + L.s);
         __nv_bfloat16* PT = reinterpret_cast<__nv_bfloat16*>(sm + L.p);
         float* s_al = reinterpret_cast<float*>(sm + L.p + kHG * kPPitch * 2);
-        float *s_m = s_al + kHG, *s_l = s_m + kHG;
+        float *s_m = s_al + kHG, *s_l = s_m + kHG, *s_ss = s_l + kHG;      // s_ss: [8 warps][8 heads]
         const uint32_t p_addr = base + L.p + ((lane & 15) * kPPitch + (lane >> 4) * 8) * 2;
         int it = 0, sg = 0;
         for (int u = u0; u < u1; ++sg) {
             const Seg g = segment(u);
             u += g.p1 - g.p0;
-            const int pos = s_pos[g.row], first = first_key(pos), key0 = first / kPageTokens * kPageTokens;
-            const int n_heads = min(kHG, sh.heads - g.hg * kHG);
+            const int pos = s_pos[g.row];
+            const Pages pg(sh, pos);
+            const int n_heads = kDiff ? sh.per : min(kHG, sh.heads - g.hg * kHG);
             mbar_wait_warp(q_full(sg & 1), (sg >> 1) & 1, abort_flag);
             uint32_t qf[KQ][4];
             {
-                const uint32_t a_addr = base + L.q + (sg & 1) * L.q_bytes + ((lane & 15) * pitch + (lane >> 4) * 8) * 2;
+                const uint32_t a_addr = base + L.q + (sg & 1) * L.q_bytes + ((lane & 15) * qpitch + (lane >> 4) * 8) * 2;
 #pragma unroll
                 for (int k = 0; k < KQ; ++k)
                     if (k0 + k < ksteps) ldm_x4(qf[k], a_addr + (k0 + k) * 32);
@@ -230,11 +260,11 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
                     const float4 a = *reinterpret_cast<const float4*>(S), b = *reinterpret_cast<const float4*>(S + kHG * kSPitch);
                     const float4 c = *reinterpret_cast<const float4*>(S + 2 * kHG * kSPitch), d = *reinterpret_cast<const float4*>(S + 3 * kHG * kSPitch);
                     float v[4] = {(a.x + b.x) + (c.x + d.x), (a.y + b.y) + (c.y + d.y), (a.z + b.z) + (c.z + d.z), (a.w + b.w) + (c.w + d.w)};
-                    const int kpos = key0 + p * kPageTokens + skey;
+                    const int kpos = pg.at(p) * kPageTokens + skey;
                     float mx = -INFINITY;
 #pragma unroll
                     for (int e = 0; e < 4; ++e) {
-                        v[e] = (kpos + e >= first && kpos + e <= pos) ? v[e] * sc : -INFINITY;
+                        v[e] = ((kpos + e >= pg.first || kpos + e < sh.keep) && kpos + e <= pos) ? v[e] * sc : -INFINITY;
                         mx = fmaxf(mx, v[e]);
                     }
 #pragma unroll
@@ -257,10 +287,10 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
                     uint32_t a[4];
                     ldm_x4(a, p_addr + k * 32);
                     // value tiles: 16 keys x 16 columns per transposed load
-                    const uint32_t v_addr = st + ((16 * k + (lane & 15)) * pitch + warp * 8 * NT + (lane >> 4) * 8) * 2;
+                    const uint32_t v_addr = st + ((16 * k + (lane & 15)) * pitch + sh.vcol0 + warp * 8 * NT + (lane >> 4) * 8) * 2;
 #pragma unroll
                     for (int n = 0; n < NT; n += 2) {
-                        if (warp * 8 * NT + 8 * n >= sh.rank) break;      // tiles behind the latent: never stored, and past the stage's end
+                        if (warp * 8 * NT + 8 * n >= sh.vcols) break;     // tiles behind the values: never stored, and past the stage's end
                         uint32_t bb[4];
                         ldm_x4_t(bb, v_addr + n * 16);
                         mma_bf16(o[n], a, bb[0], bb[1]);
@@ -278,7 +308,31 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
             auto store = [&] {
                 const float i0 = 1.f / l0, i1 = 1.f / l1;
                 const int col = warp * 8 * NT + 2 * t4;
-                __nv_bfloat16* orow = out + ((size_t)g.row * sh.heads + g.hg * kHG) * sh.rank;
+                if constexpr (kDiff) {            // rows g4 and g4 + 8 are the two maps of one head
+                    float ss = 0.f;
+#pragma unroll
+                    for (int n = 0; n < NT; ++n) {
+                        const bool in = warp * 8 * NT + 8 * n < sh.vcols;
+                        o[n][0] = in ? o[n][0] * i0 - sh.lambda * (o[n][2] * i1) : 0.f;
+                        o[n][1] = in ? o[n][1] * i0 - sh.lambda * (o[n][3] * i1) : 0.f;
+                        ss += o[n][0] * o[n][0] + o[n][1] * o[n][1];
+                    }
+                    ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+                    ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+                    if (t4 == 0) s_ss[warp * 8 + g4] = ss;
+                    sync_consumers();
+                    ss = 0.f;
+#pragma unroll
+                    for (int w = 0; w < 8; ++w) ss += s_ss[w * 8 + g4];
+                    const float f = sh.out_scale / sqrtf(ss / (float)sh.vdim + sh.eps);
+                    if (g4 >= n_heads) return;
+                    __nv_bfloat16* dst = out + ((size_t)g.row * sh.heads + g.hg * sh.per + g4) * sh.vcols + col;
+#pragma unroll
+                    for (int n = 0; n < NT; ++n)
+                        if (col + 8 * n < sh.vcols) *reinterpret_cast<uint32_t*>(dst + 8 * n) = pack_bf16x2(o[n][0] * f, o[n][1] * f);
+                    return;
+                }
+                __nv_bfloat16* orow = out + ((size_t)g.row * sh.heads + g.hg * kHG) * sh.vcols;
 #pragma unroll
                 for (int n = 0; n < NT; ++n)
 #pragma unroll
@@ -286,12 +340,12 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
                         const int hd = g4 + 8 * e, c = col + 8 * n;
                         const float x = o[n][2 * e] * (e ? i1 : i0), y = o[n][2 * e + 1] * (e ? i1 : i0);
                         if (hd >= n_heads) continue;
-                        __nv_bfloat16* dst = orow + (size_t)hd * sh.rank + c;
-                        if ((sh.rank & 1) == 0) {
-                            if (c < sh.rank) *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(x, y);
+                        __nv_bfloat16* dst = orow + (size_t)hd * sh.vcols + c;
+                        if ((sh.vcols & 1) == 0) {
+                            if (c < sh.vcols) *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(x, y);
                         } else {
-                            if (c < sh.rank) dst[0] = __float2bfloat16_rn(x);
-                            if (c + 1 < sh.rank) dst[1] = __float2bfloat16_rn(y);
+                            if (c < sh.vcols) dst[0] = __float2bfloat16_rn(x);
+                            if (c + 1 < sh.vcols) dst[1] = __float2bfloat16_rn(y);
                         }
                     }
             };
@@ -355,22 +409,18 @@ latent_decode_kernel(const LatentShape sh, const __nv_bfloat16* __restrict__ qa,
     if (tid == 0 && *abort_flag) atomicExch(cache.error, 3);
 }
 
-static int ld_tiles(int rank) { return rank <= 64 ? 1 : rank <= 128 ? 2 : rank <= 256 ? 4 : 8; }
-static int ld_steps(const LatentShape& sh) { return ceil_div(sh.row_pitch() - 8, 64); }       // contraction steps per warp
+static int ld_tiles(int vcols) { return vcols <= 64 ? 1 : vcols <= 128 ? 2 : vcols <= 256 ? 4 : 8; }
 
-bool latent_decode_fits(const LatentShape& sh, int max_rows) {
-    return sh.rank <= 512 && ld_steps(sh) <= 12 && max_rows <= kLdMaxRows && ld_layout(sh.row_pitch(), max_rows).stages >= 2;
+static bool page_decode_fits(const LdShape& sh, int max_rows) {
+    return sh.vcols <= 512 && sh.ksteps <= 48 && max_rows <= kLdMaxRows && ld_layout(sh.pitch, sh.qpitch, max_rows).stages >= 2;
 }
 
-size_t latent_decode_scratch_floats(const LatentShape& sh, int max_rows) {
-    return (size_t)max_rows * ceil_div(sh.heads, kHG) * kLdParts * (ld_tiles(sh.rank) * 1024 + 32);
-}
-
-int launch_latent_decode(const LatentShape& sh, const void* qa, const LatentView& cache, const int* row_slot, const int* row_pos, int rows,
-                         float* part, int* counters, void* out, cudaStream_t s) {
+template <bool kDiff>
+static int launch_page_decode(const LdShape& sh, const void* qa, const LatentView& cache, const int* row_slot, const int* row_pos, int rows, float* part,
+                              int* counters, void* out, cudaStream_t s) {
     int n_sm = 0;
     B2_TRY(device_sm_count(&n_sm));
-    const uint32_t smem = ld_layout(sh.row_pitch(), rows).total;
+    const uint32_t smem = ld_layout(sh.pitch, sh.qpitch, rows).total;
     unsigned long long* stamp = prof_stamp_slot(PROF_FA_DECODE);
     auto go = [&](auto kernel) {
         launch_pdl(kernel, dim3(n_sm), dim3(kLdThreads), smem, s, sh, (const __nv_bfloat16*)qa, cache, row_slot, row_pos, rows, part, counters,
@@ -380,15 +430,16 @@ int launch_latent_decode(const LatentShape& sh, const void* qa, const LatentView
         constexpr int NT = decltype(nt)::value;
         static PerDeviceOnce once;
         B2_PER_DEVICE_ONCE(once,
-            B2_CUDA(cudaFuncSetAttribute(latent_decode_kernel<NT, 3>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
-            B2_CUDA(cudaFuncSetAttribute(latent_decode_kernel<NT, 9>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
-            B2_CUDA(cudaFuncSetAttribute(latent_decode_kernel<NT, 12>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024)));
-        if (ld_steps(sh) <= 3) go(latent_decode_kernel<NT, 3>);
-        else if (ld_steps(sh) <= 9) go(latent_decode_kernel<NT, 9>);
-        else go(latent_decode_kernel<NT, 12>);
+            B2_CUDA(cudaFuncSetAttribute(page_decode_kernel<NT, 3, kDiff>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+            B2_CUDA(cudaFuncSetAttribute(page_decode_kernel<NT, 9, kDiff>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+            B2_CUDA(cudaFuncSetAttribute(page_decode_kernel<NT, 12, kDiff>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024)));
+        const int kq = ceil_div(sh.ksteps, 4);                    // contraction steps per warp
+        if (kq <= 3) go(page_decode_kernel<NT, 3, kDiff>);
+        else if (kq <= 9) go(page_decode_kernel<NT, 9, kDiff>);
+        else go(page_decode_kernel<NT, 12, kDiff>);
         return 0;
     };
-    switch (ld_tiles(sh.rank)) {
+    switch (ld_tiles(sh.vcols)) {
         case 1: B2_TRY(pick(std::integral_constant<int, 1>{})); break;
         case 2: B2_TRY(pick(std::integral_constant<int, 2>{})); break;
         case 4: B2_TRY(pick(std::integral_constant<int, 4>{})); break;
@@ -396,6 +447,63 @@ int launch_latent_decode(const LatentShape& sh, const void* qa, const LatentView
     }
     B2_LAUNCH_CHECK();
     return 0;
+}
+
+constexpr float kLdLog2e = 1.4426950408889634f;
+
+static LdShape latent_rows(const LatentShape& sh) {
+    LdShape r{};
+    r.pitch = r.qpitch = sh.row_pitch();
+    r.groups = ceil_div(sh.heads, kHG);
+    r.ksteps = (sh.row_pitch() - 8) / 16;
+    r.vcols = sh.rank;
+    r.window = sh.window;
+    r.sc = sh.scale * kLdLog2e;
+    r.heads = sh.heads;
+    r.per = kHG;
+    return r;
+}
+
+bool latent_decode_fits(const LatentShape& sh, int max_rows) { return page_decode_fits(latent_rows(sh), max_rows); }
+
+size_t latent_decode_scratch_floats(const LatentShape& sh, int max_rows) {
+    return (size_t)max_rows * ceil_div(sh.heads, kHG) * kLdParts * (ld_tiles(sh.rank) * 1024 + 32);
+}
+
+int launch_latent_decode(const LatentShape& sh, const void* qa, const LatentView& cache, const int* row_slot, const int* row_pos, int rows,
+                         float* part, int* counters, void* out, cudaStream_t s) {
+    return launch_page_decode<false>(latent_rows(sh), qa, cache, row_slot, row_pos, rows, part, counters, out, s);
+}
+
+static LdShape diff_rows(const DiffShape& sh, float lambda) {
+    LdShape r{};
+    r.pitch = sh.hp();
+    r.qpitch = sh.qp();
+    r.groups = sh.kv_heads;
+    r.ksteps = 2 * sh.dp / 16;
+    r.vcol0 = 2 * sh.dp;
+    r.vcols = sh.vp;
+    r.window = sh.window;
+    r.keep = sh.keep;
+    r.sc = sh.scale * kLdLog2e;
+    r.heads = sh.heads;
+    r.per = sh.heads / sh.kv_heads;
+    r.vdim = sh.vdim;
+    r.lambda = lambda;
+    r.out_scale = 1.0f - sh.diff;
+    r.eps = sh.eps;
+    return r;
+}
+
+bool diff_decode_fits(const DiffShape& sh, int max_rows) { return sh.heads / sh.kv_heads <= 8 && page_decode_fits(diff_rows(sh, 0.f), max_rows); }
+
+size_t diff_decode_scratch_floats(const DiffShape& sh, int max_rows) {
+    return (size_t)max_rows * sh.kv_heads * kLdParts * (ld_tiles(sh.vp) * 1024 + 32);
+}
+
+int launch_diff_decode(const DiffShape& sh, float lambda, const void* qd, const LatentView& cache, const int* row_slot, const int* row_pos, int rows,
+                       float* part, int* counters, void* out, cudaStream_t s) {
+    return launch_page_decode<true>(diff_rows(sh, lambda), qd, cache, row_slot, row_pos, rows, part, counters, out, s);
 }
 
 }  // namespace b200

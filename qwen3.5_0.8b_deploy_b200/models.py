@@ -1,10 +1,11 @@
 """Model registry: config.json's "architecture" selects the entry that turns a configuration into a stack.
 
-An entry is a function (config, limits, ops) -> stack with its `load` method set on it through `load_tensors`; both kinds of
-stack share prefill, decode, capture and continuous batching (ops.Stack), so everything above works on either.
+An entry is a function (config, limits, shapes) -> stack, where `shapes` names the model's tensors with their shapes; `load_tensors`
+gives the stack its weights.  Both kinds of stack share prefill, decode, capture and continuous batching (ops.Stack), so everything above works on either.
 """
 from __future__ import annotations
 
+import ctypes
 import os
 from dataclasses import dataclass
 
@@ -65,7 +66,7 @@ def nuzopel_layers(config: dict, ops) -> list:
 
 
 @register("Nuzopel")
-def build_nuzopel(config: dict, limits: Limits):
+def build_nuzopel(config: dict, limits: Limits, shapes: dict):
     ops = _ops()
     cfg = ops.ModelConfig(config["width"], config["vocab"], limits.max_seqs, limits.max_seq_len, limits.num_pages, limits.max_pass_rows,
                           {"bfloat16": ops.DTYPE_BF16, "float32": ops.DTYPE_F32}[limits.dtype],
@@ -73,9 +74,48 @@ def build_nuzopel(config: dict, limits: Limits):
     return ops.LayerStack(cfg, nuzopel_layers(config, ops))
 
 
+# ---- Gutenex: lightning, channel-wise delta rule and differential attention, norms on the sublayers' inputs, looped layers ---
+def gutenex_layers(config: dict, shapes: dict, ops) -> list:
+    """`shapes`: tensor name -> shape; it alone gives the inner sizes of the low-rank gates."""
+    out = []
+    for i, layer in enumerate(config["layers"]):
+        m, mlp = layer["mixer"], layer["mlp"]
+        d = ops.LayerDesc(heads=m["heads"], dim=m["dim"], vdim=m["vdim"], kv_from=-1, act=ops.ACT_SILU)
+        if layer["type"] == "lightning":
+            if len(m["decay"]) != m["heads"]:
+                raise ValueError(f"layer {i}: {len(m['decay'])} decays for {m['heads']} heads")
+            d.mixer = ops.MIXER_LIGHTNING
+            d.decay = (ctypes.c_double * m["heads"])(*m["decay"])
+        elif layer["type"] == "channel_delta":
+            d.mixer, d.kv_heads, d.conv_taps = ops.MIXER_CHANNEL_DELTA, m["kv_heads"], m["conv"]
+            d.a_rank, d.g_rank = (shapes[f"l{i}.mix.{n}"][0] for n in ("a1", "g1"))
+        elif layer["type"] == "attention":
+            d.mixer, d.kv_heads, d.scale, d.diff = ops.MIXER_DIFF, m["kv_heads"], m["scale"], m["diff"]
+            d.window, d.keep_first = m["mask"]["size"], m["mask"]["keep_first"]
+            d.rot_dim, d.rot_base = m["rot"]["dims"], m["rot"]["base"]
+        else:
+            raise ValueError(f"layer {i}: unknown type {layer['type']!r}")
+        if mlp is not None:
+            if mlp["kind"] != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+            d.ff = mlp["ff"]
+        out.append(d)
+    return out
+
+
+@register("Gutenex")
+def build_gutenex(config: dict, limits: Limits, shapes: dict):
+    ops = _ops()
+    loop = config.get("loop") or dict(start=0, stop=0, times=1)
+    cfg = ops.ModelConfig(config["width"], config["vocab"], limits.max_seqs, limits.max_seq_len, limits.num_pages, limits.max_pass_rows,
+                          {"bfloat16": ops.DTYPE_BF16, "float32": ops.DTYPE_F32}[limits.dtype], config["norm"]["eps"], 1.0, 1.0,
+                          config["logit_softcap"], 1, 1, loop["start"], loop["stop"], loop["times"])
+    return ops.LayerStack(cfg, gutenex_layers(config, shapes, ops))
+
+
 # ---- the hybrid stack: Gated DeltaNet and gated full attention ---------------------------------------------------------------
 @register("Qwen3_5Hybrid")
-def build_hybrid(config: dict, limits: Limits):
+def build_hybrid(config: dict, limits: Limits, shapes: dict):
     """Keys: num_layers, intermediate_size, vocab_size, rms_eps, kv_dtype ("fp16" or "int8"), int8_weights."""
     ops = _ops()
     if limits.dtype != "bfloat16":
@@ -106,15 +146,16 @@ def load_tensors(stack, tensors: dict) -> None:
     stack.set_embedding(f32(tensors["embed"]), f32(tensors["final_norm"]))
 
 
-def build_model(config: dict, limits: Limits):
+def build_model(config: dict, limits: Limits, shapes: dict | None = None):
     arch = config.get("architecture")
     if arch not in REGISTRY:
         raise ValueError(f"unknown architecture {arch!r}; known: {sorted(REGISTRY)}")
-    return REGISTRY[arch](config, limits)
+    return REGISTRY[arch](config, limits, shapes or {})
 
 
 def load_model(folder: str, limits: Limits):
     """config.json and model.safetensors of `folder` -> a stack ready to run."""
-    stack = build_model(weights.read_config(folder), limits)
-    load_tensors(stack, weights.read_safetensors(os.path.join(folder, "model.safetensors")))
+    tensors = weights.read_safetensors(os.path.join(folder, "model.safetensors"))
+    stack = build_model(weights.read_config(folder), limits, {k: v.shape for k, v in tensors.items()})
+    load_tensors(stack, tensors)
     return stack

@@ -21,7 +21,8 @@ OK, ERR_INVALID, ERR_CUDA, ERR_NOMEM, ERR_NOT_READY, ERR_UNSUPPORTED, ERR_DEVICE
 PROJ_FP32, PROJ_FP16 = 0, 1
 KV_INT8, KV_FP16 = 0, 1
 DTYPE_BF16, DTYPE_F32 = 0, 1
-MIXER_MLSTM, MIXER_LATENT = 1, 2
+MIXER_MLSTM, MIXER_LATENT, MIXER_LIGHTNING, MIXER_CHANNEL_DELTA, MIXER_DIFF = 1, 2, 3, 4, 5
+ACT_GELU_TANH, ACT_SILU = 0, 1
 
 # Every symbol include/b200attn.h declares (tests check the library exports exactly these).
 ABI_SYMBOLS = [
@@ -145,12 +146,15 @@ class StackConfig(C.Structure):
 
 class ModelConfig(C.Structure):
     _fields_ = [(n, C.c_int) for n in ("width", "vocab_size", "max_seqs", "max_seq_len", "num_pages", "max_pass_rows", "dtype")] + \
-               [(n, C.c_double) for n in ("norm_eps", "embed_scale", "logit_scale")]
+               [(n, C.c_double) for n in ("norm_eps", "embed_scale", "logit_scale", "logit_softcap")] + \
+               [(n, C.c_int) for n in ("pre_norm", "own_head", "loop_start", "loop_stop", "loop_times")]
 
 
 class LayerDesc(C.Structure):
     _fields_ = [("mixer", C.c_int), ("heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("gate_cap", C.c_double), ("kv_rank", C.c_int),
-                ("rot_dim", C.c_int), ("window", C.c_int), ("kv_from", C.c_int), ("rot_base", C.c_double), ("scale", C.c_double), ("ff", C.c_int)]
+                ("rot_dim", C.c_int), ("window", C.c_int), ("kv_from", C.c_int), ("rot_base", C.c_double), ("scale", C.c_double), ("ff", C.c_int)] + \
+               [(n, C.c_int) for n in ("act", "kv_heads", "conv_taps", "a_rank", "g_rank", "keep_first")] + \
+               [("diff", C.c_double), ("decay", C.POINTER(C.c_double))]
 
 
 class LayerWeights(C.Structure):

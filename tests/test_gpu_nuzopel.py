@@ -87,18 +87,22 @@ def make(layers, width=80, vocab=97, seed=0, eps=1e-5, embed_scale=3.0, logit_sc
 
 class Case:
     """A model in both implementations; weights rounded to bf16 for both."""
+    plain_model = plain.PlainModel
 
     def __init__(self, models, wts, cfg, tensors, dtype, **limits):
         self.bits = {k: wts.bf16_bits(v) for k, v in tensors.items()}
-        self.plain = plain.PlainModel(cfg, {k: wts.bf16_to_f32(v) for k, v in self.bits.items()})
+        self.plain = self.plain_model(cfg, {k: wts.bf16_to_f32(v) for k, v in self.bits.items()})
         args = dict(max_seqs=4, max_seq_len=1024, num_pages=0, max_pass_rows=0, dtype=dtype)
         args.update(limits)
-        self.stack = models.build_model(cfg, models.Limits(**args))
+        self.stack = models.build_model(cfg, models.Limits(**args), {k: v.shape for k, v in self.bits.items()})
         models.load_tensors(self.stack, self.bits)
         self.cfg, self.dtype, self.vocab = cfg, dtype, cfg["vocab"]
 
     def tokens(self, n, seed=1):
         return np.random.default_rng(seed).integers(0, self.vocab, n)
+
+    def residual_unit(self, residual):
+        return 1.0                          # norms on the sublayers' outputs
 
     def expect(self, tokens):
         """Logits, residual stream, and the limits of the two by row."""
@@ -109,7 +113,7 @@ class Case:
         for seed in range(3):
             rng, tr = np.random.default_rng(seed), []
             lg = self.plain.forward(self.plain.start(), tokens, tr, lambda a: a * (1.0 + 1.2e-3 * rng.standard_normal(a.shape)))
-            for k, (d, unit) in enumerate(((lg - logits, std), (tr[-1] - trace[-1], 1.0))):
+            for k, (d, unit) in enumerate(((lg - logits, std), (tr[-1] - trace[-1], self.residual_unit(trace[-1])))):
                 worst[k] = np.maximum(worst[k], np.sqrt(np.mean((d / unit) ** 2, axis=-1)))
         return logits, trace[-1], FLOOR[self.dtype] + 8.0 * SHARE[self.dtype] * worst
 
@@ -126,7 +130,7 @@ class Case:
         return torch.cat(out).cpu().numpy(), torch.cat(res).cpu().numpy()
 
     def judge(self, got, want, what=""):
-        for k, (name, unit) in enumerate((("logits", max(float(np.std(want[0])), 1e-3)), ("residual", 1.0))):
+        for k, (name, unit) in enumerate((("logits", max(float(np.std(want[0])), 1e-3)), ("residual", self.residual_unit(want[1])))):
             assert np.isfinite(got[k]).all(), f"{what}: {name} not finite"
             row = np.sqrt(np.mean(((got[k] - want[k]) / unit) ** 2, axis=-1))
             ratio = row / want[2][k]
