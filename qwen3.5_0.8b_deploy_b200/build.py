@@ -18,7 +18,7 @@ OUT = os.path.join(HERE, "libb200attn.so")
 OBJ = os.path.join(HERE, "build")
 SOURCES = ["gemm.cu", "kv_cache.cu", "fa_decode.cu", "fa_prefill.cu", "fa_ops.cu", "la_kernels.cu", "la_chunk.cu",
            "la_ops.cu", "stack.cu", "fa_decode_static.cu", "gemm_tc.cu",
-           "block_model.cu", "block_mixers.cu", "block_kernels.cu", "channel_delta.cu", "diff_attn.cu", "diff_prefill.cu", "mlstm.cu", "mlstm_chunk.cu", "latent.cu", "page_decode.cu", "latent_prefill.cu"]
+           "block_model.cu", "block_mixers.cu", "block_kernels.cu", "channel_delta.cu", "channel_delta_chunk.cu", "diff_attn.cu", "diff_prefill.cu", "mlstm.cu", "mlstm_chunk.cu", "latent.cu", "page_decode.cu", "latent_prefill.cu"]
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "-Xcompiler", "-fPIC",
          "--expt-relaxed-constexpr", "-Xptxas", "-v"]

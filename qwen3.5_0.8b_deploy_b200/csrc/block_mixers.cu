@@ -103,7 +103,12 @@ int make_delta(const b200attn_layer_desc& d, const b200attn_model_config& c, Ele
     z.low = std::max(z.low, (size_t)sh.low());
     z.gates = std::max(z.gates, (size_t)sh.gate_cols());
     z.mixed = std::max(z.mixed, (size_t)sh.heads * sh.vp);
-    if (sh.n_vt > 1) z.core = std::max(z.core, (size_t)sh.heads * sh.vp);
+    op.chunk = elem == ELEM_BF16 && delta_chunk_fits(sh);
+    if (op.chunk) {
+        z.gates = std::max(z.gates, (size_t)sh.gate_cols() + sh.heads);
+        z.chunk = std::max(z.chunk, delta_chunk_bytes(sh));
+    }
+    if (op.chunk || sh.n_vt > 1) z.core = std::max(z.core, (size_t)sh.heads * sh.vp);
     return op.norm_w.alloc((size_t)sh.vp * 4);
 }
 
@@ -150,6 +155,23 @@ int delta_forward(BlockModel& m, DeltaOp& op, const LayerRun& run, const PassRow
     const int W = m.cfg.width;
     float* state = m.state->d_recurrent + m.state->block_offset[run.state_layer];
     B2_TRY(gemm_typed(s, m.xt.p, W, op.w_low.p, m.low.p, sh.low(), op.elem, op.elem, p.rows, sh.low(), W));
+    if (!p.decode && op.chunk && p.max_count >= 16) {
+        // q | k | v in bf16; decay and beta pre-activations in fp32, those of the output gate in bf16 behind them
+        const int acols = sh.heads * sh.dp, gcols = sh.heads * sh.vp, qkv = sh.off_b();
+        float *a = m.gates.f(), *b = a + (size_t)p.rows * acols;
+        void* g = b + ((size_t)p.rows * sh.heads + 3) / 4 * 4;
+        const size_t e = elem_bytes(op.elem);
+        B2_TRY(gemm_typed(s, m.xt.p, W, op.w_in.p, m.proj.p, qkv, op.elem, op.elem, p.rows, qkv, W));
+        B2_TRY(gemm_typed(s, m.xt.p, W, (const char*)op.w_in.p + (size_t)qkv * W * e, b, sh.heads, op.elem, ELEM_F32, p.rows, sh.heads, W));
+        B2_TRY(gemm_typed(s, m.low.p, sh.low(), op.w_gate.p, a, acols, op.elem, ELEM_F32, p.rows, acols, sh.low()));
+        B2_TRY(gemm_typed(s, m.low.p, sh.low(), (const char*)op.w_gate.p + (size_t)acols * sh.low() * e, g, gcols, op.elem, op.elem, p.rows, gcols, sh.low()));
+        {
+            ProfScope prof(PROF_LA_PREFILL, s);
+            B2_TRY(launch_delta_chunk(sh, m.proj.p, a, b, op.conv.f(), op.a_log.f(), op.dt_bias.f(), p.d_seqs, p.n_seqs, p.max_count, m.cfg.max_seqs, state,
+                                      m.chunk.p, m.core.f(), m.error.i(), s));
+        }
+        return launch_delta_head_norm(op.elem, sh, m.core.f(), g, false, gcols, op.norm_w.f(), p.rows, m.mixed.p, s);
+    }
     B2_TRY(gemm_typed(s, m.xt.p, W, op.w_in.p, m.proj.p, sh.pitch(), op.elem, ELEM_F32, p.rows, sh.pitch(), W));
     B2_TRY(gemm_typed(s, m.low.p, sh.low(), op.w_gate.p, m.gates.p, sh.gate_cols(), op.elem, ELEM_F32, p.rows, sh.gate_cols(), sh.low()));
     DeltaStepArgs a{sh, m.proj.f(), m.gates.f(), op.conv.f(), op.a_log.f(), op.dt_bias.f(), op.norm_w.f(), state, p.decode ? p.d_slots : nullptr,

@@ -217,6 +217,7 @@ int block_model_create(const b200attn_model_config* cfg, const b200attn_layer_de
     B2_TRY(m.r_stage.alloc((size_t)m.ctx_rows * z.rst * e));
     B2_TRY(m.k_up.alloc((size_t)m.ctx_rows * z.kup * e));
     B2_TRY(m.v_up.alloc((size_t)m.ctx_rows * z.vup * e));
+    B2_TRY(m.chunk.alloc((R / 64 + m.max_spans + 1) * z.chunk));
     B2_TRY(m.part.alloc(z.part * 4));
     B2_TRY(m.counters.alloc(z.counters * 4));
     const size_t tiles = R / 128 + m.max_spans + 1;

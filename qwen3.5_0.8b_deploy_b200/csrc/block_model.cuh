@@ -215,6 +215,14 @@ int launch_delta_step(ElemType t, const DeltaStepArgs& a, int n, cudaStream_t s)
 int launch_delta_head_norm(ElemType t, const DeltaShape& sh, const float* core, const void* g, bool g_f32, int g_pitch, const float* norm_w, int rows,
                            void* gated, cudaStream_t s);
 
+// channel_delta_chunk.cu: prefill in chunks of 64 tokens.
+bool delta_chunk_fits(const DeltaShape& sh);
+size_t delta_chunk_bytes(const DeltaShape& sh);        // scratch per 64 rows of a pass (and one more such piece per sequence)
+// qkv: bf16 [rows][off_b]; a: fp32 [rows][heads * dp], b: fp32 [rows][heads], the gates' pre-activations.
+int launch_delta_chunk(const DeltaShape& sh, const void* qkv, const float* a, const float* b, const float* conv, const float* a_log, const float* dt_bias,
+                       const LaSeqMeta* d_seqs, int n_seqs, int max_count, int max_seqs, float* state, void* scratch, float* core, int* d_error,
+                       cudaStream_t s);
+
 struct DeltaOp {
     DeltaShape sh;
     ElemType elem = ELEM_BF16;
@@ -298,6 +306,7 @@ struct LayerRun {                      // one run of a layer in a pass over the 
 // What the mixers of a model need of the working buffers (per row unless said otherwise), gathered while its layers are made.
 struct BlockSizes {
     size_t proj = 0, mixed = 0, core = 0, gates = 0, low = 0, ff = 0, q = 0, qa = 0, olat = 0, cst = 0, rst = 0, kup = 0, vup = 0;
+    size_t chunk = 0;                  // bytes per 64 rows
     size_t part = 0, counters = 0;     // whole buffers
     int max_window = 0;
 };
@@ -314,7 +323,7 @@ struct BlockModel {
     int max_rows = 0, abs_rows = 0, ctx_rows = 0, max_spans = 0;
     b200attn_kv_pool pool = nullptr;   // owned by the stack
     b200attn_la_state state = nullptr;
-    DevBuf x, x0, xt, low, proj, gates, core, mixed, y, gu, act, q, qa, olat, c_stage, r_stage, k_up, v_up, part, counters, meta, error;
+    DevBuf x, x0, xt, low, proj, gates, core, mixed, y, gu, act, q, qa, olat, c_stage, r_stage, k_up, v_up, part, counters, chunk, meta, error;
     int* row_slot() const { return meta.i(); }
     int* row_pos() const { return meta.i() + max_rows; }
     LaSeqMeta* seqs() const { return reinterpret_cast<LaSeqMeta*>(meta.i() + 2 * (size_t)max_rows); }

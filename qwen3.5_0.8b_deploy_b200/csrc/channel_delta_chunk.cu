@@ -1,0 +1,781 @@
+// Chunk-64 prefill of the channel-wise gated delta rule (channel_delta.cu) in two kernels.
+//
+// With G_t the running sums of the log decays inside a chunk (one per key channel) and S_0 the state at its start:
+//     A_ts = beta_t sum_d k_t k_s e^{G_t - G_s}  (s < t),    M_ts = sum_d q_t k_s e^{G_t - G_s}  (s <= t),    T = (I + A)^-1
+//     W = T diag(beta) (e^G K),   U' = T diag(beta) V,   U = U' - W S_0
+//     O = (e^G Q) S_0 + M U,      S_C = diag(e^{G_C}) S_0 + (e^{G_C - G} K)^T U
+// Everything but the lines with S_0 needs no state: the first kernel does it for all chunks at once (convolutions, unit vectors and
+// gates included) and leaves W, e^G Q, e^{G_C - G} K, M and U' as images of the shared-memory tiles that the second kernel, which
+// walks the chunks of a sequence, multiplies with the state on tcgen05.
+//
+// A decay is always the product of factors <= 1, never a quotient: pairs of tokens inside a group of four get their factors as
+// running products in registers; pairs of groups inside a block of 16, and pairs of blocks, meet on mma.sync with the later
+// token decayed from the start of its group (block) and the earlier one decayed up to there, in one copy per later group (block).
+// Operands are fp16: unit vectors, decays, beta and T are at most 1, and 11 bits are kept of values.
+#include "block_model.cuh"
+#include "channel_delta.cuh"
+#include "delta_inverse.cuh"
+#include "elem.cuh"
+#include "tc05.cuh"
+
+#include <algorithm>
+
+namespace b200 {
+
+namespace {
+constexpr int kDC = 64;
+constexpr uint32_t kTile = kDC * 128;                  // 64 rows of 64 fp16, 128-byte swizzle
+constexpr float kDL2e = 1.4426950408889634f;
+
+// An item (chunk and head) of the scratch: W | e^G Q | e^{G_C - G} K (ND tiles each) | M | e^{G_C} | U' per state tile (NV tiles of [64 values][64 tokens])
+struct DeltaItem {
+    int nd, nv, n_vt;
+    __host__ __device__ uint32_t off_q() const { return nd * kTile; }
+    __host__ __device__ uint32_t off_k() const { return 2 * nd * kTile; }
+    __host__ __device__ uint32_t off_m() const { return 3 * nd * kTile; }
+    __host__ __device__ uint32_t off_e() const { return off_m() + kTile; }
+    __host__ __device__ uint32_t off_u() const { return off_e() + nd * 256; }
+    __host__ __device__ uint32_t bytes() const { return off_u() + n_vt * nv * kTile; }
+};
+// Items of a sequence start at row0 / 64 + its index: no two sequences meet.
+__device__ __forceinline__ size_t first_chunk(int row0, int seq) { return (size_t)(row0 / kDC) + seq; }
+
+__device__ __forceinline__ float ex2c(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ uint32_t sw(int r, int p) { return (uint32_t)(r * 128 + ((p ^ (r & 7)) << 4)); }   // 16-byte piece p of row r
+__device__ __forceinline__ float2 unpack_half2(uint32_t v) { return __half22float2(*reinterpret_cast<const __half2*>(&v)); }
+__device__ __forceinline__ void ldm4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldm4t(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldm2(uint32_t& a, uint32_t& b, uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(a), "=r"(b) : "r"(addr));
+}
+
+struct DeltaChunkArgs {
+    DeltaShape sh;
+    DeltaItem item;
+    const __nv_bfloat16* qkv;          // [rows][off_b]
+    const float* a;                    // [rows][heads * dp] decay pre-activations
+    const float* b;                    // [rows][heads]
+    const float *conv, *a_log, *dt_bias;
+    const float* state;
+    const LaSeqMeta* seqs;
+    int max_seqs;
+    unsigned char* scratch;
+};
+
+// Four consecutive tokens x eight channels behind a short convolution and silu; tokens before the pass come from hist
+// ([taps - 1][stride] floats, `hn` of the eight channels exist there), tokens from `count` on are zero.
+template <int TAPS>
+__device__ __forceinline__ void conv_piece(const __nv_bfloat16* raw, int pitch, const float* hist, int stride, int hn, const float* w, int taps, int t0,
+                                           int count, float (&o)[4][8]) {
+    auto row = [&](int t, float (&x)[8]) {
+        if (t >= count) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[e] = 0.f;
+        } else if (t >= 0) {
+            const uint4 v = *reinterpret_cast<const uint4*>(raw + (size_t)t * pitch);
+            const float2 a = unpack_bf16x2(v.x), b = unpack_bf16x2(v.y), c = unpack_bf16x2(v.z), d = unpack_bf16x2(v.w);
+            x[0] = a.x; x[1] = a.y; x[2] = b.x; x[3] = b.y; x[4] = c.x; x[5] = c.y; x[6] = d.x; x[7] = d.y;
+        } else {
+            const float* h = hist + (size_t)(taps - 1 + t) * stride;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[e] = e < hn ? h[e] : 0.f;
+        }
+    };
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o[i][e] = 0.f;
+    if constexpr (TAPS > 0) {
+        float wv[8 * TAPS];
+#pragma unroll
+        for (int i = 0; i < 2 * TAPS; ++i) {
+            const float4 v = *reinterpret_cast<const float4*>(w + 4 * i);
+            wv[4 * i] = v.x; wv[4 * i + 1] = v.y; wv[4 * i + 2] = v.z; wv[4 * i + 3] = v.w;
+        }
+#pragma unroll
+        for (int r = 1 - TAPS; r < 4; ++r) {
+            float x[8];
+            row(t0 + r, x);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int j = r - i + TAPS - 1;
+                if (j < 0 || j >= TAPS) continue;
+#pragma unroll
+                for (int e = 0; e < 8; ++e) o[i][e] += x[e] * wv[e * TAPS + j];
+            }
+        }
+    } else {
+        for (int j = 0; j < taps; ++j)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                float x[8];
+                row(t0 + i + j - taps + 1, x);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) o[i][e] += x[e] * w[e * taps + j];
+            }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o[i][e] = t0 + i < count ? __fdividef(o[i][e], 1.0f + __expf(-o[i][e])) : 0.f;
+}
+
+// Shared memory of the first kernel; rows of K-major tiles are 64 ND + 8 halves apart (an odd number of 16-byte units).
+constexpr uint32_t kRegion = 17408;                    // 64 rows of 136 halves
+constexpr uint32_t kOffKA = 0;                         // decayed keys (rows), e^G K, then the image of U'
+constexpr uint32_t kOffQA = kRegion;                   // decayed queries (rows), then V
+constexpr uint32_t kOffKB = 2 * kRegion;               // keys decayed to the end of their group, then the image of W
+constexpr uint32_t kOffCOL = 3 * kRegion;              // 96 rows of decayed keys (columns), then T
+constexpr uint32_t kOffAM = kOffCOL + 26112;           // A, fp32 [64][kLd]
+constexpr uint32_t kOffM = kOffAM + 17408;             // image of M
+constexpr uint32_t kOffG = kOffM + kTile;              // [17][64 ND] log2 decays up to the start of every group
+constexpr uint32_t kOffB = kOffG + 17 * 128 * 4;       // beta [64]
+constexpr uint32_t kPrepSmem = kOffB + 256;
+}  // namespace
+
+// grid (heads, chunks, sequences), block 256, two CTAs per SM.  Thread (tg, c8): tokens 4 tg .. 4 tg + 3, channels 8 c8 .. 8 c8 + 7.
+template <int ND, int TAPS>
+__global__ void __launch_bounds__(256, 2)
+delta_prep_kernel(const DeltaChunkArgs A) {
+    extern __shared__ __align__(128) unsigned char sm[];
+    constexpr int DK = 64 * ND, LN = 8 * ND, kP = DK + 8;          // channels, lanes per token, row pitch in halves
+    const DeltaShape& sh = A.sh;
+    const LaSeqMeta sq = A.seqs[blockIdx.z];
+    const int h = blockIdx.x, chunk = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
+    if (chunk * kDC >= sq.count || sq.slot < 0 || sq.slot >= A.max_seqs) return;
+    const uint32_t base = smem_u32(sm);
+    float* AM = reinterpret_cast<float*>(sm + kOffAM);
+    float* TF = reinterpret_cast<float*>(sm + kOffCOL);
+    float* s_g = reinterpret_cast<float*>(sm + kOffG);
+    float* s_beta = reinterpret_cast<float*>(sm + kOffB);
+    unsigned char* item = A.scratch + ((first_chunk(sq.row0, blockIdx.z) + chunk) * sh.heads + h) * A.item.bytes();
+    const int tok0 = chunk * kDC, left = sq.count - tok0, D4 = (sh.dim + 3) / 4 * 4, taps = sh.taps;
+    const float* st = A.state + (size_t)sq.slot * sh.state_floats() + (size_t)h * sh.n_vt * sh.tile_floats();
+
+    for (int i = tid; i < 64 * kLd / 4; i += 256) reinterpret_cast<float4*>(AM)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = tid; i < (int)kTile / 16; i += 256) reinterpret_cast<uint4*>(sm + kOffM)[i] = make_uint4(0u, 0u, 0u, 0u);
+    if (tid < 64) s_beta[tid] = tid < left ? 1.0f / (1.0f + __expf(-A.b[(size_t)(sq.row0 + tok0 + tid) * sh.heads + h])) : 0.f;
+
+    const int tg = tid / LN, c8 = tid % LN, ch = 8 * c8, t0 = 4 * tg;
+    const bool act = tg < 16;                                       // whole warps
+    uint32_t qh[4][4], kh[4][4];                                    // unit vectors, fp16 pairs
+    float g[4][8];                                                  // decays of the four tokens
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) qh[i][e] = kh[i][e] = 0u;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) g[i][e] = 1.f;
+    }
+    if (act) {
+        const bool in = ch < sh.dp;
+        const int kvh = h / (sh.heads / sh.kv_heads), hn = min(8, sh.dim - ch);
+        const float* hist = st + (size_t)sh.dim * sh.vt;
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+            const int col = n * sh.off_k() + kvh * sh.dp + ch;
+            float o[4][8];
+            if (in) {
+                conv_piece<TAPS>(A.qkv + (size_t)sq.row0 * sh.off_b() + col, sh.off_b(), hist + n * (taps - 1) * D4 + ch, D4, hn, A.conv + (size_t)col * taps,
+                                 taps, tok0 + t0, sq.count, o);
+            } else {
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) o[i][e] = 0.f;
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                float ss = 0.f;
+#pragma unroll
+                for (int e = 0; e < 8; ++e) ss += o[i][e] * o[i][e];
+#pragma unroll
+                for (int x = LN / 2; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+                const float inv = (n ? 1.0f : 1.0f / sqrtf((float)sh.dim)) / sqrtf(ss + 1e-6f);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) (n ? kh : qh)[i][e] = pack_half2(o[i][2 * e] * inv, o[i][2 * e + 1] * inv);
+            }
+        }
+        float sum[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+        if (in) {
+            const float ea = -expf(A.a_log[h]) * kDL2e;
+            float dt[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) dt[e] = A.dt_bias[h * sh.dp + ch + e];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                if (t0 + i >= left) continue;
+                const float* z = A.a + (size_t)(sq.row0 + tok0 + t0 + i) * (sh.heads * sh.dp) + h * sh.dp + ch;
+                const float4 z0 = load4(z), z1 = load4(z + 4);
+                const float zz[8] = {z0.x, z0.y, z0.z, z0.w, z1.x, z1.y, z1.z, z1.w};
+#pragma unroll
+                for (int e = 0; e < 8; ++e) {
+                    const float l = ea * delta_softplus_fast(zz[e] + dt[e]);
+                    sum[e] += l;
+                    g[i][e] = ex2c(l);
+                }
+            }
+        }
+        store4(s_g + (tg + 1) * DK + ch, make_float4(sum[0], sum[1], sum[2], sum[3]));
+        store4(s_g + (tg + 1) * DK + ch + 4, make_float4(sum[4], sum[5], sum[6], sum[7]));
+    }
+    __syncthreads();
+    if (tid < DK) {                                                 // log2 decays from the chunk's start to the start of every group
+        float run = 0.f;
+        s_g[tid] = 0.f;
+#pragma unroll
+        for (int j = 1; j <= 16; ++j) { run += s_g[j * DK + tid]; s_g[j * DK + tid] = run; }
+        reinterpret_cast<float*>(item + A.item.off_e())[tid] = ex2c(run);
+    }
+    if (act) {
+        // ---- pairs inside the group: factors are running products ----
+        float acc[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) acc[i] = 0.f;
+#pragma unroll
+        for (int e2 = 0; e2 < 4; ++e2) {
+            float2 q[4], k[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) { q[i] = unpack_half2(qh[i][e2]); k[i] = unpack_half2(kh[i][e2]); }
+            int na = 0, nm = 6;
+#pragma unroll
+            for (int t = 0; t < 4; ++t) {
+#pragma unroll
+                for (int s = 0; s <= t; ++s) {
+                    float wx = k[s].x, wy = k[s].y;
+#pragma unroll
+                    for (int j = s + 1; j <= t; ++j) { wx *= g[j][2 * e2]; wy *= g[j][2 * e2 + 1]; }
+                    if (s < t) { acc[na] += k[t].x * wx + k[t].y * wy; ++na; }
+                    acc[nm] += q[t].x * wx + q[t].y * wy;
+                    ++nm;
+                }
+            }
+        }
+        // sixteen sums over the lanes of a token: halve the values while halving the lanes
+        int n = 16, at = 0;
+#pragma unroll
+        for (int x = LN / 2; x > 0; x >>= 1) {
+            n >>= 1;
+            const bool top = c8 & x;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                if (e >= n) continue;
+                const float y = __shfl_xor_sync(0xffffffffu, top ? acc[e] : acc[e + n], x);
+                acc[e] = (top ? acc[e + n] : acc[e]) + y;
+            }
+            if (top) at += n;
+        }
+#pragma unroll
+        for (int e = 0; e < 2 / ND; ++e) {
+            const int idx = at + e;
+            // pairs (t, s): A: 10 20 21 30 31 32, M: 00 10 11 20 21 22 30 31 32 33, packed as 4 t + s
+            const uint32_t packed = idx < 8 ? 0x40EDC984u : 0xFEDCA985u;
+            const int p = (int)(packed >> (4 * (idx & 7))) & 15, t = t0 + (p >> 2), s = t0 + (p & 3);
+            if (idx < 6) AM[t * kLd + s] = s_beta[t] * acc[e];
+            else *reinterpret_cast<__half*>(sm + kOffM + sw(t, s >> 3) + 2 * (s & 7)) = __float2half_rn(acc[e]);
+        }
+    }
+    __syncthreads();
+    const float* r0 = s_g + tg * DK + ch;                           // up to this group's start / end, up to the chunk's end
+    const float *r1 = r0 + DK, *rC = s_g + 16 * DK + ch;
+    auto piece = [&](uint32_t off, int row) { return reinterpret_cast<uint4*>(sm + off + row * kP * 2 + ch * 2); };
+    auto scaled = [](uint4 v, const float (&f)[8]) {
+        const float2 a = unpack_half2(v.x), b = unpack_half2(v.y), c = unpack_half2(v.z), d = unpack_half2(v.w);
+        return make_uint4(pack_half2(a.x * f[0], a.y * f[1]), pack_half2(b.x * f[2], b.y * f[3]), pack_half2(c.x * f[4], c.y * f[5]),
+                          pack_half2(d.x * f[6], d.y * f[7]));
+    };
+    auto factors = [](float (&f)[8], const float* to, const float* from) {     // 2^(to - from)
+        const float4 a = load4(to), b = load4(to + 4), c = load4(from), d = load4(from + 4);
+        f[0] = ex2c(a.x - c.x); f[1] = ex2c(a.y - c.y); f[2] = ex2c(a.z - c.z); f[3] = ex2c(a.w - c.w);
+        f[4] = ex2c(b.x - d.x); f[5] = ex2c(b.y - d.y); f[6] = ex2c(b.z - d.z); f[7] = ex2c(b.w - d.w);
+    };
+    const int blk = tg >> 2, own = tg & 3;
+    if (act) {
+        unsigned char* img = item + (c8 >> 3) * kTile;
+        {
+            float f[8], x[8];
+            factors(x, r0, s_g + ch);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) f[e] = 1.f;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) f[e] *= g[i][e];
+                const uint4 q = scaled(make_uint4(qh[i][0], qh[i][1], qh[i][2], qh[i][3]), f);
+                *piece(kOffQA, t0 + i) = q;
+                *piece(kOffKA, t0 + i) = scaled(make_uint4(kh[i][0], kh[i][1], kh[i][2], kh[i][3]), f);
+                *reinterpret_cast<uint4*>(img + A.item.off_q() + sw(t0 + i, c8 & 7)) = scaled(q, x);
+            }
+        }
+        {
+            float f[8], x[8];
+            factors(x, rC, r1);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) f[e] = 1.f;
+#pragma unroll
+            for (int i = 3; i >= 0; --i) {
+                const uint4 k = scaled(make_uint4(kh[i][0], kh[i][1], kh[i][2], kh[i][3]), f);
+                *piece(kOffKB, t0 + i) = k;
+                *reinterpret_cast<uint4*>(img + A.item.off_k() + sw(t0 + i, c8 & 7)) = scaled(k, x);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) f[e] *= g[i][e];
+            }
+        }
+        // copies for the later groups of the block: 24 rows per block, 4 + 8 + 12
+#pragma unroll 1
+        for (int i = own + 1; i < 4; ++i) {
+            float f[8];
+            factors(f, s_g + (4 * blk + i) * DK + ch, r1);
+            const int row = 24 * blk + (i == 1 ? 0 : i == 2 ? 4 : 12) + 4 * own;
+#pragma unroll
+            for (int s = 0; s < 4; ++s) *piece(kOffCOL, row + s) = scaled(*piece(kOffKB, t0 + s), f);
+        }
+    }
+    __syncthreads();
+    auto a_addr = [&](uint32_t off, int row) { return base + off + ((row + (lane & 15)) * kP + (lane >> 4) * 8) * 2; };
+    auto b_addr = [&](uint32_t off, int row) { return base + off + ((row + (lane & 7)) * kP + ((lane >> 3) & 1) * 8) * 2; };
+    auto put2 = [&](bool q, int t, int s, float x, float y) {       // entries (t, s), (t, s + 1) of M or A
+        if (q) *reinterpret_cast<uint32_t*>(sm + kOffM + sw(t, s >> 3) + 2 * (s & 7)) = pack_half2(x, y);
+        else *reinterpret_cast<float2*>(AM + t * kLd + s) = make_float2(s_beta[t] * x, s_beta[t] * y);
+    };
+    {   // ---- groups against groups: a block's 16 rows x 24 columns per warp ----
+        const int b = warp >> 1;
+        const bool q = warp & 1;
+        float d[3][4];
+#pragma unroll
+        for (int n = 0; n < 3; ++n) d[n][0] = d[n][1] = d[n][2] = d[n][3] = 0.f;
+        const uint32_t aa = a_addr(q ? kOffQA : kOffKA, 16 * b), ba = b_addr(kOffCOL, 24 * b);
+#pragma unroll
+        for (int k = 0; k < 4 * ND; ++k) {
+            uint32_t a[4], b0, b1;
+            ldm4(a, aa + k * 32);
+#pragma unroll
+            for (int n = 0; n < 3; ++n) {
+                ldm2(b0, b1, ba + n * 8 * kP * 2 + k * 32);
+                mma_16816(d[n], a[0], a[1], a[2], a[3], b0, b1);
+            }
+        }
+#pragma unroll
+        for (int n = 0; n < 3; ++n) {
+            const int c = 8 * n + 2 * t4, i = c < 4 ? 1 : c < 12 ? 2 : 3, s = 16 * b + c - (i == 1 ? 0 : i == 2 ? 4 : 12);
+            if ((g4 >> 2) == i) put2(q, 16 * b + g4, s, d[n][0], d[n][1]);
+            if (((g4 + 8) >> 2) == i) put2(q, 16 * b + g4 + 8, s, d[n][2], d[n][3]);
+        }
+    }
+    __syncthreads();
+    if (act) {
+        // ---- rows decay on from the start of their block, columns up to the start of a later one: 16 + 32 + 48 rows ----
+        float f[8];
+        factors(f, r0, s_g + 4 * blk * DK + ch);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            *piece(kOffQA, t0 + i) = scaled(*piece(kOffQA, t0 + i), f);
+            *piece(kOffKA, t0 + i) = scaled(*piece(kOffKA, t0 + i), f);
+        }
+#pragma unroll 1
+        for (int I = blk + 1; I < 4; ++I) {
+            factors(f, s_g + 4 * I * DK + ch, r1);
+            const int row = (I == 1 ? 0 : I == 2 ? 16 : 48) + t0;
+#pragma unroll
+            for (int s = 0; s < 4; ++s) *piece(kOffCOL, row + s) = scaled(*piece(kOffKB, t0 + s), f);
+        }
+    }
+    __syncthreads();
+#pragma unroll 1
+    for (int u = warp; u < 24; u += 8) {   // ---- blocks against blocks: 16 rows x 8 columns at a time ----
+        const bool q = u & 1;
+        const int v = u >> 1, I = v < 2 ? 1 : v < 6 ? 2 : 3, n = v - (I == 1 ? 0 : I == 2 ? 2 : 6);
+        float d[4] = {0.f, 0.f, 0.f, 0.f};
+        const uint32_t aa = a_addr(q ? kOffQA : kOffKA, 16 * I), ba = b_addr(kOffCOL, (I == 1 ? 0 : I == 2 ? 16 : 48) + 8 * n);
+#pragma unroll
+        for (int k = 0; k < 4 * ND; ++k) {
+            uint32_t a[4], b0, b1;
+            ldm4(a, aa + k * 32);
+            ldm2(b0, b1, ba + k * 32);
+            mma_16816(d, a[0], a[1], a[2], a[3], b0, b1);
+        }
+        put2(q, 16 * I + g4, 8 * n + 2 * t4, d[0], d[1]);
+        put2(q, 16 * I + g4 + 8, 8 * n + 2 * t4, d[2], d[3]);
+    }
+    __syncthreads();
+    // ---- T = (I + A)^-1 over the column copies; meanwhile M goes out and the keys decay from the chunk's start ----
+    if (tid < 64) invert_diagonal(AM, TF, tid);
+    for (int i = tid; i < (int)kTile / 16; i += 256) reinterpret_cast<uint4*>(item + A.item.off_m())[i] = reinterpret_cast<uint4*>(sm + kOffM)[i];
+    if (act) {
+        float f[8];
+        factors(f, s_g + 4 * blk * DK + ch, s_g + ch);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) *piece(kOffKA, t0 + i) = scaled(*piece(kOffKA, t0 + i), f);
+    }
+    __syncthreads();
+    if (warp < 6) scale_blocks(AM, TF, warp, lane);
+    __syncthreads();
+    solve_columns(AM, TF, warp, lane);
+    // ---- the values of a state tile: behind their convolution, over the queries ----
+    const int nv = A.item.nv, vln = 8 * nv, kVP = 64 * nv + 8;      // lanes per token, row pitch
+    auto load_values = [&](int tile) {
+        const int vtg = tid / vln, vc = 8 * (tid % vln), c = tile * kMlstmTile + vc, t = 4 * vtg;
+        if (vtg >= 16) return;
+        float o[4][8];
+        if (c < sh.vp) {
+            const int col = sh.off_v() + h * sh.vp + c;
+            const float* hv = st + tile * sh.tile_floats() + (size_t)sh.dim * sh.vt + 2 * (taps - 1) * D4;
+            conv_piece<TAPS>(A.qkv + (size_t)sq.row0 * sh.off_b() + col, sh.off_b(), hv + vc, sh.vt, min(8, sh.vdim - c), A.conv + (size_t)col * taps, taps,
+                             tok0 + t, sq.count, o);
+        } else {
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int e = 0; e < 8; ++e) o[i][e] = 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+            *reinterpret_cast<uint4*>(sm + kOffQA + ((t + i) * kVP + vc) * 2) =
+                make_uint4(pack_half2(o[i][0], o[i][1]), pack_half2(o[i][2], o[i][3]), pack_half2(o[i][4], o[i][5]), pack_half2(o[i][6], o[i][7]));
+    };
+    load_values(0);
+    __syncthreads();
+    // (T diag(beta)) entries (t, s), (t, s + 1) as fp16 hi and lo
+    auto t_pair = [&](int t, int s, uint32_t& hi, uint32_t& lo) {
+        const float2 v = *reinterpret_cast<const float2*>(TF + t * kLd + s), b = *reinterpret_cast<const float2*>(s_beta + s);
+        const float x = v.x * b.x, y = v.y * b.y;
+        hi = pack_half2(x, y);
+        const float2 hf = unpack_half2(hi);
+        lo = pack_half2(x - hf.x, y - hf.y);
+    };
+    {   // ---- W = (T diag(beta)) (e^G K): 16 rows x 32 ND columns per warp ----
+        const int i = warp >> 1, c0 = (warp & 1) * 32 * ND;
+        float d[4 * ND][4];
+#pragma unroll
+        for (int n = 0; n < 4 * ND; ++n) d[n][0] = d[n][1] = d[n][2] = d[n][3] = 0.f;
+        for (int k = 0; k <= i; ++k) {
+            uint32_t hi[4], lo[4];
+            t_pair(16 * i + g4, 16 * k + 2 * t4, hi[0], lo[0]);
+            t_pair(16 * i + g4 + 8, 16 * k + 2 * t4, hi[1], lo[1]);
+            t_pair(16 * i + g4, 16 * k + 2 * t4 + 8, hi[2], lo[2]);
+            t_pair(16 * i + g4 + 8, 16 * k + 2 * t4 + 8, hi[3], lo[3]);
+            const uint32_t ka = base + kOffKA + ((16 * k + (lane & 15)) * kP + c0 + (lane >> 4) * 8) * 2;
+#pragma unroll
+            for (int n = 0; n < 4 * ND; n += 2) {
+                uint32_t b[4];
+                ldm4t(b, ka + n * 16);
+                mma_16816(d[n], hi[0], hi[1], hi[2], hi[3], b[0], b[1]);
+                mma_16816(d[n], lo[0], lo[1], lo[2], lo[3], b[0], b[1]);
+                mma_16816(d[n + 1], hi[0], hi[1], hi[2], hi[3], b[2], b[3]);
+                mma_16816(d[n + 1], lo[0], lo[1], lo[2], lo[3], b[2], b[3]);
+            }
+        }
+#pragma unroll
+        for (int n = 0; n < 4 * ND; ++n) {
+            const int c = c0 + 8 * n;
+            unsigned char* w = sm + kOffKB + (c >> 6) * kTile;
+            *reinterpret_cast<uint32_t*>(w + sw(16 * i + g4, (c >> 3) & 7) + 4 * t4) = pack_half2(d[n][0], d[n][1]);
+            *reinterpret_cast<uint32_t*>(w + sw(16 * i + g4 + 8, (c >> 3) & 7) + 4 * t4) = pack_half2(d[n][2], d[n][3]);
+        }
+    }
+    __syncthreads();
+    for (int i = tid; i < (int)(ND * kTile) / 16; i += 256) reinterpret_cast<uint4*>(item)[i] = reinterpret_cast<uint4*>(sm + kOffKB)[i];
+    // ---- U'^T = V^T (T diag(beta))^T of every state tile: 16 values x 64 (or 32) tokens per warp ----
+    for (int tile = 0;; ++tile) {
+        const int mt = warp % (4 * nv), n0 = nv == 2 ? 0 : (warp >> 2) * 4, n1 = nv == 2 ? 8 : n0 + 4;
+        for (int n = n0; n < n1; ++n) {
+            float d[4] = {0.f, 0.f, 0.f, 0.f};
+            for (int k = 0; k <= n >> 1; ++k) {
+                uint32_t a[4], h0, l0, h1, l1;
+                ldm4t(a, base + kOffQA + ((16 * k + (lane & 7) + ((lane >> 4) & 1) * 8) * kVP + 16 * mt + ((lane >> 3) & 1) * 8) * 2);
+                t_pair(8 * n + g4, 16 * k + 2 * t4, h0, l0);
+                t_pair(8 * n + g4, 16 * k + 2 * t4 + 8, h1, l1);
+                mma_16816(d, a[0], a[1], a[2], a[3], h0, h1);
+                mma_16816(d, a[0], a[1], a[2], a[3], l0, l1);
+            }
+            *reinterpret_cast<uint32_t*>(sm + kOffKA + sw(16 * mt + g4, n) + 4 * t4) = pack_half2(d[0], d[1]);
+            *reinterpret_cast<uint32_t*>(sm + kOffKA + sw(16 * mt + g4 + 8, n) + 4 * t4) = pack_half2(d[2], d[3]);
+        }
+        __syncthreads();
+        uint4* dst = reinterpret_cast<uint4*>(item + A.item.off_u() + tile * nv * kTile);
+        for (int i = tid; i < (int)(nv * kTile) / 16; i += 256) dst[i] = reinterpret_cast<uint4*>(sm + kOffKA)[i];
+        if (tile + 1 == sh.n_vt) break;
+        load_values(tile + 1);
+        __syncthreads();
+    }
+}
+
+// ---- the walk over a sequence's chunks -----------------------------------------------------------------------------------------------
+namespace {
+constexpr int kWalkThreads = 288;                      // 8 compute warps, copies + MMA issuer
+constexpr uint32_t kOffWQ = 0;                         // W | e^G Q
+constexpr uint32_t kOffWK = 4 * kTile;                 // e^{G_C - G} K | M
+constexpr uint32_t kOffWS = 7 * kTile;                 // S_0^T [128 values][64 ND]
+constexpr uint32_t kOffWU = 11 * kTile;                // U^T [128 values][64 tokens]
+constexpr uint32_t kOffWE = 13 * kTile;                // e^{G_C}
+constexpr uint32_t kOffWBar = kOffWE + 512;
+constexpr uint32_t kWalkSmem = kOffWBar + 128;
+enum { W_WQ = 0, W_KM, W_B2, W_C2, W_B3, W_C3, W_BARS };
+}  // namespace
+
+// grid (heads * state tiles, sequences), two CTAs per SM.  TMEM: S^T (lane = value, up to 128 columns), X = S_0^T W^T, O^T.
+template <int ND, int NV>
+__global__ void __launch_bounds__(kWalkThreads, 2)
+delta_walk_kernel(const DeltaShape sh, const DeltaItem it, const __nv_bfloat16* __restrict__ qkv, const LaSeqMeta* __restrict__ seqs, int max_seqs,
+                  const unsigned char* __restrict__ scratch, float* __restrict__ state, float* __restrict__ core, int* __restrict__ error_word) {
+    extern __shared__ __align__(1024) unsigned char sm[];
+    const uint32_t base = smem_u32(sm);
+    if (base & 1023u) {            // the 128-byte swizzle needs 1024-byte aligned tiles
+        if (threadIdx.x == 0) atomicExch(error_word, 8);
+        return;
+    }
+    uint64_t* bars = reinterpret_cast<uint64_t*>(sm + kOffWBar);
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + W_BARS);
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+    auto bar = [&](int i) { return base + kOffWBar + 8u * i; };
+    const int h = blockIdx.x / sh.n_vt, tile = blockIdx.x % sh.n_vt, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const LaSeqMeta sq = seqs[blockIdx.y];
+    const int n_chunks = (sq.count + kDC - 1) / kDC;
+    if (n_chunks <= 0 || sq.slot < 0 || sq.slot >= max_seqs) return;
+    if (*reinterpret_cast<volatile int*>(error_word) != 0) return;   // an earlier CTA gave up: do not queue more bounded waits
+    float* Sg = state + (size_t)sq.slot * sh.state_floats() + (size_t)(h * sh.n_vt + tile) * sh.tile_floats();
+    const unsigned char* item0 = scratch + (first_chunk(sq.row0, blockIdx.y) * sh.heads + h) * it.bytes();
+    const size_t step = (size_t)sh.heads * it.bytes();
+
+    if (tid == 0) {
+        for (int i = 0; i < W_BARS; ++i) mbar_init(bar(i), (i == W_B2 || i == W_B3) ? 256 : 1);
+        *abort_flag = 0;
+        mbar_fence_init();
+    }
+    if (warp == 8) {
+        tmem_alloc(smem_u32(tmem_slot), 256);
+        tmem_relinquish();
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = *tmem_slot, tm_s = tmem, tm_x = tmem + 128, tm_o = tmem + 192;
+
+    if (warp == 8) {
+        // ------------------------------ copies + MMA issuer ------------------------------
+        if (lane == 0) {
+            constexpr uint32_t id64 = umma_idesc(kFmtF16, 128, 64, 0, 0);
+            constexpr uint32_t id_u = umma_idesc(kFmtF16, 128, 64 * ND, 0, 1);      // B MN-major
+            auto load_wq = [&](int c) {
+                mbar_arrive_expect_tx(bar(W_WQ), 2 * ND * kTile + ND * 256);
+                bulk_g2s(base + kOffWQ, item0 + c * step, 2 * ND * kTile, bar(W_WQ));
+                bulk_g2s(base + kOffWE, item0 + c * step + it.off_e(), ND * 256, bar(W_WQ));
+            };
+            auto load_km = [&](int c) {
+                mbar_arrive_expect_tx(bar(W_KM), (ND + 1) * kTile);
+                bulk_g2s(base + kOffWK, item0 + c * step + it.off_k(), (ND + 1) * kTile, bar(W_KM));
+            };
+            load_wq(0);
+            load_km(0);
+            for (int c = 0; c < n_chunks; ++c) {
+                const uint32_t par = c & 1;
+                if (!mbar_wait(bar(W_WQ), par, abort_flag)) break;
+                if (!mbar_wait(bar(W_B2), par, abort_flag)) break;
+                tc_fence_after();
+#pragma unroll
+                for (int ks = 0; ks < 4 * ND; ++ks) {          // X = S_0^T W^T,  O^T = S_0^T (e^G Q)^T
+                    const uint64_t a = umma_smem_desc(base + kOffWS + (ks >> 2) * 2 * kTile + (ks & 3) * 32, 16, 1024);
+                    const uint32_t off = (ks >> 2) * kTile + (ks & 3) * 32;
+                    umma_f16(tm_x, a, umma_smem_desc(base + kOffWQ + off, 16, 1024), id64, ks > 0 ? 1u : 0u);
+                    umma_f16(tm_o, a, umma_smem_desc(base + kOffWQ + ND * kTile + off, 16, 1024), id64, ks > 0 ? 1u : 0u);
+                }
+                umma_commit(bar(W_C2));
+                if (c + 1 < n_chunks) {
+                    if (!mbar_wait(bar(W_C2), par, abort_flag)) break;
+                    load_wq(c + 1);
+                }
+                if (!mbar_wait(bar(W_KM), par, abort_flag)) break;
+                if (!mbar_wait(bar(W_B3), par, abort_flag)) break;
+                tc_fence_after();
+#pragma unroll
+                for (int ks = 0; ks < 4; ++ks) {               // O^T += U^T M^T,  S^T += U^T (e^{G_C - G} K)
+                    const uint64_t a = umma_smem_desc(base + kOffWU + ks * 32, 16, 1024);
+                    umma_f16(tm_o, a, umma_smem_desc(base + kOffWK + ND * kTile + ks * 32, 16, 1024), id64, 1u);
+                    umma_f16(tm_s, a, umma_smem_desc(base + kOffWK + ks * 2048, kTile, 1024), id_u, 1u);
+                }
+                umma_commit(bar(W_C3));
+                if (c + 1 < n_chunks) {
+                    if (!mbar_wait(bar(W_C3), par, abort_flag)) break;
+                    load_km(c + 1);
+                }
+            }
+        }
+    } else {
+        // ------------------------------ compute warps ------------------------------
+        const int r = tid & 127, hf = tid >> 7;                // value of S^T, X and O^T; half of the columns
+        const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
+        const float* s_e = reinterpret_cast<const float*>(sm + kOffWE);
+        const int col = tile * kMlstmTile + r;
+        bool ok = true;
+#pragma unroll 1
+        for (int cc = 0; cc < ND; ++cc) {
+            const int ch = hf * ND + cc;
+            uint32_t sv[32];
+#pragma unroll
+            for (int e = 0; e < 32; ++e) {
+                const int d = ch * 32 + e;
+                sv[e] = (d < sh.dim && r < sh.vt) ? __float_as_uint(Sg[(size_t)d * sh.vt + r]) : 0u;
+            }
+            tmem_st32(tm_s + lane_base + ch * 32, sv);
+        }
+        tmem_wait_st();
+        auto store_out = [&](int c, bool do_store) {           // O^T of chunk c -> core[token][head][value]
+            uint32_t ov[32];
+            tmem_ld32(tm_o + lane_base + hf * 32, ov);
+            tmem_wait_ld();
+            if (!do_store || col >= sh.vp || r >= 64 * NV) return;
+            const int n_valid = sq.count - c * kDC - hf * 32;
+            float* dst = core + (size_t)(sq.row0 + c * kDC + hf * 32) * (sh.heads * sh.vp) + h * sh.vp + col;
+#pragma unroll
+            for (int j = 0; j < 32; ++j)
+                if (j < n_valid) dst[(size_t)j * sh.heads * sh.vp] = __uint_as_float(ov[j]);
+        };
+        for (int c = 0; c < n_chunks; ++c) {   // after a failed wait the warp keeps the barrier protocol going, without waiting or storing
+            const uint32_t par = c & 1;
+            uint4 u4[4];                       // U' of this thread's 32 tokens
+            if (r < 64 * NV) {
+                const unsigned char* u = item0 + c * step + it.off_u() + tile * NV * kTile;
+#pragma unroll
+                for (int q = 0; q < 4; ++q) u4[q] = __ldcs(reinterpret_cast<const uint4*>(u + sw(r, hf * 4 + q)));
+            } else {
+#pragma unroll
+                for (int q = 0; q < 4; ++q) u4[q] = make_uint4(0u, 0u, 0u, 0u);
+            }
+            if (c > 0) {                       // the previous chunk's last products: its outputs and the state are complete
+                if (!mbar_wait_warp(bar(W_C3), (c - 1) & 1, abort_flag)) ok = false;
+                tc_fence_after();
+            }
+            if (!mbar_wait_warp(bar(W_WQ), par, abort_flag)) ok = false;
+            // ---- S^T -> fp16 tile, and back decayed to the chunk's end ----
+#pragma unroll 1
+            for (int cc = 0; cc < ND; ++cc) {
+                const int ch = hf * ND + cc;
+                uint32_t sv[32];
+                tmem_ld32(tm_s + lane_base + ch * 32, sv);
+                tmem_wait_ld();
+                unsigned char* row = sm + kOffWS + (ch >> 1) * 2 * kTile;
+#pragma unroll
+                for (int q = 0; q < 4; ++q) {
+                    uint32_t pk[4];
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) pk[e] = pack_half2(__uint_as_float(sv[q * 8 + 2 * e]), __uint_as_float(sv[q * 8 + 2 * e + 1]));
+                    *reinterpret_cast<uint4*>(row + sw(r, (ch & 1) * 4 + q)) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+                }
+#pragma unroll
+                for (int e = 0; e < 32; e += 4) {
+                    const float4 f = *reinterpret_cast<const float4*>(s_e + ch * 32 + e);
+                    sv[e] = __float_as_uint(__uint_as_float(sv[e]) * f.x); sv[e + 1] = __float_as_uint(__uint_as_float(sv[e + 1]) * f.y);
+                    sv[e + 2] = __float_as_uint(__uint_as_float(sv[e + 2]) * f.z); sv[e + 3] = __float_as_uint(__uint_as_float(sv[e + 3]) * f.w);
+                }
+                tmem_st32(tm_s + lane_base + ch * 32, sv);
+            }
+            if (c > 0) store_out(c - 1, ok);   // ahead of the products that overwrite O^T
+            tmem_wait_st();
+            fence_proxy_async_smem();
+            tc_fence_before();
+            mbar_arrive(bar(W_B2));
+            // ---- U = U' - W S_0 ----
+            if (!mbar_wait_warp(bar(W_C2), par, abort_flag)) ok = false;
+            tc_fence_after();
+            {
+                uint32_t x[32];
+                tmem_ld32(tm_x + lane_base + hf * 32, x);
+                tmem_wait_ld();
+#pragma unroll
+                for (int q = 0; q < 4; ++q) {
+                    const uint32_t us[4] = {u4[q].x, u4[q].y, u4[q].z, u4[q].w};
+                    uint32_t pk[4];
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const float2 f = unpack_half2(us[e]);
+                        pk[e] = pack_half2(f.x - __uint_as_float(x[q * 8 + 2 * e]), f.y - __uint_as_float(x[q * 8 + 2 * e + 1]));
+                    }
+                    *reinterpret_cast<uint4*>(sm + kOffWU + sw(r, hf * 4 + q)) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+                }
+            }
+            fence_proxy_async_smem();
+            tc_fence_before();
+            mbar_arrive(bar(W_B3));
+        }
+        if (ok && mbar_wait_warp(bar(W_C3), (n_chunks - 1) & 1, abort_flag)) {
+            tc_fence_after();
+            store_out(n_chunks - 1, true);
+#pragma unroll 1
+            for (int cc = 0; cc < ND; ++cc) {
+                const int ch = hf * ND + cc;
+                uint32_t sv[32];
+                tmem_ld32(tm_s + lane_base + ch * 32, sv);
+                tmem_wait_ld();
+#pragma unroll
+                for (int e = 0; e < 32; ++e) {
+                    const int d = ch * 32 + e;
+                    if (d < sh.dim && r < sh.vt) Sg[(size_t)d * sh.vt + r] = __uint_as_float(sv[e]);
+                }
+            }
+            // ---- the convolutions' last inputs: a thread per channel, older tokens first ----
+            const int D4 = (sh.dim + 3) / 4 * 4, n = sh.taps - 1, kvh = h / (sh.heads / sh.kv_heads), pitch = sh.off_b();
+            float* hist = Sg + (size_t)sh.dim * sh.vt;
+            auto keep = [&](float* hs, int stride, int c) {
+                for (int j = 0; j < n; ++j) {
+                    const int t = sq.count - n + j;
+                    hs[(size_t)j * stride] = t >= 0 ? __bfloat162float(qkv[(size_t)(sq.row0 + t) * pitch + c]) : hs[(size_t)(n + t) * stride];
+                }
+            };
+            for (int d = tid; d < sh.dim; d += 256) {
+                keep(hist + d, D4, kvh * sh.dp + d);
+                keep(hist + n * D4 + d, D4, sh.off_k() + kvh * sh.dp + d);
+            }
+            for (int v = tid; v < sh.vt; v += 256)
+                if (tile * kMlstmTile + v < sh.vdim) keep(hist + 2 * n * D4 + v, sh.vt, sh.off_v() + h * sh.vp + tile * kMlstmTile + v);
+        }
+    }
+    tc_fence_before();
+    __syncthreads();
+    if (warp == 8) {
+        tc_fence_after();
+        tmem_dealloc(tmem, 256);
+    }
+    if (tid == 0 && *abort_flag) atomicExch(error_word, 10);
+}
+
+static DeltaItem delta_item(const DeltaShape& sh) { return DeltaItem{ceil_div(sh.dim, 64), sh.vt > 64 ? 2 : 1, sh.n_vt}; }
+
+bool delta_chunk_fits(const DeltaShape& sh) { return sh.dim <= 128; }
+
+size_t delta_chunk_bytes(const DeltaShape& sh) { return (size_t)sh.heads * delta_item(sh).bytes(); }
+
+int launch_delta_chunk(const DeltaShape& sh, const void* qkv, const float* a, const float* b, const float* conv, const float* a_log, const float* dt_bias,
+                       const LaSeqMeta* d_seqs, int n_seqs, int max_count, int max_seqs, float* state, void* scratch, float* core, int* d_error,
+                       cudaStream_t s) {
+    const DeltaItem it = delta_item(sh);
+    static PerDeviceOnce once;
+    B2_PER_DEVICE_ONCE(once,
+        for (auto k : {delta_prep_kernel<1, 4>, delta_prep_kernel<2, 4>, delta_prep_kernel<1, 0>, delta_prep_kernel<2, 0>})
+            B2_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, kPrepSmem));
+        for (auto k : {delta_walk_kernel<1, 1>, delta_walk_kernel<1, 2>, delta_walk_kernel<2, 1>, delta_walk_kernel<2, 2>})
+            B2_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, kWalkSmem)));
+    DeltaChunkArgs A{sh, it, (const __nv_bfloat16*)qkv, a, b, conv, a_log, dt_bias, state, d_seqs, max_seqs, (unsigned char*)scratch};
+    const dim3 gp(sh.heads, ceil_div(max_count, kDC), n_seqs);
+    auto prep = [&](auto kernel) { kernel<<<gp, 256, kPrepSmem, s>>>(A); };
+    if (it.nd == 2) { if (sh.taps == 4) prep(delta_prep_kernel<2, 4>); else prep(delta_prep_kernel<2, 0>); }
+    else { if (sh.taps == 4) prep(delta_prep_kernel<1, 4>); else prep(delta_prep_kernel<1, 0>); }
+    B2_LAUNCH_CHECK();
+    const dim3 gw(sh.heads * sh.n_vt, n_seqs);
+    auto walk = [&](auto kernel) {
+        kernel<<<gw, kWalkThreads, kWalkSmem, s>>>(sh, it, (const __nv_bfloat16*)qkv, d_seqs, max_seqs, (const unsigned char*)scratch, state, core, d_error);
+    };
+    if (it.nd == 2) { if (it.nv == 2) walk(delta_walk_kernel<2, 2>); else walk(delta_walk_kernel<2, 1>); }
+    else { if (it.nv == 2) walk(delta_walk_kernel<1, 2>); else walk(delta_walk_kernel<1, 1>); }
+    B2_LAUNCH_CHECK();
+    return 0;
+}
+
+}  // namespace b200
