@@ -241,16 +241,16 @@ def main():
     ap.add_argument("--cpu-prompt", type=int, default=24)
     ap.add_argument("--cpu-gen", type=int, default=8)
     ap.add_argument("--no-cpu-baseline", action="store_true")
-    ap.add_argument("--workload", default="hybrid", choices=["hybrid", "nuzopel"],
-                    help="nuzopel: prefill and decode of the mLSTM / latent-attention model at a few sizes, beside the hybrid stack (1 GPU)")
+    ap.add_argument("--workload", default="hybrid", choices=["hybrid", "nuzopel", "gutenex"],
+                    help="nuzopel, gutenex: prefill and decode of a layer-described model at a few sizes, beside the hybrid stack (1 GPU)")
     args = ap.parse_args()
 
     if args.impl == "reference":
         run_reference_arm(args)
         return
-    if args.workload == "nuzopel":
+    if args.workload != "hybrid":
         import model_bench
-        print(json.dumps(model_bench.run(read_peaks(), args.steps, ClockSampler(0))))
+        print(json.dumps(model_bench.run(read_peaks(), args.steps, ClockSampler(0), args.workload)))
         return
 
     import importlib

@@ -490,7 +490,8 @@ long long b200attn_launch_count(int reset);
  * also work for launches captured by b200attn_decode_graph_capture while profiling is on: every replay fills its
  * slots again, b200attn_profile_read sums and re-arms them.  Names: "fa_prefill", "fa_decode", "la_prefill",
  * "la_decode", "kv_append", and for the projections of the fused decode step "gemm_in" (input projections),
- * "gemm_ffn" (gate / up + SwiGLU), "gemm_res" (output projections with the residual add), "lm_head".  b200attn_profile_read synchronises the device and returns the summed device time and
+ * "gemm_ffn" (gate / up + SwiGLU), "gemm_res" (output projections with the residual add), "lm_head".  In layer-described stacks "la_*" are
+ * the matrix memories, "fa_*" the attention kernels, "delta_*" the channel-wise delta rule.  b200attn_profile_read synchronises the device and returns the summed device time and
  * launch count; b200attn_profile_reset forgets all pairs and slots (re-capture a graph that carried stamps).
  * ---------------------------------------------------------------------------------------------- */
 int b200attn_profile_enable(int on);

@@ -5,7 +5,7 @@ and prints its roofline line.  Sized by flags so the same command serves as a sm
     python kernel_bench.py --kernel fa_decode  --seqs 128 --ctx 1280 --kv fp16
     python kernel_bench.py --kernel fa_prefill --seqs 16  --ctx 1024
     python kernel_bench.py --kernel la_prefill --seqs 10  --ctx 1024
-    python kernel_bench.py --kernel mlstm_prefill  --seqs 16 --ctx 1024      # also mlstm_decode, latent_prefill, latent_decode
+    python kernel_bench.py --kernel mlstm_prefill  --seqs 16 --ctx 1024      # also latent_, lightning_, delta_, diff_ and _decode
 
 Inputs are synthetic (unit-RMS q/k, N(0, 0.6) v, decays as in the model) and stay larger than L2 for the
 decode kernels by rotating over `--layers` independent caches.
@@ -47,7 +47,7 @@ def time_ms(fn, iters, warmup):
 
 
 def measure_in_stack(kernel: str, seqs: int, ctx: int, iters: int, warmup: int) -> dict:
-    """mLSTM and latent-attention kernels inside a small stack (width 1024, 16 heads; one layer of each kind, layer sizes of
+    """Mixer kernels of layer-described models inside a small stack (width 1024, 16 heads; one layer of each kind, layer sizes of
     model_bench.py), timed by the library's own stamps and event pairs: prefill passes of all sequences, or eager decode steps
     behind a prompt of `ctx` tokens."""
     import importlib
@@ -55,12 +55,15 @@ def measure_in_stack(kernel: str, seqs: int, ctx: int, iters: int, warmup: int) 
     ops = entry.load_ops()
     models = importlib.import_module(entry.PKG_NAME + ".models")
     case = dict(width=1024, ff=1024, vocab=1024, layers=4, batch=seqs, prompt=ctx, gen=0)
-    cfg = model_bench.nuzopel_config(case)
-    cfg["layers"] = cfg["layers"][2:4]
+    kind, synth = ("nuzopel" if kernel.startswith(("mlstm", "latent")) else "gutenex"), entry.load_package().synth
+    cfg = getattr(model_bench, kind + "_config")(case)
+    cfg["layers"] = cfg["layers"][2 if kind == "nuzopel" else 1:4]
+    tensors = synth.nuzopel_tensors(cfg, 3) if kind == "nuzopel" else synth.gutenex_tensors(cfg, model_bench.GATE_RANKS, 3)
     prefill = kernel.endswith("prefill")
-    st = models.build_model(cfg, models.Limits(seqs, ctx + iters + warmup + 1, 0, seqs * ctx if prefill else 8192, "bfloat16"))
-    models.load_tensors(st, entry.load_package().synth.nuzopel_tensors(cfg, 3))
-    cls = ("la_" if kernel.startswith("mlstm") else "fa_") + ("prefill" if prefill else "decode")
+    st = models.build_model(cfg, models.Limits(seqs, ctx + iters + warmup + 1, 0, seqs * ctx if prefill else 8192, "bfloat16"),
+                            {k: v.shape for k, v in tensors.items()})
+    models.load_tensors(st, tensors)
+    cls = dict(mlstm="la", lightning="la", delta="delta", latent="fa", diff="fa")[kernel.split("_")[0]] + ("_prefill" if prefill else "_decode")
     toks = torch.randint(0, 1024, (seqs, ctx), dtype=torch.int32, device="cuda")
     with torch.cuda.stream(torch.cuda.Stream()):
         nxt = None if prefill else st.forward_batch_prefill(toks)
@@ -77,7 +80,7 @@ def measure_in_stack(kernel: str, seqs: int, ctx: int, iters: int, warmup: int) 
         ms, n = ops.profile_read(cls)
         ops.profile_enable(False); ops.profile_reset()
     assert st.device_status() == 0
-    bound, work = model_bench.kernel_work("nuzopel", case)[cls]
+    bound, work = model_bench.kernel_work(kind, case)[cls]
     hbm, tfl, src = peaks()
     scale = 1e9 if bound == "hbm" else 1e12
     out = dict(kernel=kernel, seqs=seqs, ctx=ctx, ms=ms / n, bound=bound, unit="GB/s" if bound == "hbm" else "TFLOP/s", peak=hbm if bound == "hbm" else tfl,
@@ -89,7 +92,7 @@ def measure_in_stack(kernel: str, seqs: int, ctx: int, iters: int, warmup: int) 
 def measure(kernel: str, seqs: int = 128, ctx: int = 1024, kv: str = "fp16", layers: int = 4, iters: int = 20, warmup: int = 3,
             serial: bool = False) -> dict:
     """Times `iters` back-to-back launches of one kernel class on the current device and returns its roofline record."""
-    if kernel.startswith(("mlstm", "latent")):
+    if kernel.split("_")[0] in ("mlstm", "latent", "lightning", "delta", "diff"):
         return measure_in_stack(kernel, seqs, ctx, iters, warmup)
     args = argparse.Namespace(kernel=kernel, seqs=seqs, ctx=ctx, kv=kv, layers=layers, iters=iters, warmup=warmup, serial=serial)
     ops = entry.load_ops()
@@ -171,7 +174,8 @@ def measure(kernel: str, seqs: int = 128, ctx: int = 1024, kv: str = "fp16", lay
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--kernel", required=True, choices=["la_decode", "fa_decode", "fa_prefill", "la_prefill", "mlstm_prefill", "mlstm_decode",
-                                                        "latent_prefill", "latent_decode"])
+                                                        "latent_prefill", "latent_decode", "lightning_prefill", "lightning_decode", "delta_prefill",
+                                                        "delta_decode", "diff_prefill", "diff_decode"])
     ap.add_argument("--seqs", type=int, default=128)
     ap.add_argument("--ctx", type=int, default=1024)
     ap.add_argument("--kv", default="fp16", choices=["fp16", "int8"])

@@ -1,4 +1,5 @@
-"""Prefill and decode throughput of layer-described models beside the hybrid stack at equal size (bench.py --workload nuzopel).
+"""Prefill and decode throughput of layer-described models beside the hybrid stack at equal size (bench.py --workload nuzopel
+or gutenex).
 
 Every case runs both stacks with the same width, feed-forward, vocabulary, number of layers, batch and lengths: random weights,
 random token ids, one prefill pass over the batch's prompts and captured decode steps behind it, timed with CUDA events after
@@ -41,6 +42,37 @@ def build_nuzopel(pkg, models, c):
     return st
 
 
+KEEP, GATE_RANKS = 64, (128, 128)
+
+
+def gutenex_config(c: dict) -> dict:
+    """Every fourth layer differential attention, the others channel-wise delta rule, lightning, channel-wise delta rule; every layer
+    with a feed-forward, no loop: as many layers, heads and cached values per token as the hybrid stack beside it."""
+    heads = c["width"] // 64
+    mlp = dict(kind="dense", ff=c["ff"])
+    layers = []
+    for i in range(c["layers"]):
+        if i % 4 == 3:
+            layers.append(dict(type="attention", mlp=mlp, mixer=dict(heads=heads, kv_heads=heads // 4, dim=64, vdim=128, scale=64 ** -0.5, diff=0.5,
+                                                                     mask=dict(size=WINDOW, keep_first=KEEP), rot=dict(base=1e4, dims=32))))
+        elif i % 4 == 1:
+            layers.append(dict(type="lightning", mlp=mlp, mixer=dict(heads=heads, dim=128, vdim=128, decay=[1.0 - 2.0 ** (-3 - h % 8) for h in range(heads)])))
+        else:
+            layers.append(dict(type="channel_delta", mlp=mlp, mixer=dict(heads=heads, kv_heads=heads, dim=128, vdim=128, conv=4)))
+    return dict(architecture="Gutenex", width=c["width"], vocab=c["vocab"], layers=layers, norm=dict(eps=1e-6), logit_softcap=30.0)
+
+
+def build_gutenex(pkg, models, c):
+    cfg = gutenex_config(c)
+    t = pkg.synth.gutenex_tensors(cfg, GATE_RANKS, 1234)
+    st = models.build_model(cfg, models.Limits(c["batch"], c["prompt"] + c["gen"], 0, c["batch"] * c["prompt"], "bfloat16"), {k: v.shape for k, v in t.items()})
+    models.load_tensors(st, t)
+    return st
+
+
+BUILDERS = dict(nuzopel=build_nuzopel, gutenex=build_gutenex)
+
+
 def build_hybrid(pkg, ops, c):
     st = ops.HybridStack(c["layers"], c["ff"], c["vocab"], c["batch"], c["prompt"] + c["gen"],
                          -(-c["batch"] * c["prompt"] // (c["prompt"] + c["gen"])), ops.KV_FP16, False)
@@ -68,6 +100,14 @@ def kernel_work(kind: str, c: dict) -> dict:
                     la_decode=("hbm", B * (2 * 16 * 128 * 128 * 4 + 2 * 3 * 6144 * 4 + 8224 * 4 + 2048 * 2)),
                     fa_decode=("hbm", B * (2048.0 * ctx + 8 * 256 * 6)))
     H = c["width"] // 64
+    if kind == "gutenex":
+        chunks = -(-P // 64)
+        return dict(la_prefill=("tensor", B * H * chunks * (2 * 2 * 64 * 64 * 128 + 2 * 2 * 64 * 128 * 128)),
+                    delta_prefill=("tensor", B * H * chunks * (5 * 2 * 64 * 64 * 128 + 3 * 2 * 64 * 128 * 128 + 64 ** 3 / 3)),
+                    fa_prefill=("tensor", B * H * 2 * 2 * (64 + 128) * window_pairs(P, WINDOW)),
+                    la_decode=("hbm", B * H * (2 * 128 * 128 * 4 + 3 * 128 * 4 + 128 * 4)),
+                    delta_decode=("hbm", B * H * (2 * (128 * 128 + 3 * 3 * 128) * 4 + (3 * 128 + 1) * 4 + 2 * 128 * 4 + 128 * 2)),
+                    fa_decode=("hbm", B * (min(WINDOW, ctx) * (H // 4) * 256 * 2 + (H // 4) * 16 * 128 * 2 + H * 128 * 2)))
     return dict(la_prefill=("tensor", B * H * -(-P // 64) * (2 * 2 * 64 * 64 * 128 + 2 * 2 * 64 * 128 * 128)),     # QK^T, PV, Q S, K^T V in chunks of 64
                 fa_prefill=("tensor", B * H * 2 * (192 + 128) * window_pairs(P, WINDOW)),
                 la_decode=("hbm", B * (2 * H * (128 * 128 + 128 + 1) * 4 + H * (4 * 128 + 2) * 4 + H * 128 * 2)),
@@ -101,13 +141,13 @@ def measure(torch, ops, st, kind: str, c: dict, peaks: dict, steps: int) -> dict
     ops.profile_reset(); ops.profile_enable(True)
     st.set_tokens(st.forward_batch_prefill(toks))
     s.synchronize()
-    t = {n: ops.profile_read(n) for n in ("la_prefill", "fa_prefill")}
+    t = {n: ops.profile_read(n) for n in ("la_prefill", "delta_prefill", "fa_prefill")}
     ops.profile_reset()
     st.capture_decode(B)
     ops.profile_enable(False)
     st.launch_decode(G // 2)
     s.synchronize()
-    acc = {n: [0.0, 0] for n in ("la_decode", "fa_decode")}
+    acc = {n: [0.0, 0] for n in ("la_decode", "delta_decode", "fa_decode")}
     for n in acc:
         ops.profile_read(n)
     for _ in range(8):
@@ -134,7 +174,7 @@ def measure(torch, ops, st, kind: str, c: dict, peaks: dict, steps: int) -> dict
     return dict(prefill_ms=mp, prefill_tok_s=B * P / mp * 1e3, decode_step_ms=md, decode_tok_s=B / md * 1e3, kernels=kernels)
 
 
-def run(peaks: dict, steps: int, clocks) -> dict:
+def run(peaks: dict, steps: int, clocks, model: str = "nuzopel") -> dict:
     import torch
     pkg = entry.load_package()
     ops = entry.load_ops()
@@ -145,11 +185,11 @@ def run(peaks: dict, steps: int, clocks) -> dict:
     with torch.cuda.stream(torch.cuda.Stream()):
         for c in CASES:
             row = dict(case=c)
-            for kind in (("nuzopel", "hybrid") if c["hybrid"] else ("nuzopel",)):
-                st = build_nuzopel(pkg, models, c) if kind == "nuzopel" else build_hybrid(pkg, ops, c)
+            for kind in ((model, "hybrid") if c["hybrid"] else (model,)):
+                st = build_hybrid(pkg, ops, c) if kind == "hybrid" else BUILDERS[kind](pkg, models, c)
                 row[kind] = measure(torch, ops, st, kind, c, peaks, steps)
                 del st
                 torch.cuda.synchronize()
             out.append(row)
-    return dict(workload="nuzopel", data="synthetic", dtype="bf16 (hybrid: fp16)", peaks=peaks, steps=steps, warmup=3, cases=out, clocks=clocks.stop(),
+    return dict(workload=model, data="synthetic", dtype="bf16 (hybrid: fp16)", peaks=peaks, steps=steps, warmup=3, cases=out, clocks=clocks.stop(),
                 l2="a pass's activations and a step's state and weights exceed L2, except the state and latents of the small batches")

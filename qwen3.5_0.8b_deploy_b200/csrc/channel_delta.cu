@@ -199,7 +199,7 @@ int launch_delta_step(ElemType t, const DeltaStepArgs& a, int n, cudaStream_t s)
     const DeltaShape& sh = a.sh;
     const size_t smem = (3 * (size_t)round_up(sh.dim, 4) + 17 * kMlstmTile + 32 + sh.hist_floats()) * 4;
     const dim3 grid(n, sh.heads, sh.n_vt);
-    unsigned long long* stamp = a.seqs ? nullptr : prof_stamp_slot(PROF_LA_DECODE);
+    unsigned long long* stamp = a.seqs ? nullptr : prof_stamp_slot(PROF_DELTA_DECODE);
     int rc = 0;
     dispatch_elem(t, [&](auto tag) {
         using T = decltype(tag);

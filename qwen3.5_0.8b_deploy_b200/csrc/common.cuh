@@ -68,7 +68,7 @@ inline void count_launch(int n = 1) { g_launches += n; }
 
 // ---- per-kernel event timing (gemm.cu) ------------------------------------------------------------------
 enum ProfKind { PROF_FA_PREFILL = 0, PROF_FA_DECODE, PROF_LA_PREFILL, PROF_LA_DECODE, PROF_KV_APPEND, PROF_GEMM_IN, PROF_GEMM_FFN, PROF_GEMM_RES,
-                PROF_LM_HEAD, PROF_COUNT };
+                PROF_LM_HEAD, PROF_DELTA_PREFILL, PROF_DELTA_DECODE, PROF_COUNT };
 extern bool g_prof_on;
 void prof_begin(ProfKind k, cudaStream_t s);
 void prof_end(ProfKind k, cudaStream_t s);

@@ -76,6 +76,41 @@ def hidden_states(seed: int, name: str, rows: int) -> np.ndarray:
     return normal(seed, name, (rows, HIDDEN), 1.0)
 
 
+def gutenex_tensors(config: dict, ranks: tuple, seed: int, std: float = 0.02) -> dict:
+    """Random weights of a Gutenex configuration under the names a model file has: matrices ~ N(0, std), norms 1, short
+    convolutions ~ N(0, 0.5), decay gates around e^-0.05 per token; `ranks` are the inner sizes of the decay and output gates."""
+    w, vocab = config["width"], config["vocab"]
+    out = {"embed": normal(seed, "embed", (vocab, w), std), "head": normal(seed, "head", (vocab, w), std), "final.norm": np.ones(w, np.float32)}
+    for i, layer in enumerate(config["layers"]):
+        m, p = layer["mixer"], f"l{i}."
+        heads, dim, vdim = m["heads"], m["dim"], m["vdim"]
+        shapes = {"o": (w, heads * vdim)}
+        if layer["type"] == "lightning":
+            shapes.update(q=(heads * dim, w), k=(heads * dim, w), v=(heads * vdim, w), g=(heads * vdim, w))
+            out[p + "mix.norm"] = np.ones(heads * vdim, np.float32)
+        elif layer["type"] == "channel_delta":
+            kv, a, g = m["kv_heads"], *ranks
+            shapes.update(q=(kv * dim, w), k=(kv * dim, w), v=(heads * vdim, w), b=(heads, w), a1=(a, w), a2=(heads * dim, a), g1=(g, w), g2=(heads * vdim, g))
+            for n in "qkv":
+                out[p + f"mix.{n}.conv"] = normal(seed, p + n + ".conv", (shapes[n][0], m["conv"]), 0.5)
+            out.update({p + "mix.A_log": np.zeros(heads, np.float32), p + "mix.dt_bias": np.full(heads * dim, -3.0, np.float32),
+                        p + "mix.norm": np.ones(vdim, np.float32)})
+        else:
+            kv = m["kv_heads"]
+            shapes.update(q=(heads * 2 * dim, w), k=(kv * 2 * dim, w), v=(kv * vdim, w))
+            out.update({p + f"mix.{n}.norm": np.ones(dim, np.float32) for n in "qk"})
+            out.update({p + "mix." + n: normal(seed, p + n, (dim,), 0.05) for n in ("lq1", "lk1", "lq2", "lk2")})
+        for n, shape in shapes.items():
+            out[p + "mix." + n] = normal(seed, p + "mix." + n, shape, std)
+        out[p + "norm1"] = np.ones(w, np.float32)
+        if layer["mlp"] is not None:
+            ff = layer["mlp"]["ff"]
+            out[p + "norm2"] = np.ones(w, np.float32)
+            for n, shape in (("gate", (ff, w)), ("up", (ff, w)), ("down", (w, ff))):
+                out[p + "mlp." + n] = normal(seed, p + "mlp." + n, shape, std)
+    return out
+
+
 def nuzopel_tensors(config: dict, seed: int, std: float = 0.02) -> dict:
     """Random weights of a Nuzopel configuration under the names a model file has: matrices ~ N(0, std), norms 1, gate biases
     0 (input) and 3 (forget)."""
