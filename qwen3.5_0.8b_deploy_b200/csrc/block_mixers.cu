@@ -97,6 +97,7 @@ int make_delta(const b200attn_layer_desc& d, const b200attn_model_config& c, Ele
     B2_TRY(op.w_gate.alloc((size_t)sh.gate_cols() * sh.low() * e));      // block diagonal: decay gates from the first inner columns, output gates from the others
     B2_TRY(op.w_out.alloc((size_t)c.width * sh.heads * sh.vp * e));
     B2_TRY(op.conv.alloc((size_t)sh.off_b() * sh.taps * 4));
+    if (sh.taps <= 4) B2_TRY(op.conv4.alloc((size_t)4 * sh.off_b() * 4));
     B2_TRY(op.a_log.alloc((size_t)sh.heads * 4));
     B2_TRY(op.dt_bias.alloc((size_t)sh.heads * sh.dp * 4));
     z.proj = std::max(z.proj, (size_t)sh.pitch());
@@ -124,6 +125,9 @@ int set_delta(DeltaOp& op, const std::string& n, const char* name, const Source&
         }
         if (n == std::string(p.n) + ".conv" && n != "b.conv") {
             B2_TRY(check_shape(t, name, (long long)p.heads * p.size, sh.taps));
+            for (int j = 0; j < sh.taps && sh.taps <= 4; ++j)
+                for (int h = 0; h < p.heads; ++h)
+                    B2_TRY(put(op.conv4, ELEM_F32, 1, (size_t)(4 - sh.taps + j) * sh.off_b() + p.row0 + (size_t)h * p.stride, 0, t, (size_t)h * p.size, j, p.size, 1));
             return put_heads(op.conv, ELEM_F32, p.row0, p.stride, t, p.heads, p.size, sh.taps, p.size, 0);
         }
     }
@@ -167,7 +171,7 @@ int delta_forward(BlockModel& m, DeltaOp& op, const LayerRun& run, const PassRow
         B2_TRY(gemm_typed(s, m.low.p, sh.low(), (const char*)op.w_gate.p + (size_t)acols * sh.low() * e, g, gcols, op.elem, op.elem, p.rows, gcols, sh.low()));
         {
             ProfScope prof(PROF_DELTA_PREFILL, s);
-            B2_TRY(launch_delta_chunk(sh, m.proj.p, a, b, op.conv.f(), op.a_log.f(), op.dt_bias.f(), p.d_seqs, p.n_seqs, p.max_count, m.cfg.max_seqs, state,
+            B2_TRY(launch_delta_chunk(sh, m.proj.p, a, b, sh.taps <= 4 ? op.conv4.f() : op.conv.f(), op.a_log.f(), op.dt_bias.f(), p.d_seqs, p.n_seqs, p.max_count, m.cfg.max_seqs, state,
                                       m.chunk.p, m.core.f(), m.error.i(), s));
         }
         return launch_delta_head_norm(op.elem, sh, m.core.f(), g, false, gcols, op.norm_w.f(), p.rows, m.mixed.p, s);

@@ -218,7 +218,7 @@ int launch_delta_head_norm(ElemType t, const DeltaShape& sh, const float* core, 
 // channel_delta_chunk.cu: prefill in chunks of 64 tokens.
 bool delta_chunk_fits(const DeltaShape& sh);
 size_t delta_chunk_bytes(const DeltaShape& sh);        // scratch per 64 rows of a pass (and one more such piece per sequence)
-// qkv: bf16 [rows][off_b]; a: fp32 [rows][heads * dp], b: fp32 [rows][heads], the gates' pre-activations.
+// qkv: bf16 [rows][off_b]; conv: conv4 with up to four taps; a: fp32 [rows][heads * dp], b: fp32 [rows][heads], the gates' pre-activations.
 int launch_delta_chunk(const DeltaShape& sh, const void* qkv, const float* a, const float* b, const float* conv, const float* a_log, const float* dt_bias,
                        const LaSeqMeta* d_seqs, int n_seqs, int max_count, int max_seqs, float* state, void* scratch, float* core, int* d_error,
                        cudaStream_t s);
@@ -228,7 +228,7 @@ struct DeltaOp {
     ElemType elem = ELEM_BF16;
     int width = 0;
     bool chunk = false;                // prefill through the chunked tensor-core kernels
-    DevBuf w_in, w_low, w_gate, w_out, conv, a_log, dt_bias, norm_w;
+    DevBuf w_in, w_low, w_gate, w_out, conv, conv4, a_log, dt_bias, norm_w;     // conv4: [4][off_b], up to four taps behind leading zeros
 };
 
 // ---- diff_attn.cu, diff_prefill.cu: differential attention ----------------------------------------------------------------------

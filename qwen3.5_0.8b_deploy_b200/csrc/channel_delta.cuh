@@ -6,10 +6,12 @@
 namespace b200 {
 
 __device__ __forceinline__ float delta_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
-// The same with the fast exponential and logarithm; a short series where 1 + x would lose x.
-__device__ __forceinline__ float delta_softplus_fast(float z) {
-    const float x = __expf(-fabsf(z));
-    return fmaxf(z, 0.f) + (x < 0.02f ? x * (1.f - x * (0.5f - x * (1.f / 3.f))) : __logf(1.f + x));
+// log2(1 + 2^y) on the special-function unit: softplus in units of ln 2.
+__device__ __forceinline__ float delta_softplus2(float y) {
+    float x;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(x) : "f"(fminf(y, 100.f)));
+    asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(x) : "f"(1.f + x));
+    return y > 24.f ? y : x;
 }
 
 }  // namespace b200

@@ -47,6 +47,10 @@ __device__ __forceinline__ float ex2c(float x) {
 }
 __device__ __forceinline__ uint32_t sw(int r, int p) { return (uint32_t)(r * 128 + ((p ^ (r & 7)) << 4)); }   // 16-byte piece p of row r
 __device__ __forceinline__ float2 unpack_half2(uint32_t v) { return __half22float2(*reinterpret_cast<const __half2*>(&v)); }
+__device__ __forceinline__ uint32_t mul_half2(uint32_t a, uint32_t b) {
+    const __half2 r = __hmul2(*reinterpret_cast<const __half2*>(&a), *reinterpret_cast<const __half2*>(&b));
+    return *reinterpret_cast<const uint32_t*>(&r);
+}
 __device__ __forceinline__ void ldm4(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
@@ -63,76 +67,101 @@ struct DeltaChunkArgs {
     const __nv_bfloat16* qkv;          // [rows][off_b]
     const float* a;                    // [rows][heads * dp] decay pre-activations
     const float* b;                    // [rows][heads]
-    const float *conv, *a_log, *dt_bias;
+    const float *conv, *a_log, *dt_bias;   // conv: [4][off_b] for up to four taps, [off_b][taps] for more
     const float* state;
     const LaSeqMeta* seqs;
     int max_seqs;
     unsigned char* scratch;
 };
 
-// Four consecutive tokens x eight channels behind a short convolution and silu; tokens before the pass come from hist
-// ([taps - 1][stride] floats, `hn` of the eight channels exist there), tokens from `count` on are zero.
-template <int TAPS>
-__device__ __forceinline__ void conv_piece(const __nv_bfloat16* raw, int pitch, const float* hist, int stride, int hn, const float* w, int taps, int t0,
-                                           int count, float (&o)[4][8]) {
-    auto row = [&](int t, float (&x)[8]) {
-        if (t >= count) {
-#pragma unroll
-            for (int e = 0; e < 8; ++e) x[e] = 0.f;
-        } else if (t >= 0) {
-            const uint4 v = *reinterpret_cast<const uint4*>(raw + (size_t)t * pitch);
-            const float2 a = unpack_bf16x2(v.x), b = unpack_bf16x2(v.y), c = unpack_bf16x2(v.z), d = unpack_bf16x2(v.w);
-            x[0] = a.x; x[1] = a.y; x[2] = b.x; x[3] = b.y; x[4] = c.x; x[5] = c.y; x[6] = d.x; x[7] = d.y;
+__device__ __forceinline__ void unpack8(uint4 v, float (&x)[8]) {
+    const float2 a = unpack_bf16x2(v.x), b = unpack_bf16x2(v.y), c = unpack_bf16x2(v.z), d = unpack_bf16x2(v.w);
+    x[0] = a.x; x[1] = a.y; x[2] = b.x; x[3] = b.y; x[4] = c.x; x[5] = c.y; x[6] = d.x; x[7] = d.y;
+}
+// Where a pass's inputs of a short convolution are: rows of bf16, and [taps - 1][stride] floats from before the pass.
+struct ConvSource {
+    const __nv_bfloat16* raw;          // the head's first channel in the pass's first row
+    const float* hist;
+    int pitch, stride, count, channels, padded;     // channels exist in hist, padded ones in raw
+};
+// Rows tok0 - 3 .. tok0 + 63 of up to 64 * blocks channels -> shared memory, 128 * blocks bytes per row; zeros outside the sequence.
+__device__ __forceinline__ void stage_raw(uint32_t dst, unsigned char* dst_ptr, const ConvSource& c, int blocks, int taps, int tok0, int tid) {
+    const int pieces = 8 * blocks;
+    for (int i = tid; i < 67 * pieces; i += 256) {
+        const int r = i / pieces, p = i % pieces, t = tok0 - 3 + r, ch = 8 * p;
+        const bool in = ch < c.padded;
+        if (t >= 0 || !in) {
+            const bool get = in && t < c.count;
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + i * 16), "l"(c.raw + (get ? (size_t)t * c.pitch + ch : 0)), "r"(get ? 16 : 0)
+                         : "memory");
         } else {
-            const float* h = hist + (size_t)(taps - 1 + t) * stride;
+            float x[8];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) x[e] = e < hn ? h[e] : 0.f;
+            for (int e = 0; e < 8; ++e) x[e] = (taps - 1 + t >= 0 && ch + e < c.channels) ? c.hist[(size_t)(taps - 1 + t) * c.stride + ch + e] : 0.f;
+            *reinterpret_cast<uint4*>(dst_ptr + i * 16) = make_uint4(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]), pack_bf16x2(x[4], x[5]), pack_bf16x2(x[6], x[7]));
         }
-    };
+    }
+}
+__device__ __forceinline__ void staged() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+
+// Four consecutive tokens x eight channels behind a short convolution and silu; tokens from `count` on are zero.
+// TAPS 4: from staged rows (the tokens are rows t .. t + 3 of the chunk), w4 [4][w_pitch] with leading zeros for fewer taps.
+// TAPS 0: any number of taps, from global memory, w [channel][taps].
+template <int TAPS>
+__device__ __forceinline__ void conv_piece(const unsigned char* tile, int row_bytes, const ConvSource& c, int ch, const float* w, int w_pitch, int taps, int tok0,
+                                           int t, float (&o)[4][8]) {
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
         for (int e = 0; e < 8; ++e) o[i][e] = 0.f;
     if constexpr (TAPS > 0) {
-        float wv[8 * TAPS];
+        float wv[TAPS][8];
 #pragma unroll
-        for (int i = 0; i < 2 * TAPS; ++i) {
-            const float4 v = *reinterpret_cast<const float4*>(w + 4 * i);
-            wv[4 * i] = v.x; wv[4 * i + 1] = v.y; wv[4 * i + 2] = v.z; wv[4 * i + 3] = v.w;
+        for (int j = 0; j < TAPS; ++j) {
+            const float4 a = load4(w + (size_t)j * w_pitch), b = load4(w + (size_t)j * w_pitch + 4);
+            wv[j][0] = a.x; wv[j][1] = a.y; wv[j][2] = a.z; wv[j][3] = a.w; wv[j][4] = b.x; wv[j][5] = b.y; wv[j][6] = b.z; wv[j][7] = b.w;
         }
 #pragma unroll
-        for (int r = 1 - TAPS; r < 4; ++r) {
+        for (int r = 0; r < TAPS + 3; ++r) {
             float x[8];
-            row(t0 + r, x);
+            unpack8(*reinterpret_cast<const uint4*>(tile + (t + r) * row_bytes + ch * 2), x);
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
-                const int j = r - i + TAPS - 1;
+                const int j = r - i;
                 if (j < 0 || j >= TAPS) continue;
 #pragma unroll
-                for (int e = 0; e < 8; ++e) o[i][e] += x[e] * wv[e * TAPS + j];
+                for (int e = 0; e < 8; ++e) o[i][e] += x[e] * wv[j][e];
             }
         }
     } else {
+#pragma unroll 1
         for (int j = 0; j < taps; ++j)
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
-                float x[8];
-                row(t0 + i + j - taps + 1, x);
+                const int at = tok0 + t + i + j - taps + 1;
+                float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+                if (at >= 0) {
+                    if (at < c.count) unpack8(*reinterpret_cast<const uint4*>(c.raw + (size_t)at * c.pitch + ch), x);
+                } else {
 #pragma unroll
-                for (int e = 0; e < 8; ++e) o[i][e] += x[e] * w[e * taps + j];
+                    for (int e = 0; e < 8; ++e)
+                        if (ch + e < c.channels) x[e] = c.hist[(size_t)(taps - 1 + at) * c.stride + ch + e];
+                }
+#pragma unroll
+                for (int e = 0; e < 8; ++e) o[i][e] += x[e] * w[(size_t)e * taps + j];
             }
     }
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int e = 0; e < 8; ++e) o[i][e] = t0 + i < count ? __fdividef(o[i][e], 1.0f + __expf(-o[i][e])) : 0.f;
+        for (int e = 0; e < 8; ++e) o[i][e] = tok0 + t + i < c.count ? __fdividef(o[i][e], 1.0f + __expf(-o[i][e])) : 0.f;
 }
 
 // Shared memory of the first kernel; rows of K-major tiles are 64 ND + 8 halves apart (an odd number of 16-byte units).
 constexpr uint32_t kRegion = 17408;                    // 64 rows of 136 halves
-constexpr uint32_t kOffKA = 0;                         // decayed keys (rows), e^G K, then the image of U'
-constexpr uint32_t kOffQA = kRegion;                   // decayed queries (rows), then V
-constexpr uint32_t kOffKB = 2 * kRegion;               // keys decayed to the end of their group, then the image of W
+constexpr uint32_t kOffKA = 0;                         // staged q, decayed keys (rows), e^G K, then the image of U'
+constexpr uint32_t kOffQA = kRegion;                   // staged k, decayed queries (rows), staged v, then the image of W
+constexpr uint32_t kOffKB = 2 * kRegion;               // keys decayed to the end of their group, then V
 constexpr uint32_t kOffCOL = 3 * kRegion;              // 96 rows of decayed keys (columns), then T
 constexpr uint32_t kOffAM = kOffCOL + 26112;           // A, fp32 [64][kLd]
 constexpr uint32_t kOffM = kOffAM + 17408;             // image of M
@@ -160,6 +189,15 @@ delta_prep_kernel(const DeltaChunkArgs A) {
     const int tok0 = chunk * kDC, left = sq.count - tok0, D4 = (sh.dim + 3) / 4 * 4, taps = sh.taps;
     const float* st = A.state + (size_t)sq.slot * sh.state_floats() + (size_t)h * sh.n_vt * sh.tile_floats();
 
+    const int kvh = h / (sh.heads / sh.kv_heads);
+    const __nv_bfloat16* rows = A.qkv + (size_t)sq.row0 * sh.off_b();
+    const float* hist = st + (size_t)sh.dim * sh.vt;
+    const ConvSource cq{rows + kvh * sh.dp, hist, sh.off_b(), D4, sq.count, sh.dim, sh.dp};
+    const ConvSource ck{rows + sh.off_k() + kvh * sh.dp, hist + (taps - 1) * D4, sh.off_b(), D4, sq.count, sh.dim, sh.dp};
+    if constexpr (TAPS > 0) {
+        stage_raw(base + kOffKA, sm + kOffKA, cq, ND, taps, tok0, tid);
+        stage_raw(base + kOffQA, sm + kOffQA, ck, ND, taps, tok0, tid);
+    }
     for (int i = tid; i < 64 * kLd / 4; i += 256) reinterpret_cast<float4*>(AM)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int i = tid; i < (int)kTile / 16; i += 256) reinterpret_cast<uint4*>(sm + kOffM)[i] = make_uint4(0u, 0u, 0u, 0u);
     if (tid < 64) s_beta[tid] = tid < left ? 1.0f / (1.0f + __expf(-A.b[(size_t)(sq.row0 + tok0 + tid) * sh.heads + h])) : 0.f;
@@ -175,18 +213,25 @@ delta_prep_kernel(const DeltaChunkArgs A) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) g[i][e] = 1.f;
     }
+    if constexpr (TAPS > 0) {
+        staged();
+        __syncthreads();
+    }
     if (act) {
         const bool in = ch < sh.dp;
-        const int kvh = h / (sh.heads / sh.kv_heads), hn = min(8, sh.dim - ch);
-        const float* hist = st + (size_t)sh.dim * sh.vt;
+        float4 z0[4], z1[4];                                        // decay pre-activations: requested ahead of the convolutions
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float* z = A.a + (size_t)(sq.row0 + tok0 + min(t0 + i, left - 1)) * (sh.heads * sh.dp) + h * sh.dp + (in ? ch : 0);
+            z0[i] = load4(z);
+            z1[i] = load4(z + 4);
+        }
 #pragma unroll
         for (int n = 0; n < 2; ++n) {
-            const int col = n * sh.off_k() + kvh * sh.dp + ch;
+            const int col = n * sh.off_k() + kvh * sh.dp + (in ? ch : 0);
             float o[4][8];
-            if (in) {
-                conv_piece<TAPS>(A.qkv + (size_t)sq.row0 * sh.off_b() + col, sh.off_b(), hist + n * (taps - 1) * D4 + ch, D4, hn, A.conv + (size_t)col * taps,
-                                 taps, tok0 + t0, sq.count, o);
-            } else {
+            conv_piece<TAPS>(sm + (n ? kOffQA : kOffKA), 16 * LN, n ? ck : cq, in ? ch : 0, A.conv + (size_t)col * (TAPS > 0 ? 1 : taps), sh.off_b(), taps, tok0, t0, o);
+            if (!in) {
 #pragma unroll
                 for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -199,26 +244,24 @@ delta_prep_kernel(const DeltaChunkArgs A) {
                 for (int e = 0; e < 8; ++e) ss += o[i][e] * o[i][e];
 #pragma unroll
                 for (int x = LN / 2; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
-                const float inv = (n ? 1.0f : 1.0f / sqrtf((float)sh.dim)) / sqrtf(ss + 1e-6f);
+                const float inv = (n ? 1.0f : rsqrtf((float)sh.dim)) * rsqrtf(ss + 1e-6f);
 #pragma unroll
                 for (int e = 0; e < 4; ++e) (n ? kh : qh)[i][e] = pack_half2(o[i][2 * e] * inv, o[i][2 * e + 1] * inv);
             }
         }
         float sum[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
         if (in) {
-            const float ea = -expf(A.a_log[h]) * kDL2e;
+            const float ea = -expf(A.a_log[h]);
             float dt[8];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) dt[e] = A.dt_bias[h * sh.dp + ch + e];
+            for (int e = 0; e < 8; ++e) dt[e] = A.dt_bias[h * sh.dp + ch + e] * kDL2e;
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 if (t0 + i >= left) continue;
-                const float* z = A.a + (size_t)(sq.row0 + tok0 + t0 + i) * (sh.heads * sh.dp) + h * sh.dp + ch;
-                const float4 z0 = load4(z), z1 = load4(z + 4);
-                const float zz[8] = {z0.x, z0.y, z0.z, z0.w, z1.x, z1.y, z1.z, z1.w};
+                const float zz[8] = {z0[i].x, z0[i].y, z0[i].z, z0[i].w, z1[i].x, z1[i].y, z1[i].z, z1[i].w};
 #pragma unroll
                 for (int e = 0; e < 8; ++e) {
-                    const float l = ea * delta_softplus_fast(zz[e] + dt[e]);
+                    const float l = ea * delta_softplus2(fmaf(zz[e], kDL2e, dt[e]));
                     sum[e] += l;
                     g[i][e] = ex2c(l);
                 }
@@ -287,28 +330,32 @@ delta_prep_kernel(const DeltaChunkArgs A) {
     const float* r0 = s_g + tg * DK + ch;                           // up to this group's start / end, up to the chunk's end
     const float *r1 = r0 + DK, *rC = s_g + 16 * DK + ch;
     auto piece = [&](uint32_t off, int row) { return reinterpret_cast<uint4*>(sm + off + row * kP * 2 + ch * 2); };
-    auto scaled = [](uint4 v, const float (&f)[8]) {
-        const float2 a = unpack_half2(v.x), b = unpack_half2(v.y), c = unpack_half2(v.z), d = unpack_half2(v.w);
-        return make_uint4(pack_half2(a.x * f[0], a.y * f[1]), pack_half2(b.x * f[2], b.y * f[3]), pack_half2(c.x * f[4], c.y * f[5]),
-                          pack_half2(d.x * f[6], d.y * f[7]));
+    auto scaled = [](uint4 v, const uint32_t (&f)[4]) {
+        return make_uint4(mul_half2(v.x, f[0]), mul_half2(v.y, f[1]), mul_half2(v.z, f[2]), mul_half2(v.w, f[3]));
     };
-    auto factors = [](float (&f)[8], const float* to, const float* from) {     // 2^(to - from)
+    auto packed = [](const float (&x)[8], uint32_t (&f)[4]) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) f[e] = pack_half2(x[2 * e], x[2 * e + 1]);
+    };
+    auto factors = [](uint32_t (&f)[4], const float* to, const float* from) {     // 2^(to - from)
         const float4 a = load4(to), b = load4(to + 4), c = load4(from), d = load4(from + 4);
-        f[0] = ex2c(a.x - c.x); f[1] = ex2c(a.y - c.y); f[2] = ex2c(a.z - c.z); f[3] = ex2c(a.w - c.w);
-        f[4] = ex2c(b.x - d.x); f[5] = ex2c(b.y - d.y); f[6] = ex2c(b.z - d.z); f[7] = ex2c(b.w - d.w);
+        f[0] = pack_half2(ex2c(a.x - c.x), ex2c(a.y - c.y)); f[1] = pack_half2(ex2c(a.z - c.z), ex2c(a.w - c.w));
+        f[2] = pack_half2(ex2c(b.x - d.x), ex2c(b.y - d.y)); f[3] = pack_half2(ex2c(b.z - d.z), ex2c(b.w - d.w));
     };
     const int blk = tg >> 2, own = tg & 3;
     if (act) {
         unsigned char* img = item + (c8 >> 3) * kTile;
         {
-            float f[8], x[8];
+            float run[8];
+            uint32_t f[4], x[4];
             factors(x, r0, s_g + ch);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) f[e] = 1.f;
+            for (int e = 0; e < 8; ++e) run[e] = 1.f;
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
 #pragma unroll
-                for (int e = 0; e < 8; ++e) f[e] *= g[i][e];
+                for (int e = 0; e < 8; ++e) run[e] *= g[i][e];
+                packed(run, f);
                 const uint4 q = scaled(make_uint4(qh[i][0], qh[i][1], qh[i][2], qh[i][3]), f);
                 *piece(kOffQA, t0 + i) = q;
                 *piece(kOffKA, t0 + i) = scaled(make_uint4(kh[i][0], kh[i][1], kh[i][2], kh[i][3]), f);
@@ -316,23 +363,25 @@ delta_prep_kernel(const DeltaChunkArgs A) {
             }
         }
         {
-            float f[8], x[8];
+            float run[8];
+            uint32_t f[4], x[4];
             factors(x, rC, r1);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) f[e] = 1.f;
+            for (int e = 0; e < 8; ++e) run[e] = 1.f;
 #pragma unroll
             for (int i = 3; i >= 0; --i) {
+                packed(run, f);
                 const uint4 k = scaled(make_uint4(kh[i][0], kh[i][1], kh[i][2], kh[i][3]), f);
                 *piece(kOffKB, t0 + i) = k;
                 *reinterpret_cast<uint4*>(img + A.item.off_k() + sw(t0 + i, c8 & 7)) = scaled(k, x);
 #pragma unroll
-                for (int e = 0; e < 8; ++e) f[e] *= g[i][e];
+                for (int e = 0; e < 8; ++e) run[e] *= g[i][e];
             }
         }
         // copies for the later groups of the block: 24 rows per block, 4 + 8 + 12
 #pragma unroll 1
         for (int i = own + 1; i < 4; ++i) {
-            float f[8];
+            uint32_t f[4];
             factors(f, s_g + (4 * blk + i) * DK + ch, r1);
             const int row = 24 * blk + (i == 1 ? 0 : i == 2 ? 4 : 12) + 4 * own;
 #pragma unroll
@@ -373,7 +422,7 @@ delta_prep_kernel(const DeltaChunkArgs A) {
     __syncthreads();
     if (act) {
         // ---- rows decay on from the start of their block, columns up to the start of a later one: 16 + 32 + 48 rows ----
-        float f[8];
+        uint32_t f[4];
         factors(f, r0, s_g + 4 * blk * DK + ch);
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
@@ -406,11 +455,35 @@ delta_prep_kernel(const DeltaChunkArgs A) {
         put2(q, 16 * I + g4 + 8, 8 * n + 2 * t4, d[2], d[3]);
     }
     __syncthreads();
+    const int nv = A.item.nv, vln = 8 * nv, kVP = 64 * nv + 8;      // lanes per token, row pitch of V
+    auto values = [&](int tile) {
+        const float* hv = hist + tile * sh.tile_floats() + 2 * (taps - 1) * D4;
+        return ConvSource{rows + sh.off_v() + h * sh.vp + tile * kMlstmTile, hv, sh.off_b(), sh.vt, sq.count, sh.vdim - tile * kMlstmTile, sh.vp - tile * kMlstmTile};
+    };
+    auto load_values = [&](int tile) {                              // behind the staging of the same tile
+        const int vtg = tid / vln, vc = 8 * (tid % vln), t = 4 * vtg;
+        const ConvSource c = values(tile);
+        if constexpr (TAPS > 0) {
+            staged();
+            __syncthreads();
+        }
+        if (vtg >= 16) return;
+        const bool in = vc < c.padded;
+        const int col = sh.off_v() + h * sh.vp + tile * kMlstmTile + (in ? vc : 0);
+        float o[4][8];
+        conv_piece<TAPS>(sm + kOffQA, 128 * nv, c, in ? vc : 0, A.conv + (size_t)col * (TAPS > 0 ? 1 : taps), sh.off_b(), taps, tok0, t, o);
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+            *reinterpret_cast<uint4*>(sm + kOffKB + ((t + i) * kVP + vc) * 2) =
+                in ? make_uint4(pack_half2(o[i][0], o[i][1]), pack_half2(o[i][2], o[i][3]), pack_half2(o[i][4], o[i][5]), pack_half2(o[i][6], o[i][7]))
+                   : make_uint4(0u, 0u, 0u, 0u);
+    };
+    if constexpr (TAPS > 0) stage_raw(base + kOffQA, sm + kOffQA, values(0), nv, taps, tok0, tid);
     // ---- T = (I + A)^-1 over the column copies; meanwhile M goes out and the keys decay from the chunk's start ----
     if (tid < 64) invert_diagonal(AM, TF, tid);
     for (int i = tid; i < (int)kTile / 16; i += 256) reinterpret_cast<uint4*>(item + A.item.off_m())[i] = reinterpret_cast<uint4*>(sm + kOffM)[i];
     if (act) {
-        float f[8];
+        uint32_t f[4];
         factors(f, s_g + 4 * blk * DK + ch, s_g + ch);
 #pragma unroll
         for (int i = 0; i < 4; ++i) *piece(kOffKA, t0 + i) = scaled(*piece(kOffKA, t0 + i), f);
@@ -419,82 +492,65 @@ delta_prep_kernel(const DeltaChunkArgs A) {
     if (warp < 6) scale_blocks(AM, TF, warp, lane);
     __syncthreads();
     solve_columns(AM, TF, warp, lane);
-    // ---- the values of a state tile: behind their convolution, over the queries ----
-    const int nv = A.item.nv, vln = 8 * nv, kVP = 64 * nv + 8;      // lanes per token, row pitch
-    auto load_values = [&](int tile) {
-        const int vtg = tid / vln, vc = 8 * (tid % vln), c = tile * kMlstmTile + vc, t = 4 * vtg;
-        if (vtg >= 16) return;
-        float o[4][8];
-        if (c < sh.vp) {
-            const int col = sh.off_v() + h * sh.vp + c;
-            const float* hv = st + tile * sh.tile_floats() + (size_t)sh.dim * sh.vt + 2 * (taps - 1) * D4;
-            conv_piece<TAPS>(A.qkv + (size_t)sq.row0 * sh.off_b() + col, sh.off_b(), hv + vc, sh.vt, min(8, sh.vdim - c), A.conv + (size_t)col * taps, taps,
-                             tok0 + t, sq.count, o);
-        } else {
-#pragma unroll
-            for (int i = 0; i < 4; ++i)
-#pragma unroll
-                for (int e = 0; e < 8; ++e) o[i][e] = 0.f;
-        }
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-            *reinterpret_cast<uint4*>(sm + kOffQA + ((t + i) * kVP + vc) * 2) =
-                make_uint4(pack_half2(o[i][0], o[i][1]), pack_half2(o[i][2], o[i][3]), pack_half2(o[i][4], o[i][5]), pack_half2(o[i][6], o[i][7]));
-    };
+    // ---- the values of a state tile: staged over the queries (requested ahead of the inverse), behind their convolution over KB ----
     load_values(0);
     __syncthreads();
-    // (T diag(beta)) entries (t, s), (t, s + 1) as fp16 hi and lo
-    auto t_pair = [&](int t, int s, uint32_t& hi, uint32_t& lo) {
-        const float2 v = *reinterpret_cast<const float2*>(TF + t * kLd + s), b = *reinterpret_cast<const float2*>(s_beta + s);
-        const float x = v.x * b.x, y = v.y * b.y;
-        hi = pack_half2(x, y);
-        const float2 hf = unpack_half2(hi);
-        lo = pack_half2(x - hf.x, y - hf.y);
-    };
+    {   // T diag(beta) as a swizzled fp16 tile over A, a quarter of a row per thread; blocks above the diagonal are never read
+        const int i = tid >> 2, qd = tid & 3;
+        if (qd <= i >> 4) {
+#pragma unroll
+            for (int p = 0; p < 2; ++p) {
+                const int s = 16 * qd + 8 * p;
+                const float4 a = load4(TF + i * kLd + s), b = load4(TF + i * kLd + s + 4), c = load4(s_beta + s), d = load4(s_beta + s + 4);
+                *reinterpret_cast<uint4*>(sm + kOffAM + sw(i, 2 * qd + p)) = make_uint4(pack_half2(a.x * c.x, a.y * c.y), pack_half2(a.z * c.z, a.w * c.w),
+                                                                                       pack_half2(b.x * d.x, b.y * d.y), pack_half2(b.z * d.z, b.w * d.w));
+            }
+        }
+    }
+    __syncthreads();
     {   // ---- W = (T diag(beta)) (e^G K): 16 rows x 32 ND columns per warp ----
         const int i = warp >> 1, c0 = (warp & 1) * 32 * ND;
         float d[4 * ND][4];
 #pragma unroll
         for (int n = 0; n < 4 * ND; ++n) d[n][0] = d[n][1] = d[n][2] = d[n][3] = 0.f;
         for (int k = 0; k <= i; ++k) {
-            uint32_t hi[4], lo[4];
-            t_pair(16 * i + g4, 16 * k + 2 * t4, hi[0], lo[0]);
-            t_pair(16 * i + g4 + 8, 16 * k + 2 * t4, hi[1], lo[1]);
-            t_pair(16 * i + g4, 16 * k + 2 * t4 + 8, hi[2], lo[2]);
-            t_pair(16 * i + g4 + 8, 16 * k + 2 * t4 + 8, hi[3], lo[3]);
+            uint32_t a[4];
+            ldm4(a, base + kOffAM + sw(16 * i + (lane & 15), 2 * k + (lane >> 4)));
             const uint32_t ka = base + kOffKA + ((16 * k + (lane & 15)) * kP + c0 + (lane >> 4) * 8) * 2;
 #pragma unroll
             for (int n = 0; n < 4 * ND; n += 2) {
                 uint32_t b[4];
                 ldm4t(b, ka + n * 16);
-                mma_16816(d[n], hi[0], hi[1], hi[2], hi[3], b[0], b[1]);
-                mma_16816(d[n], lo[0], lo[1], lo[2], lo[3], b[0], b[1]);
-                mma_16816(d[n + 1], hi[0], hi[1], hi[2], hi[3], b[2], b[3]);
-                mma_16816(d[n + 1], lo[0], lo[1], lo[2], lo[3], b[2], b[3]);
+                mma_16816(d[n], a[0], a[1], a[2], a[3], b[0], b[1]);
+                mma_16816(d[n + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
             }
         }
 #pragma unroll
         for (int n = 0; n < 4 * ND; ++n) {
             const int c = c0 + 8 * n;
-            unsigned char* w = sm + kOffKB + (c >> 6) * kTile;
+            unsigned char* w = sm + kOffQA + (c >> 6) * kTile;
             *reinterpret_cast<uint32_t*>(w + sw(16 * i + g4, (c >> 3) & 7) + 4 * t4) = pack_half2(d[n][0], d[n][1]);
             *reinterpret_cast<uint32_t*>(w + sw(16 * i + g4 + 8, (c >> 3) & 7) + 4 * t4) = pack_half2(d[n][2], d[n][3]);
         }
     }
     __syncthreads();
-    for (int i = tid; i < (int)(ND * kTile) / 16; i += 256) reinterpret_cast<uint4*>(item)[i] = reinterpret_cast<uint4*>(sm + kOffKB)[i];
+    for (int i = tid; i < (int)(ND * kTile) / 16; i += 256) reinterpret_cast<uint4*>(item)[i] = reinterpret_cast<uint4*>(sm + kOffQA)[i];
     // ---- U'^T = V^T (T diag(beta))^T of every state tile: 16 values x 64 (or 32) tokens per warp ----
     for (int tile = 0;; ++tile) {
-        const int mt = warp % (4 * nv), n0 = nv == 2 ? 0 : (warp >> 2) * 4, n1 = nv == 2 ? 8 : n0 + 4;
-        for (int n = n0; n < n1; ++n) {
+        const int mt = warp % (4 * nv), part = nv == 2 ? 0 : warp >> 2, parts = nv == 2 ? 1 : 2;      // token tiles part, part + parts, ..
+        uint32_t a[4][4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+            ldm4t(a[k], base + kOffKB + ((16 * k + (lane & 7) + ((lane >> 4) & 1) * 8) * kVP + 16 * mt + ((lane >> 3) & 1) * 8) * 2);
+#pragma unroll
+        for (int n = 0; n < 8; ++n) {
+            if (n % parts != part) continue;
             float d[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
             for (int k = 0; k <= n >> 1; ++k) {
-                uint32_t a[4], h0, l0, h1, l1;
-                ldm4t(a, base + kOffQA + ((16 * k + (lane & 7) + ((lane >> 4) & 1) * 8) * kVP + 16 * mt + ((lane >> 3) & 1) * 8) * 2);
-                t_pair(8 * n + g4, 16 * k + 2 * t4, h0, l0);
-                t_pair(8 * n + g4, 16 * k + 2 * t4 + 8, h1, l1);
-                mma_16816(d, a[0], a[1], a[2], a[3], h0, h1);
-                mma_16816(d, a[0], a[1], a[2], a[3], l0, l1);
+                uint32_t b0, b1;
+                ldm2(b0, b1, base + kOffAM + sw(8 * n + (lane & 7), 2 * k + ((lane >> 3) & 1)));
+                mma_16816(d, a[k][0], a[k][1], a[k][2], a[k][3], b0, b1);
             }
             *reinterpret_cast<uint32_t*>(sm + kOffKA + sw(16 * mt + g4, n) + 4 * t4) = pack_half2(d[0], d[1]);
             *reinterpret_cast<uint32_t*>(sm + kOffKA + sw(16 * mt + g4 + 8, n) + 4 * t4) = pack_half2(d[2], d[3]);
@@ -503,6 +559,7 @@ delta_prep_kernel(const DeltaChunkArgs A) {
         uint4* dst = reinterpret_cast<uint4*>(item + A.item.off_u() + tile * nv * kTile);
         for (int i = tid; i < (int)(nv * kTile) / 16; i += 256) dst[i] = reinterpret_cast<uint4*>(sm + kOffKA)[i];
         if (tile + 1 == sh.n_vt) break;
+        if constexpr (TAPS > 0) stage_raw(base + kOffQA, sm + kOffQA, values(tile + 1), nv, taps, tok0, tid);
         load_values(tile + 1);
         __syncthreads();
     }
@@ -765,8 +822,8 @@ int launch_delta_chunk(const DeltaShape& sh, const void* qkv, const float* a, co
     DeltaChunkArgs A{sh, it, (const __nv_bfloat16*)qkv, a, b, conv, a_log, dt_bias, state, d_seqs, max_seqs, (unsigned char*)scratch};
     const dim3 gp(sh.heads, ceil_div(max_count, kDC), n_seqs);
     auto prep = [&](auto kernel) { kernel<<<gp, 256, kPrepSmem, s>>>(A); };
-    if (it.nd == 2) { if (sh.taps == 4) prep(delta_prep_kernel<2, 4>); else prep(delta_prep_kernel<2, 0>); }
-    else { if (sh.taps == 4) prep(delta_prep_kernel<1, 4>); else prep(delta_prep_kernel<1, 0>); }
+    if (it.nd == 2) { if (sh.taps <= 4) prep(delta_prep_kernel<2, 4>); else prep(delta_prep_kernel<2, 0>); }
+    else { if (sh.taps <= 4) prep(delta_prep_kernel<1, 4>); else prep(delta_prep_kernel<1, 0>); }
     B2_LAUNCH_CHECK();
     const dim3 gw(sh.heads * sh.n_vt, n_seqs);
     auto walk = [&](auto kernel) {
