@@ -74,9 +74,9 @@ struct DeltaChunkArgs {
     unsigned char* scratch;
 };
 
-__device__ __forceinline__ void unpack8(uint4 v, float (&x)[8]) {
-    const float2 a = unpack_bf16x2(v.x), b = unpack_bf16x2(v.y), c = unpack_bf16x2(v.z), d = unpack_bf16x2(v.w);
-    x[0] = a.x; x[1] = a.y; x[2] = b.x; x[3] = b.y; x[4] = c.x; x[5] = c.y; x[6] = d.x; x[7] = d.y;
+__device__ __forceinline__ float4 unpack4(uint2 v) {
+    const float2 a = unpack_bf16x2(v.x), b = unpack_bf16x2(v.y);
+    return make_float4(a.x, a.y, b.x, b.y);
 }
 // Where a pass's inputs of a short convolution are: rows of bf16, and [taps - 1][stride] floats from before the pass.
 struct ConvSource {
@@ -84,11 +84,10 @@ struct ConvSource {
     const float* hist;
     int pitch, stride, count, channels, padded;     // channels exist in hist, padded ones in raw
 };
-// Rows tok0 - 3 .. tok0 + 63 of up to 64 * blocks channels -> shared memory, 128 * blocks bytes per row; zeros outside the sequence.
-__device__ __forceinline__ void stage_raw(uint32_t dst, unsigned char* dst_ptr, const ConvSource& c, int blocks, int taps, int tok0, int tid) {
-    const int pieces = 8 * blocks;
-    for (int i = tid; i < 67 * pieces; i += 256) {
-        const int r = i / pieces, p = i % pieces, t = tok0 - 3 + r, ch = 8 * p;
+// Rows tok0 - 3 .. tok0 + 63 of 8 << shift channels -> shared memory, 16 << shift bytes per row, by n threads; zeros outside the sequence.
+__device__ __forceinline__ void stage_raw(uint32_t dst, unsigned char* dst_ptr, const ConvSource& c, int shift, int taps, int tok0, int tid, int n) {
+    for (int i = tid; i < 67 << shift; i += n) {
+        const int t = tok0 - 3 + (i >> shift), ch = 8 * (i & ((1 << shift) - 1));
         const bool in = ch < c.padded;
         if (t >= 0 || !in) {
             const bool get = in && t < c.count;
@@ -104,78 +103,79 @@ __device__ __forceinline__ void stage_raw(uint32_t dst, unsigned char* dst_ptr, 
 }
 __device__ __forceinline__ void staged() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
-// Four consecutive tokens x eight channels behind a short convolution and silu; tokens from `count` on are zero.
-// TAPS 4: from staged rows (the tokens are rows t .. t + 3 of the chunk), w4 [4][w_pitch] with leading zeros for fewer taps.
+// Four consecutive tokens x four channels behind a short convolution and silu.  Tokens behind the sequence's end get finite values
+// that meet a beta of zero.
+// TAPS 4: from staged rows (the tokens are rows t .. t + 3 of the chunk), w [4][w_pitch] with leading zeros for fewer taps.
 // TAPS 0: any number of taps, from global memory, w [channel][taps].
 template <int TAPS>
 __device__ __forceinline__ void conv_piece(const unsigned char* tile, int row_bytes, const ConvSource& c, int ch, const float* w, int w_pitch, int taps, int tok0,
-                                           int t, float (&o)[4][8]) {
+                                           int t, float (&o)[4][4]) {
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
-#pragma unroll
-        for (int e = 0; e < 8; ++e) o[i][e] = 0.f;
+    for (int i = 0; i < 4; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+    auto add = [&](int i, float4 x, float4 k) { o[i][0] += x.x * k.x; o[i][1] += x.y * k.y; o[i][2] += x.z * k.z; o[i][3] += x.w * k.w; };
     if constexpr (TAPS > 0) {
-        float wv[TAPS][8];
+        float4 wv[TAPS];
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) {
-            const float4 a = load4(w + (size_t)j * w_pitch), b = load4(w + (size_t)j * w_pitch + 4);
-            wv[j][0] = a.x; wv[j][1] = a.y; wv[j][2] = a.z; wv[j][3] = a.w; wv[j][4] = b.x; wv[j][5] = b.y; wv[j][6] = b.z; wv[j][7] = b.w;
-        }
+        for (int j = 0; j < TAPS; ++j) wv[j] = load4(w + j * w_pitch);
+        const unsigned char* p = tile + t * row_bytes + ch * 2;
 #pragma unroll
         for (int r = 0; r < TAPS + 3; ++r) {
-            float x[8];
-            unpack8(*reinterpret_cast<const uint4*>(tile + (t + r) * row_bytes + ch * 2), x);
+            const float4 x = unpack4(*reinterpret_cast<const uint2*>(p + r * row_bytes));
 #pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                const int j = r - i;
-                if (j < 0 || j >= TAPS) continue;
-#pragma unroll
-                for (int e = 0; e < 8; ++e) o[i][e] += x[e] * wv[j][e];
-            }
+            for (int i = 0; i < 4; ++i)
+                if (r - i >= 0 && r - i < TAPS) add(i, x, wv[r - i]);
         }
     } else {
 #pragma unroll 1
         for (int j = 0; j < taps; ++j)
-#pragma unroll
+#pragma unroll 1
             for (int i = 0; i < 4; ++i) {
                 const int at = tok0 + t + i + j - taps + 1;
-                float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+                float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
                 if (at >= 0) {
-                    if (at < c.count) unpack8(*reinterpret_cast<const uint4*>(c.raw + (size_t)at * c.pitch + ch), x);
+                    if (at < c.count) x = load4(c.raw + (size_t)at * c.pitch + ch);
                 } else {
-#pragma unroll
-                    for (int e = 0; e < 8; ++e)
-                        if (ch + e < c.channels) x[e] = c.hist[(size_t)(taps - 1 + at) * c.stride + ch + e];
+                    const float* h = c.hist + (size_t)(taps - 1 + at) * c.stride + ch;
+                    if (ch < c.channels) x.x = h[0];
+                    if (ch + 1 < c.channels) x.y = h[1];
+                    if (ch + 2 < c.channels) x.z = h[2];
+                    if (ch + 3 < c.channels) x.w = h[3];
                 }
+                const float* wj = w + j;
+                const float4 k = make_float4(wj[0], wj[taps], wj[2 * taps], wj[3 * taps]);
 #pragma unroll
-                for (int e = 0; e < 8; ++e) o[i][e] += x[e] * w[(size_t)e * taps + j];
+                for (int e = 0; e < 4; ++e)
+                    if (e == i) add(e, x, k);
             }
     }
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int e = 0; e < 8; ++e) o[i][e] = tok0 + t + i < c.count ? __fdividef(o[i][e], 1.0f + __expf(-o[i][e])) : 0.f;
+        for (int e = 0; e < 4; ++e) o[i][e] = __fdividef(o[i][e], 1.0f + __expf(-o[i][e]));
 }
 
 // Shared memory of the first kernel; rows of K-major tiles are 64 ND + 8 halves apart (an odd number of 16-byte units).
+constexpr int kPrepThreads = 512;
 constexpr uint32_t kRegion = 17408;                    // 64 rows of 136 halves
 constexpr uint32_t kOffKA = 0;                         // staged q, decayed keys (rows), e^G K, then the image of U'
 constexpr uint32_t kOffQA = kRegion;                   // staged k, decayed queries (rows), staged v, then the image of W
 constexpr uint32_t kOffKB = 2 * kRegion;               // keys decayed to the end of their group, then V
 constexpr uint32_t kOffCOL = 3 * kRegion;              // 96 rows of decayed keys (columns), then T
-constexpr uint32_t kOffAM = kOffCOL + 26112;           // A, fp32 [64][kLd]
+constexpr uint32_t kOffAM = kOffCOL + 26112;           // A, fp32 [64][kLd], then T diag(beta) in fp16
 constexpr uint32_t kOffM = kOffAM + 17408;             // image of M
 constexpr uint32_t kOffG = kOffM + kTile;              // [17][64 ND] log2 decays up to the start of every group
 constexpr uint32_t kOffB = kOffG + 17 * 128 * 4;       // beta [64]
 constexpr uint32_t kPrepSmem = kOffB + 256;
+__device__ __forceinline__ void sync_half(int which) { asm volatile("bar.sync %0, 256;" ::"r"(1 + which) : "memory"); }
 }  // namespace
 
-// grid (heads, chunks, sequences), block 256, two CTAs per SM.  Thread (tg, c8): tokens 4 tg .. 4 tg + 3, channels 8 c8 .. 8 c8 + 7.
+// grid (heads, chunks, sequences), block 512, two CTAs per SM.  Thread (tg, c4): tokens 4 tg .. 4 tg + 3, channels 4 c4 .. 4 c4 + 3; with
+// more than 64 channels a group of tokens is a warp's.
 template <int ND, int TAPS>
-__global__ void __launch_bounds__(256, 2)
+__global__ void __launch_bounds__(kPrepThreads, 2)
 delta_prep_kernel(const DeltaChunkArgs A) {
     extern __shared__ __align__(128) unsigned char sm[];
-    constexpr int DK = 64 * ND, LN = 8 * ND, kP = DK + 8;          // channels, lanes per token, row pitch in halves
+    constexpr int DK = 64 * ND, LN = 16 * ND, kP = DK + 8;         // channels, lanes per token, row pitch in halves
     const DeltaShape& sh = A.sh;
     const LaSeqMeta sq = A.seqs[blockIdx.z];
     const int h = blockIdx.x, chunk = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
@@ -186,89 +186,76 @@ delta_prep_kernel(const DeltaChunkArgs A) {
     float* s_g = reinterpret_cast<float*>(sm + kOffG);
     float* s_beta = reinterpret_cast<float*>(sm + kOffB);
     unsigned char* item = A.scratch + ((first_chunk(sq.row0, blockIdx.z) + chunk) * sh.heads + h) * A.item.bytes();
-    const int tok0 = chunk * kDC, left = sq.count - tok0, D4 = (sh.dim + 3) / 4 * 4, taps = sh.taps;
-    const float* st = A.state + (size_t)sq.slot * sh.state_floats() + (size_t)h * sh.n_vt * sh.tile_floats();
-
-    const int kvh = h / (sh.heads / sh.kv_heads);
+    const int tok0 = chunk * kDC, left = sq.count - tok0, D4 = (sh.dim + 3) / 4 * 4, taps = sh.taps, kvh = h / (sh.heads / sh.kv_heads);
     const __nv_bfloat16* rows = A.qkv + (size_t)sq.row0 * sh.off_b();
+    const float* st = A.state + (size_t)sq.slot * sh.state_floats() + (size_t)h * sh.n_vt * sh.tile_floats();
     const float* hist = st + (size_t)sh.dim * sh.vt;
     const ConvSource cq{rows + kvh * sh.dp, hist, sh.off_b(), D4, sq.count, sh.dim, sh.dp};
     const ConvSource ck{rows + sh.off_k() + kvh * sh.dp, hist + (taps - 1) * D4, sh.off_b(), D4, sq.count, sh.dim, sh.dp};
     if constexpr (TAPS > 0) {
-        stage_raw(base + kOffKA, sm + kOffKA, cq, ND, taps, tok0, tid);
-        stage_raw(base + kOffQA, sm + kOffQA, ck, ND, taps, tok0, tid);
+        stage_raw(base + kOffKA, sm + kOffKA, cq, ND + 2, taps, tok0, tid, kPrepThreads);
+        stage_raw(base + kOffQA, sm + kOffQA, ck, ND + 2, taps, tok0, tid, kPrepThreads);
     }
-    for (int i = tid; i < 64 * kLd / 4; i += 256) reinterpret_cast<float4*>(AM)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int i = tid; i < (int)kTile / 16; i += 256) reinterpret_cast<uint4*>(sm + kOffM)[i] = make_uint4(0u, 0u, 0u, 0u);
+    const int tg = tid / LN, c4 = tid % LN, ch = 4 * c4, t0 = 4 * tg;
+    const bool act = tg < 16, in = act && ch < sh.dp;               // act: whole warps
+    float4 z[4];                                                    // decay pre-activations: requested ahead of the convolutions
+    if (in) {
+        const float* za = A.a + (size_t)(sq.row0 + tok0) * (sh.heads * sh.dp) + h * sh.dp + ch;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) z[i] = load4(za + min(t0 + i, left - 1) * (sh.heads * sh.dp));
+    }
+    for (int i = tid; i < 64 * kLd / 4; i += kPrepThreads) reinterpret_cast<float4*>(AM)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (tid < (int)kTile / 16) reinterpret_cast<uint4*>(sm + kOffM)[tid] = make_uint4(0u, 0u, 0u, 0u);
     if (tid < 64) s_beta[tid] = tid < left ? 1.0f / (1.0f + __expf(-A.b[(size_t)(sq.row0 + tok0 + tid) * sh.heads + h])) : 0.f;
 
-    const int tg = tid / LN, c8 = tid % LN, ch = 8 * c8, t0 = 4 * tg;
-    const bool act = tg < 16;                                       // whole warps
-    uint32_t qh[4][4], kh[4][4];                                    // unit vectors, fp16 pairs
-    float g[4][8];                                                  // decays of the four tokens
+    uint32_t qh[4][2], kh[4][2];                                    // unit vectors, fp16 pairs
+    float g[4][4];                                                  // decays of the four tokens
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-#pragma unroll
-        for (int e = 0; e < 4; ++e) qh[i][e] = kh[i][e] = 0u;
-#pragma unroll
-        for (int e = 0; e < 8; ++e) g[i][e] = 1.f;
+        qh[i][0] = qh[i][1] = kh[i][0] = kh[i][1] = 0u;
+        g[i][0] = g[i][1] = g[i][2] = g[i][3] = 1.f;
     }
     if constexpr (TAPS > 0) {
         staged();
         __syncthreads();
     }
     if (act) {
-        const bool in = ch < sh.dp;
-        float4 z0[4], z1[4];                                        // decay pre-activations: requested ahead of the convolutions
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const float* z = A.a + (size_t)(sq.row0 + tok0 + min(t0 + i, left - 1)) * (sh.heads * sh.dp) + h * sh.dp + (in ? ch : 0);
-            z0[i] = load4(z);
-            z1[i] = load4(z + 4);
-        }
 #pragma unroll
         for (int n = 0; n < 2; ++n) {
             const int col = n * sh.off_k() + kvh * sh.dp + (in ? ch : 0);
-            float o[4][8];
-            conv_piece<TAPS>(sm + (n ? kOffQA : kOffKA), 16 * LN, n ? ck : cq, in ? ch : 0, A.conv + (size_t)col * (TAPS > 0 ? 1 : taps), sh.off_b(), taps, tok0, t0, o);
-            if (!in) {
+            float o[4][4];
+            conv_piece<TAPS>(sm + (n ? kOffQA : kOffKA), 8 * LN, n ? ck : cq, in ? ch : 0, A.conv + col * (TAPS > 0 ? 1 : taps), sh.off_b(), taps, tok0, t0, o);
+            float ss[4];
 #pragma unroll
-                for (int i = 0; i < 4; ++i)
+            for (int i = 0; i < 4; ++i) ss[i] = in ? (o[i][0] * o[i][0] + o[i][1] * o[i][1]) + (o[i][2] * o[i][2] + o[i][3] * o[i][3]) : 0.f;
 #pragma unroll
-                    for (int e = 0; e < 8; ++e) o[i][e] = 0.f;
-            }
+            for (int x = LN / 2; x > 0; x >>= 1)
 #pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                float ss = 0.f;
+                for (int i = 0; i < 4; ++i) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], x);
+            if (in) {
 #pragma unroll
-                for (int e = 0; e < 8; ++e) ss += o[i][e] * o[i][e];
-#pragma unroll
-                for (int x = LN / 2; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
-                const float inv = (n ? 1.0f : rsqrtf((float)sh.dim)) * rsqrtf(ss + 1e-6f);
-#pragma unroll
-                for (int e = 0; e < 4; ++e) (n ? kh : qh)[i][e] = pack_half2(o[i][2 * e] * inv, o[i][2 * e + 1] * inv);
-            }
-        }
-        float sum[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-        if (in) {
-            const float ea = -expf(A.a_log[h]);
-            float dt[8];
-#pragma unroll
-            for (int e = 0; e < 8; ++e) dt[e] = A.dt_bias[h * sh.dp + ch + e] * kDL2e;
-#pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                if (t0 + i >= left) continue;
-                const float zz[8] = {z0[i].x, z0[i].y, z0[i].z, z0[i].w, z1[i].x, z1[i].y, z1[i].z, z1[i].w};
-#pragma unroll
-                for (int e = 0; e < 8; ++e) {
-                    const float l = ea * delta_softplus2(fmaf(zz[e], kDL2e, dt[e]));
-                    sum[e] += l;
-                    g[i][e] = ex2c(l);
+                for (int i = 0; i < 4; ++i) {
+                    const float inv = (n ? 1.0f : rsqrtf((float)sh.dim)) * rsqrtf(ss[i] + 1e-6f);
+                    (n ? kh : qh)[i][0] = pack_half2(o[i][0] * inv, o[i][1] * inv);
+                    (n ? kh : qh)[i][1] = pack_half2(o[i][2] * inv, o[i][3] * inv);
                 }
             }
         }
-        store4(s_g + (tg + 1) * DK + ch, make_float4(sum[0], sum[1], sum[2], sum[3]));
-        store4(s_g + (tg + 1) * DK + ch + 4, make_float4(sum[4], sum[5], sum[6], sum[7]));
+        float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (in) {
+            const float ea = -expf(A.a_log[h]);
+            const float4 d4 = load4(A.dt_bias + h * sh.dp + ch);
+            const float dt[4] = {d4.x * kDL2e, d4.y * kDL2e, d4.z * kDL2e, d4.w * kDL2e};
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                if (t0 + i >= left) continue;
+                const float l0 = ea * delta_softplus2(fmaf(z[i].x, kDL2e, dt[0])), l1 = ea * delta_softplus2(fmaf(z[i].y, kDL2e, dt[1]));
+                const float l2 = ea * delta_softplus2(fmaf(z[i].z, kDL2e, dt[2])), l3 = ea * delta_softplus2(fmaf(z[i].w, kDL2e, dt[3]));
+                sum = make_float4(sum.x + l0, sum.y + l1, sum.z + l2, sum.w + l3);
+                g[i][0] = ex2c(l0); g[i][1] = ex2c(l1); g[i][2] = ex2c(l2); g[i][3] = ex2c(l3);
+            }
+        }
+        store4(s_g + (tg + 1) * DK + ch, sum);
     }
     __syncthreads();
     if (tid < DK) {                                                 // log2 decays from the chunk's start to the start of every group
@@ -284,30 +271,31 @@ delta_prep_kernel(const DeltaChunkArgs A) {
 #pragma unroll
         for (int i = 0; i < 16; ++i) acc[i] = 0.f;
 #pragma unroll
-        for (int e2 = 0; e2 < 4; ++e2) {
+        for (int e2 = 0; e2 < 2; ++e2) {
             float2 q[4], k[4];
 #pragma unroll
             for (int i = 0; i < 4; ++i) { q[i] = unpack_half2(qh[i][e2]); k[i] = unpack_half2(kh[i][e2]); }
-            int na = 0, nm = 6;
 #pragma unroll
-            for (int t = 0; t < 4; ++t) {
+            for (int s = 0; s < 4; ++s) {
+                float wx = k[s].x, wy = k[s].y;                     // key s as token t sees it
 #pragma unroll
-                for (int s = 0; s <= t; ++s) {
-                    float wx = k[s].x, wy = k[s].y;
-#pragma unroll
-                    for (int j = s + 1; j <= t; ++j) { wx *= g[j][2 * e2]; wy *= g[j][2 * e2 + 1]; }
-                    if (s < t) { acc[na] += k[t].x * wx + k[t].y * wy; ++na; }
-                    acc[nm] += q[t].x * wx + q[t].y * wy;
-                    ++nm;
+                for (int t = 0; t < 4; ++t) {
+                    if (t < s) continue;
+                    if (t > s) {
+                        wx *= g[t][2 * e2];
+                        wy *= g[t][2 * e2 + 1];
+                        acc[t * (t - 1) / 2 + s] += k[t].x * wx + k[t].y * wy;
+                    }
+                    acc[6 + t * (t + 1) / 2 + s] += q[t].x * wx + q[t].y * wy;
                 }
             }
         }
         // sixteen sums over the lanes of a token: halve the values while halving the lanes
         int n = 16, at = 0;
 #pragma unroll
-        for (int x = LN / 2; x > 0; x >>= 1) {
+        for (int x = LN / 2; x > LN / 32; x >>= 1) {
             n >>= 1;
-            const bool top = c8 & x;
+            const bool top = c4 & x;
 #pragma unroll
             for (int e = 0; e < 8; ++e) {
                 if (e >= n) continue;
@@ -316,73 +304,57 @@ delta_prep_kernel(const DeltaChunkArgs A) {
             }
             if (top) at += n;
         }
-#pragma unroll
-        for (int e = 0; e < 2 / ND; ++e) {
-            const int idx = at + e;
-            // pairs (t, s): A: 10 20 21 30 31 32, M: 00 10 11 20 21 22 30 31 32 33, packed as 4 t + s
-            const uint32_t packed = idx < 8 ? 0x40EDC984u : 0xFEDCA985u;
-            const int p = (int)(packed >> (4 * (idx & 7))) & 15, t = t0 + (p >> 2), s = t0 + (p & 3);
-            if (idx < 6) AM[t * kLd + s] = s_beta[t] * acc[e];
-            else *reinterpret_cast<__half*>(sm + kOffM + sw(t, s >> 3) + 2 * (s & 7)) = __float2half_rn(acc[e]);
+        if constexpr (ND == 2) acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], 1);
+        // pairs (t, s): A: 10 20 21 30 31 32, M: 00 10 11 20 21 22 30 31 32 33, packed as 4 t + s
+        const uint32_t codes = at < 8 ? 0x40EDC984u : 0xFEDCA985u;
+        const int p = (int)(codes >> (4 * (at & 7))) & 15, t = t0 + (p >> 2), s = t0 + (p & 3);
+        if (ND == 1 || !(lane & 1)) {
+            if (at < 6) AM[t * kLd + s] = s_beta[t] * acc[0];
+            else *reinterpret_cast<__half*>(sm + kOffM + sw(t, s >> 3) + 2 * (s & 7)) = __float2half_rn(acc[0]);
         }
     }
     __syncthreads();
     const float* r0 = s_g + tg * DK + ch;                           // up to this group's start / end, up to the chunk's end
     const float *r1 = r0 + DK, *rC = s_g + 16 * DK + ch;
-    auto piece = [&](uint32_t off, int row) { return reinterpret_cast<uint4*>(sm + off + row * kP * 2 + ch * 2); };
-    auto scaled = [](uint4 v, const uint32_t (&f)[4]) {
-        return make_uint4(mul_half2(v.x, f[0]), mul_half2(v.y, f[1]), mul_half2(v.z, f[2]), mul_half2(v.w, f[3]));
-    };
-    auto packed = [](const float (&x)[8], uint32_t (&f)[4]) {
-#pragma unroll
-        for (int e = 0; e < 4; ++e) f[e] = pack_half2(x[2 * e], x[2 * e + 1]);
-    };
-    auto factors = [](uint32_t (&f)[4], const float* to, const float* from) {     // 2^(to - from)
-        const float4 a = load4(to), b = load4(to + 4), c = load4(from), d = load4(from + 4);
-        f[0] = pack_half2(ex2c(a.x - c.x), ex2c(a.y - c.y)); f[1] = pack_half2(ex2c(a.z - c.z), ex2c(a.w - c.w));
-        f[2] = pack_half2(ex2c(b.x - d.x), ex2c(b.y - d.y)); f[3] = pack_half2(ex2c(b.z - d.z), ex2c(b.w - d.w));
+    auto piece = [&](uint32_t off, int row) { return reinterpret_cast<uint2*>(sm + off + row * kP * 2 + ch * 2); };
+    auto image = [&](uint32_t off, int row) { return reinterpret_cast<uint2*>(item + off + (ch >> 6) * kTile + sw(row, (ch >> 3) & 7) + (ch & 4) * 2); };
+    auto scaled = [](uint2 v, uint2 f) { return make_uint2(mul_half2(v.x, f.x), mul_half2(v.y, f.y)); };
+    auto factors = [](const float* to, const float* from) {         // 2^(to - from)
+        const float4 a = load4(to), b = load4(from);
+        return make_uint2(pack_half2(ex2c(a.x - b.x), ex2c(a.y - b.y)), pack_half2(ex2c(a.z - b.z), ex2c(a.w - b.w)));
     };
     const int blk = tg >> 2, own = tg & 3;
     if (act) {
-        unsigned char* img = item + (c8 >> 3) * kTile;
         {
-            float run[8];
-            uint32_t f[4], x[4];
-            factors(x, r0, s_g + ch);
-#pragma unroll
-            for (int e = 0; e < 8; ++e) run[e] = 1.f;
+            float run[4] = {1.f, 1.f, 1.f, 1.f};
+            const uint2 x = factors(r0, s_g + ch);
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
 #pragma unroll
-                for (int e = 0; e < 8; ++e) run[e] *= g[i][e];
-                packed(run, f);
-                const uint4 q = scaled(make_uint4(qh[i][0], qh[i][1], qh[i][2], qh[i][3]), f);
+                for (int e = 0; e < 4; ++e) run[e] *= g[i][e];
+                const uint2 f = make_uint2(pack_half2(run[0], run[1]), pack_half2(run[2], run[3]));
+                const uint2 q = scaled(make_uint2(qh[i][0], qh[i][1]), f);
                 *piece(kOffQA, t0 + i) = q;
-                *piece(kOffKA, t0 + i) = scaled(make_uint4(kh[i][0], kh[i][1], kh[i][2], kh[i][3]), f);
-                *reinterpret_cast<uint4*>(img + A.item.off_q() + sw(t0 + i, c8 & 7)) = scaled(q, x);
+                *piece(kOffKA, t0 + i) = scaled(make_uint2(kh[i][0], kh[i][1]), f);
+                *image(A.item.off_q(), t0 + i) = scaled(q, x);
             }
         }
         {
-            float run[8];
-            uint32_t f[4], x[4];
-            factors(x, rC, r1);
-#pragma unroll
-            for (int e = 0; e < 8; ++e) run[e] = 1.f;
+            float run[4] = {1.f, 1.f, 1.f, 1.f};
+            const uint2 x = factors(rC, r1);
 #pragma unroll
             for (int i = 3; i >= 0; --i) {
-                packed(run, f);
-                const uint4 k = scaled(make_uint4(kh[i][0], kh[i][1], kh[i][2], kh[i][3]), f);
+                const uint2 k = scaled(make_uint2(kh[i][0], kh[i][1]), make_uint2(pack_half2(run[0], run[1]), pack_half2(run[2], run[3])));
                 *piece(kOffKB, t0 + i) = k;
-                *reinterpret_cast<uint4*>(img + A.item.off_k() + sw(t0 + i, c8 & 7)) = scaled(k, x);
+                *image(A.item.off_k(), t0 + i) = scaled(k, x);
 #pragma unroll
-                for (int e = 0; e < 8; ++e) run[e] *= g[i][e];
+                for (int e = 0; e < 4; ++e) run[e] *= g[i][e];
             }
         }
         // copies for the later groups of the block: 24 rows per block, 4 + 8 + 12
 #pragma unroll 1
         for (int i = own + 1; i < 4; ++i) {
-            uint32_t f[4];
-            factors(f, s_g + (4 * blk + i) * DK + ch, r1);
+            const uint2 f = factors(s_g + (4 * blk + i) * DK + ch, r1);
             const int row = 24 * blk + (i == 1 ? 0 : i == 2 ? 4 : 12) + 4 * own;
 #pragma unroll
             for (int s = 0; s < 4; ++s) *piece(kOffCOL, row + s) = scaled(*piece(kOffKB, t0 + s), f);
@@ -395,55 +367,8 @@ delta_prep_kernel(const DeltaChunkArgs A) {
         if (q) *reinterpret_cast<uint32_t*>(sm + kOffM + sw(t, s >> 3) + 2 * (s & 7)) = pack_half2(x, y);
         else *reinterpret_cast<float2*>(AM + t * kLd + s) = make_float2(s_beta[t] * x, s_beta[t] * y);
     };
-    {   // ---- groups against groups: a block's 16 rows x 24 columns per warp ----
-        const int b = warp >> 1;
-        const bool q = warp & 1;
-        float d[3][4];
-#pragma unroll
-        for (int n = 0; n < 3; ++n) d[n][0] = d[n][1] = d[n][2] = d[n][3] = 0.f;
-        const uint32_t aa = a_addr(q ? kOffQA : kOffKA, 16 * b), ba = b_addr(kOffCOL, 24 * b);
-#pragma unroll
-        for (int k = 0; k < 4 * ND; ++k) {
-            uint32_t a[4], b0, b1;
-            ldm4(a, aa + k * 32);
-#pragma unroll
-            for (int n = 0; n < 3; ++n) {
-                ldm2(b0, b1, ba + n * 8 * kP * 2 + k * 32);
-                mma_16816(d[n], a[0], a[1], a[2], a[3], b0, b1);
-            }
-        }
-#pragma unroll
-        for (int n = 0; n < 3; ++n) {
-            const int c = 8 * n + 2 * t4, i = c < 4 ? 1 : c < 12 ? 2 : 3, s = 16 * b + c - (i == 1 ? 0 : i == 2 ? 4 : 12);
-            if ((g4 >> 2) == i) put2(q, 16 * b + g4, s, d[n][0], d[n][1]);
-            if (((g4 + 8) >> 2) == i) put2(q, 16 * b + g4 + 8, s, d[n][2], d[n][3]);
-        }
-    }
-    __syncthreads();
-    if (act) {
-        // ---- rows decay on from the start of their block, columns up to the start of a later one: 16 + 32 + 48 rows ----
-        uint32_t f[4];
-        factors(f, r0, s_g + 4 * blk * DK + ch);
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            *piece(kOffQA, t0 + i) = scaled(*piece(kOffQA, t0 + i), f);
-            *piece(kOffKA, t0 + i) = scaled(*piece(kOffKA, t0 + i), f);
-        }
-#pragma unroll 1
-        for (int I = blk + 1; I < 4; ++I) {
-            factors(f, s_g + 4 * I * DK + ch, r1);
-            const int row = (I == 1 ? 0 : I == 2 ? 16 : 48) + t0;
-#pragma unroll
-            for (int s = 0; s < 4; ++s) *piece(kOffCOL, row + s) = scaled(*piece(kOffKB, t0 + s), f);
-        }
-    }
-    __syncthreads();
-#pragma unroll 1
-    for (int u = warp; u < 24; u += 8) {   // ---- blocks against blocks: 16 rows x 8 columns at a time ----
-        const bool q = u & 1;
-        const int v = u >> 1, I = v < 2 ? 1 : v < 6 ? 2 : 3, n = v - (I == 1 ? 0 : I == 2 ? 2 : 6);
-        float d[4] = {0.f, 0.f, 0.f, 0.f};
-        const uint32_t aa = a_addr(q ? kOffQA : kOffKA, 16 * I), ba = b_addr(kOffCOL, (I == 1 ? 0 : I == 2 ? 16 : 48) + 8 * n);
+    auto product = [&](uint32_t aa, uint32_t ba, float (&d)[4]) {   // 16 rows x 8 columns over all channels
+        d[0] = d[1] = d[2] = d[3] = 0.f;
 #pragma unroll
         for (int k = 0; k < 4 * ND; ++k) {
             uint32_t a[4], b0, b1;
@@ -451,74 +376,104 @@ delta_prep_kernel(const DeltaChunkArgs A) {
             ldm2(b0, b1, ba + k * 32);
             mma_16816(d, a[0], a[1], a[2], a[3], b0, b1);
         }
+    };
+#pragma unroll 1
+    for (int u = warp; u < 24; u += 16) {   // ---- groups against groups: a block's 16 rows x 8 of its 24 columns at a time ----
+        const bool q = u & 1;
+        const int b = (u >> 1) & 3, n = u >> 3;
+        float d[4];
+        product(a_addr(q ? kOffQA : kOffKA, 16 * b), b_addr(kOffCOL, 24 * b + 8 * n), d);
+        const int c = 8 * n + 2 * t4, i = c < 4 ? 1 : c < 12 ? 2 : 3, s = 16 * b + c - (i == 1 ? 0 : i == 2 ? 4 : 12);
+        if ((g4 >> 2) == i) put2(q, 16 * b + g4, s, d[0], d[1]);
+        if (((g4 + 8) >> 2) == i) put2(q, 16 * b + g4 + 8, s, d[2], d[3]);
+    }
+    __syncthreads();
+    if (act) {
+        // ---- rows decay on from the start of their block, columns up to the start of a later one: 16 + 32 + 48 rows ----
+        const uint2 f = factors(r0, s_g + 4 * blk * DK + ch);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            *piece(kOffQA, t0 + i) = scaled(*piece(kOffQA, t0 + i), f);
+            *piece(kOffKA, t0 + i) = scaled(*piece(kOffKA, t0 + i), f);
+        }
+#pragma unroll 1
+        for (int I = blk + 1; I < 4; ++I) {
+            const uint2 x = factors(s_g + 4 * I * DK + ch, r1);
+            const int row = (I == 1 ? 0 : I == 2 ? 16 : 48) + t0;
+#pragma unroll
+            for (int s = 0; s < 4; ++s) *piece(kOffCOL, row + s) = scaled(*piece(kOffKB, t0 + s), x);
+        }
+    }
+    __syncthreads();
+#pragma unroll 1
+    for (int u = warp; u < 24; u += 16) {   // ---- blocks against blocks ----
+        const bool q = u & 1;
+        const int v = u >> 1, I = v < 2 ? 1 : v < 6 ? 2 : 3, n = v - (I == 1 ? 0 : I == 2 ? 2 : 6);
+        float d[4];
+        product(a_addr(q ? kOffQA : kOffKA, 16 * I), b_addr(kOffCOL, (I == 1 ? 0 : I == 2 ? 16 : 48) + 8 * n), d);
         put2(q, 16 * I + g4, 8 * n + 2 * t4, d[0], d[1]);
         put2(q, 16 * I + g4 + 8, 8 * n + 2 * t4, d[2], d[3]);
     }
     __syncthreads();
-    const int nv = A.item.nv, vln = 8 * nv, kVP = 64 * nv + 8;      // lanes per token, row pitch of V
-    auto values = [&](int tile) {
+    const int nv = A.item.nv, kVP = 64 * nv + 8;                    // row pitch of V
+    auto load_values = [&](int tile, int vt, int n, int which) {    // the values of a state tile, staged over the queries, go to KB; threads vt of n, half `which`
         const float* hv = hist + tile * sh.tile_floats() + 2 * (taps - 1) * D4;
-        return ConvSource{rows + sh.off_v() + h * sh.vp + tile * kMlstmTile, hv, sh.off_b(), sh.vt, sq.count, sh.vdim - tile * kMlstmTile, sh.vp - tile * kMlstmTile};
-    };
-    auto load_values = [&](int tile) {                              // behind the staging of the same tile
-        const int vtg = tid / vln, vc = 8 * (tid % vln), t = 4 * vtg;
-        const ConvSource c = values(tile);
+        const int c0 = tile * kMlstmTile, left_v = sh.vp - c0;
+        const ConvSource c{rows + sh.off_v() + h * sh.vp + c0, hv, sh.off_b(), sh.vt, sq.count, sh.vdim - c0, left_v};
         if constexpr (TAPS > 0) {
+            stage_raw(base + kOffQA, sm + kOffQA, c, nv + 2, taps, tok0, vt, n);
             staged();
-            __syncthreads();
+            if (which < 0) __syncthreads(); else sync_half(which);
         }
-        if (vtg >= 16) return;
-        const bool in = vc < c.padded;
-        const int col = sh.off_v() + h * sh.vp + tile * kMlstmTile + (in ? vc : 0);
-        float o[4][8];
-        conv_piece<TAPS>(sm + kOffQA, 128 * nv, c, in ? vc : 0, A.conv + (size_t)col * (TAPS > 0 ? 1 : taps), sh.off_b(), taps, tok0, t, o);
+        for (int i = vt; i < 256 * nv; i += n) {
+            const int t = 4 * (i >> (nv + 3)), vc = 4 * (i & (16 * nv - 1));
+            uint2 r[4] = {};
+            if (vc < left_v) {
+                float o[4][4];
+                conv_piece<TAPS>(sm + kOffQA, 128 * nv, c, vc, A.conv + (sh.off_v() + h * sh.vp + c0 + vc) * (TAPS > 0 ? 1 : taps), sh.off_b(), taps, tok0, t, o);
 #pragma unroll
-        for (int i = 0; i < 4; ++i)
-            *reinterpret_cast<uint4*>(sm + kOffKB + ((t + i) * kVP + vc) * 2) =
-                in ? make_uint4(pack_half2(o[i][0], o[i][1]), pack_half2(o[i][2], o[i][3]), pack_half2(o[i][4], o[i][5]), pack_half2(o[i][6], o[i][7]))
-                   : make_uint4(0u, 0u, 0u, 0u);
+                for (int e = 0; e < 4; ++e) r[e] = make_uint2(pack_half2(o[e][0], o[e][1]), pack_half2(o[e][2], o[e][3]));
+            }
+#pragma unroll
+            for (int e = 0; e < 4; ++e) *reinterpret_cast<uint2*>(sm + kOffKB + ((t + e) * kVP + vc) * 2) = r[e];
+        }
     };
-    if constexpr (TAPS > 0) stage_raw(base + kOffQA, sm + kOffQA, values(0), nv, taps, tok0, tid);
-    // ---- T = (I + A)^-1 over the column copies; meanwhile M goes out and the keys decay from the chunk's start ----
-    if (tid < 64) invert_diagonal(AM, TF, tid);
-    for (int i = tid; i < (int)kTile / 16; i += 256) reinterpret_cast<uint4*>(item + A.item.off_m())[i] = reinterpret_cast<uint4*>(sm + kOffM)[i];
-    if (act) {
-        uint32_t f[4];
-        factors(f, s_g + 4 * blk * DK + ch, s_g + ch);
+    if (warp < 8) {   // ---- T = (I + A)^-1 over the column copies ----
+        if (tid < 64) invert_diagonal(AM, TF, tid);
+        sync_half(0);
+        if (warp < 6) scale_blocks(AM, TF, warp, lane);
+        sync_half(0);
+        solve_columns(AM, TF, warp, lane);
+    } else {          // ---- meanwhile M goes out and the first values come in ----
+        for (int i = tid - 256; i < (int)kTile / 16; i += 256) reinterpret_cast<uint4*>(item + A.item.off_m())[i] = reinterpret_cast<uint4*>(sm + kOffM)[i];
+        load_values(0, tid - 256, 256, 1);
+    }
+    if (act) {        // the keys decay from the chunk's start
+        const uint2 f = factors(s_g + 4 * blk * DK + ch, s_g + ch);
 #pragma unroll
         for (int i = 0; i < 4; ++i) *piece(kOffKA, t0 + i) = scaled(*piece(kOffKA, t0 + i), f);
     }
     __syncthreads();
-    if (warp < 6) scale_blocks(AM, TF, warp, lane);
-    __syncthreads();
-    solve_columns(AM, TF, warp, lane);
-    // ---- the values of a state tile: staged over the queries (requested ahead of the inverse), behind their convolution over KB ----
-    load_values(0);
-    __syncthreads();
-    {   // T diag(beta) as a swizzled fp16 tile over A, a quarter of a row per thread; blocks above the diagonal are never read
-        const int i = tid >> 2, qd = tid & 3;
-        if (qd <= i >> 4) {
-#pragma unroll
-            for (int p = 0; p < 2; ++p) {
-                const int s = 16 * qd + 8 * p;
-                const float4 a = load4(TF + i * kLd + s), b = load4(TF + i * kLd + s + 4), c = load4(s_beta + s), d = load4(s_beta + s + 4);
-                *reinterpret_cast<uint4*>(sm + kOffAM + sw(i, 2 * qd + p)) = make_uint4(pack_half2(a.x * c.x, a.y * c.y), pack_half2(a.z * c.z, a.w * c.w),
-                                                                                       pack_half2(b.x * d.x, b.y * d.y), pack_half2(b.z * d.z, b.w * d.w));
-            }
+    {   // T diag(beta) as a swizzled fp16 tile over A, eight entries per thread; blocks above the diagonal are never read
+        const int i = tid >> 3, p = tid & 7, s = 8 * p;
+        if ((p >> 1) <= i >> 4) {
+            const float4 a = load4(TF + i * kLd + s), b = load4(TF + i * kLd + s + 4), c = load4(s_beta + s), d = load4(s_beta + s + 4);
+            *reinterpret_cast<uint4*>(sm + kOffAM + sw(i, p)) = make_uint4(pack_half2(a.x * c.x, a.y * c.y), pack_half2(a.z * c.z, a.w * c.w),
+                                                                          pack_half2(b.x * d.x, b.y * d.y), pack_half2(b.z * d.z, b.w * d.w));
         }
     }
     __syncthreads();
-    {   // ---- W = (T diag(beta)) (e^G K): 16 rows x 32 ND columns per warp ----
-        const int i = warp >> 1, c0 = (warp & 1) * 32 * ND;
-        float d[4 * ND][4];
+    {   // ---- W = (T diag(beta)) (e^G K): 16 rows x 16 ND columns per warp ----
+        const int i = warp >> 2, c0 = (warp & 3) * 16 * ND;
+        float d[2 * ND][4];
 #pragma unroll
-        for (int n = 0; n < 4 * ND; ++n) d[n][0] = d[n][1] = d[n][2] = d[n][3] = 0.f;
+        for (int n = 0; n < 2 * ND; ++n) d[n][0] = d[n][1] = d[n][2] = d[n][3] = 0.f;
         for (int k = 0; k <= i; ++k) {
             uint32_t a[4];
             ldm4(a, base + kOffAM + sw(16 * i + (lane & 15), 2 * k + (lane >> 4)));
             const uint32_t ka = base + kOffKA + ((16 * k + (lane & 15)) * kP + c0 + (lane >> 4) * 8) * 2;
 #pragma unroll
-            for (int n = 0; n < 4 * ND; n += 2) {
+            for (int n = 0; n < 2 * ND; n += 2) {
                 uint32_t b[4];
                 ldm4t(b, ka + n * 16);
                 mma_16816(d[n], a[0], a[1], a[2], a[3], b[0], b[1]);
@@ -526,7 +481,7 @@ delta_prep_kernel(const DeltaChunkArgs A) {
             }
         }
 #pragma unroll
-        for (int n = 0; n < 4 * ND; ++n) {
+        for (int n = 0; n < 2 * ND; ++n) {
             const int c = c0 + 8 * n;
             unsigned char* w = sm + kOffQA + (c >> 6) * kTile;
             *reinterpret_cast<uint32_t*>(w + sw(16 * i + g4, (c >> 3) & 7) + 4 * t4) = pack_half2(d[n][0], d[n][1]);
@@ -534,17 +489,17 @@ delta_prep_kernel(const DeltaChunkArgs A) {
         }
     }
     __syncthreads();
-    for (int i = tid; i < (int)(ND * kTile) / 16; i += 256) reinterpret_cast<uint4*>(item)[i] = reinterpret_cast<uint4*>(sm + kOffQA)[i];
-    // ---- U'^T = V^T (T diag(beta))^T of every state tile: 16 values x 64 (or 32) tokens per warp ----
+    for (int i = tid; i < (int)(ND * kTile) / 16; i += kPrepThreads) reinterpret_cast<uint4*>(item)[i] = reinterpret_cast<uint4*>(sm + kOffQA)[i];
+    // ---- U'^T = V^T (T diag(beta))^T of every state tile: 16 values x every second (fourth) token tile per warp ----
     for (int tile = 0;; ++tile) {
-        const int mt = warp % (4 * nv), part = nv == 2 ? 0 : warp >> 2, parts = nv == 2 ? 1 : 2;      // token tiles part, part + parts, ..
+        const int mt = warp & (4 * nv - 1), part = warp >> (nv + 1), parts = 4 / nv;
         uint32_t a[4][4];
 #pragma unroll
         for (int k = 0; k < 4; ++k)
             ldm4t(a[k], base + kOffKB + ((16 * k + (lane & 7) + ((lane >> 4) & 1) * 8) * kVP + 16 * mt + ((lane >> 3) & 1) * 8) * 2);
 #pragma unroll
         for (int n = 0; n < 8; ++n) {
-            if (n % parts != part) continue;
+            if ((n & (parts - 1)) != part) continue;
             float d[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
             for (int k = 0; k <= n >> 1; ++k) {
@@ -557,10 +512,9 @@ delta_prep_kernel(const DeltaChunkArgs A) {
         }
         __syncthreads();
         uint4* dst = reinterpret_cast<uint4*>(item + A.item.off_u() + tile * nv * kTile);
-        for (int i = tid; i < (int)(nv * kTile) / 16; i += 256) dst[i] = reinterpret_cast<uint4*>(sm + kOffKA)[i];
+        for (int i = tid; i < (int)(nv * kTile) / 16; i += kPrepThreads) dst[i] = reinterpret_cast<uint4*>(sm + kOffKA)[i];
         if (tile + 1 == sh.n_vt) break;
-        if constexpr (TAPS > 0) stage_raw(base + kOffQA, sm + kOffQA, values(tile + 1), nv, taps, tok0, tid);
-        load_values(tile + 1);
+        load_values(tile + 1, tid, kPrepThreads, -1);
         __syncthreads();
     }
 }
@@ -821,7 +775,7 @@ int launch_delta_chunk(const DeltaShape& sh, const void* qkv, const float* a, co
             B2_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, kWalkSmem)));
     DeltaChunkArgs A{sh, it, (const __nv_bfloat16*)qkv, a, b, conv, a_log, dt_bias, state, d_seqs, max_seqs, (unsigned char*)scratch};
     const dim3 gp(sh.heads, ceil_div(max_count, kDC), n_seqs);
-    auto prep = [&](auto kernel) { kernel<<<gp, 256, kPrepSmem, s>>>(A); };
+    auto prep = [&](auto kernel) { kernel<<<gp, kPrepThreads, kPrepSmem, s>>>(A); };
     if (it.nd == 2) { if (sh.taps <= 4) prep(delta_prep_kernel<2, 4>); else prep(delta_prep_kernel<2, 0>); }
     else { if (sh.taps <= 4) prep(delta_prep_kernel<1, 4>); else prep(delta_prep_kernel<1, 0>); }
     B2_LAUNCH_CHECK();
