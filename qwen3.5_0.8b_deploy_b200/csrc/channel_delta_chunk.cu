@@ -45,6 +45,17 @@ __device__ __forceinline__ float ex2c(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+__device__ __forceinline__ float rcpc(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float rsqc(float x) {
+    float y;
+    asm("rsqrt.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float sigmoidc(float x) { return rcpc(1.0f + ex2c(x * -kDL2e)); }
 __device__ __forceinline__ uint32_t sw(int r, int p) { return (uint32_t)(r * 128 + ((p ^ (r & 7)) << 4)); }   // 16-byte piece p of row r
 __device__ __forceinline__ float2 unpack_half2(uint32_t v) { return __half22float2(*reinterpret_cast<const __half2*>(&v)); }
 __device__ __forceinline__ uint32_t mul_half2(uint32_t a, uint32_t b) {
@@ -151,7 +162,7 @@ __device__ __forceinline__ void conv_piece(const unsigned char* tile, int row_by
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) o[i][e] = __fdividef(o[i][e], 1.0f + __expf(-o[i][e]));
+        for (int e = 0; e < 4; ++e) o[i][e] *= sigmoidc(o[i][e]);
 }
 
 // Shared memory of the first kernel; rows of K-major tiles are 64 ND + 8 halves apart (an odd number of 16-byte units).
@@ -206,7 +217,7 @@ delta_prep_kernel(const DeltaChunkArgs A) {
     }
     for (int i = tid; i < 64 * kLd / 4; i += kPrepThreads) reinterpret_cast<float4*>(AM)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (tid < (int)kTile / 16) reinterpret_cast<uint4*>(sm + kOffM)[tid] = make_uint4(0u, 0u, 0u, 0u);
-    if (tid < 64) s_beta[tid] = tid < left ? 1.0f / (1.0f + __expf(-A.b[(size_t)(sq.row0 + tok0 + tid) * sh.heads + h])) : 0.f;
+    if (tid < 64) s_beta[tid] = tid < left ? sigmoidc(A.b[(size_t)(sq.row0 + tok0 + tid) * sh.heads + h]) : 0.f;
 
     uint32_t qh[4][2], kh[4][2];                                    // unit vectors, fp16 pairs
     float g[4][4];                                                  // decays of the four tokens
@@ -235,7 +246,7 @@ delta_prep_kernel(const DeltaChunkArgs A) {
             if (in) {
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
-                    const float inv = (n ? 1.0f : rsqrtf((float)sh.dim)) * rsqrtf(ss[i] + 1e-6f);
+                    const float inv = (n ? 1.0f : rsqc((float)sh.dim)) * rsqc(ss[i] + 1e-6f);
                     (n ? kh : qh)[i][0] = pack_half2(o[i][0] * inv, o[i][1] * inv);
                     (n ? kh : qh)[i][1] = pack_half2(o[i][2] * inv, o[i][3] * inv);
                 }
@@ -263,7 +274,7 @@ delta_prep_kernel(const DeltaChunkArgs A) {
         s_g[tid] = 0.f;
 #pragma unroll
         for (int j = 1; j <= 16; ++j) { run += s_g[j * DK + tid]; s_g[j * DK + tid] = run; }
-        reinterpret_cast<float*>(item + A.item.off_e())[tid] = ex2c(run);
+        reinterpret_cast<float*>(item + (3 * ND + 1) * kTile)[tid] = ex2c(run);
     }
     if (act) {
         // ---- pairs inside the group: factors are running products ----
@@ -317,7 +328,10 @@ delta_prep_kernel(const DeltaChunkArgs A) {
     const float* r0 = s_g + tg * DK + ch;                           // up to this group's start / end, up to the chunk's end
     const float *r1 = r0 + DK, *rC = s_g + 16 * DK + ch;
     auto piece = [&](uint32_t off, int row) { return reinterpret_cast<uint2*>(sm + off + row * kP * 2 + ch * 2); };
-    auto image = [&](uint32_t off, int row) { return reinterpret_cast<uint2*>(item + off + (ch >> 6) * kTile + sw(row, (ch >> 3) & 7) + (ch & 4) * 2); };
+    // image of a [64][64 ND] tile, row t0 + i (i < 4), this thread's channels: sw() with t0 a multiple of four
+    unsigned char* img = item + (ch >> 6) * kTile + t0 * 128 + (ch & 4) * 2;
+    const int pb = ((ch >> 3) & 7) ^ (t0 & 4);
+    auto image = [&](uint32_t off, int i) { return reinterpret_cast<uint2*>(img + (off + i * 128 + ((pb ^ i) << 4))); };
     auto scaled = [](uint2 v, uint2 f) { return make_uint2(mul_half2(v.x, f.x), mul_half2(v.y, f.y)); };
     auto factors = [](const float* to, const float* from) {         // 2^(to - from)
         const float4 a = load4(to), b = load4(from);
@@ -336,7 +350,7 @@ delta_prep_kernel(const DeltaChunkArgs A) {
                 const uint2 q = scaled(make_uint2(qh[i][0], qh[i][1]), f);
                 *piece(kOffQA, t0 + i) = q;
                 *piece(kOffKA, t0 + i) = scaled(make_uint2(kh[i][0], kh[i][1]), f);
-                *image(A.item.off_q(), t0 + i) = scaled(q, x);
+                *image(ND * kTile, i) = scaled(q, x);
             }
         }
         {
@@ -346,7 +360,7 @@ delta_prep_kernel(const DeltaChunkArgs A) {
             for (int i = 3; i >= 0; --i) {
                 const uint2 k = scaled(make_uint2(kh[i][0], kh[i][1]), make_uint2(pack_half2(run[0], run[1]), pack_half2(run[2], run[3])));
                 *piece(kOffKB, t0 + i) = k;
-                *image(A.item.off_k(), t0 + i) = scaled(k, x);
+                *image(2 * ND * kTile, i) = scaled(k, x);
 #pragma unroll
                 for (int e = 0; e < 4; ++e) run[e] *= g[i][e];
             }
@@ -445,7 +459,7 @@ delta_prep_kernel(const DeltaChunkArgs A) {
         sync_half(0);
         solve_columns(AM, TF, warp, lane);
     } else {          // ---- meanwhile M goes out and the first values come in ----
-        for (int i = tid - 256; i < (int)kTile / 16; i += 256) reinterpret_cast<uint4*>(item + A.item.off_m())[i] = reinterpret_cast<uint4*>(sm + kOffM)[i];
+        for (int i = tid - 256; i < (int)kTile / 16; i += 256) reinterpret_cast<uint4*>(item + 3 * ND * kTile)[i] = reinterpret_cast<uint4*>(sm + kOffM)[i];
         load_values(0, tid - 256, 256, 1);
     }
     if (act) {        // the keys decay from the chunk's start
