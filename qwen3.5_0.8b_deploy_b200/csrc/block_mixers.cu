@@ -171,7 +171,7 @@ int delta_forward(BlockModel& m, DeltaOp& op, const LayerRun& run, const PassRow
         B2_TRY(gemm_typed(s, m.low.p, sh.low(), (const char*)op.w_gate.p + (size_t)acols * sh.low() * e, g, gcols, op.elem, op.elem, p.rows, gcols, sh.low()));
         {
             ProfScope prof(PROF_DELTA_PREFILL, s);
-            B2_TRY(launch_delta_chunk(sh, m.proj.p, a, b, sh.taps <= 4 ? op.conv4.f() : op.conv.f(), op.a_log.f(), op.dt_bias.f(), p.d_seqs, p.n_seqs, p.max_count, m.cfg.max_seqs, state,
+            B2_TRY(launch_delta_chunk(sh, m.proj.p, a, b, sh.taps <= 4 ? op.conv4.f() : op.conv.f(), op.a_log.f(), op.dt_bias.f(), p.d_seqs, p.n_seqs, p.max_count, p.rows, m.cfg.max_seqs, state,
                                       m.chunk.p, m.core.f(), m.error.i(), s));
         }
         return launch_delta_head_norm(op.elem, sh, m.core.f(), g, false, gcols, op.norm_w.f(), p.rows, m.mixed.p, s);

@@ -220,7 +220,7 @@ bool delta_chunk_fits(const DeltaShape& sh);
 size_t delta_chunk_bytes(const DeltaShape& sh);        // scratch per 64 rows of a pass (and one more such piece per sequence)
 // qkv: bf16 [rows][off_b]; conv: conv4 with up to four taps; a: fp32 [rows][heads * dp], b: fp32 [rows][heads], the gates' pre-activations.
 int launch_delta_chunk(const DeltaShape& sh, const void* qkv, const float* a, const float* b, const float* conv, const float* a_log, const float* dt_bias,
-                       const LaSeqMeta* d_seqs, int n_seqs, int max_count, int max_seqs, float* state, void* scratch, float* core, int* d_error,
+                       const LaSeqMeta* d_seqs, int n_seqs, int max_count, int rows, int max_seqs, float* state, void* scratch, float* core, int* d_error,
                        cudaStream_t s);
 
 struct DeltaOp {

@@ -83,6 +83,7 @@ struct DeltaChunkArgs {
     const LaSeqMeta* seqs;
     int max_seqs;
     unsigned char* scratch;
+    int* error;
 };
 
 __device__ __forceinline__ float4 unpack4(uint2 v) {
@@ -95,28 +96,17 @@ struct ConvSource {
     const float* hist;
     int pitch, stride, count, channels, padded;     // channels exist in hist, padded ones in raw
 };
-// Rows tok0 - 3 .. tok0 + 63 of 8 << shift channels -> shared memory, 16 << shift bytes per row, by n threads; zeros outside the sequence.
-__device__ __forceinline__ void stage_raw(uint32_t dst, unsigned char* dst_ptr, const ConvSource& c, int shift, int taps, int tok0, int tid, int n) {
-    for (int i = tid; i < 67 << shift; i += n) {
-        const int t = tok0 - 3 + (i >> shift), ch = 8 * (i & ((1 << shift) - 1));
-        const bool in = ch < c.padded;
-        if (t >= 0 || !in) {
-            const bool get = in && t < c.count;
-            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + i * 16), "l"(c.raw + (get ? (size_t)t * c.pitch + ch : 0)), "r"(get ? 16 : 0)
-                         : "memory");
-        } else {
-            float x[8];
-#pragma unroll
-            for (int e = 0; e < 8; ++e) x[e] = (taps - 1 + t >= 0 && ch + e < c.channels) ? c.hist[(size_t)(taps - 1 + t) * c.stride + ch + e] : 0.f;
-            *reinterpret_cast<uint4*>(dst_ptr + i * 16) = make_uint4(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]), pack_bf16x2(x[4], x[5]), pack_bf16x2(x[6], x[7]));
-        }
+// Three rows in front of a pass's first chunk, over what a tile's load brought there: the inputs kept from before, zeros ahead of them.
+__device__ __forceinline__ void put_history(unsigned char* tile, int row_bytes, const ConvSource& c, int taps, int tid, int n) {
+    for (int i = tid; i < 3 * (row_bytes / 2); i += n) {
+        const int r = i / (row_bytes / 2), ch = i % (row_bytes / 2), t = taps - 1 - 3 + r;
+        reinterpret_cast<__nv_bfloat16*>(tile)[i] = __float2bfloat16_rn(t >= 0 && ch < c.channels ? c.hist[(size_t)t * c.stride + ch] : 0.f);
     }
 }
-__device__ __forceinline__ void staged() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
 // Four consecutive tokens x four channels behind a short convolution and silu.  Tokens behind the sequence's end get finite values
 // that meet a beta of zero.
-// TAPS 4: from staged rows (the tokens are rows t .. t + 3 of the chunk), w [4][w_pitch] with leading zeros for fewer taps.
+// TAPS 4: from a tile of rows tok0 - 3 .. tok0 + 63 (by TMA; the tokens are rows t + 3 .. t + 6), w [4][w_pitch] with leading zeros for fewer taps.
 // TAPS 0: any number of taps, from global memory, w [channel][taps].
 template <int TAPS>
 __device__ __forceinline__ void conv_piece(const unsigned char* tile, int row_bytes, const ConvSource& c, int ch, const float* w, int w_pitch, int taps, int tok0,
@@ -176,7 +166,8 @@ constexpr uint32_t kOffAM = kOffCOL + 26112;           // A, fp32 [64][kLd], the
 constexpr uint32_t kOffM = kOffAM + 17408;             // image of M
 constexpr uint32_t kOffG = kOffM + kTile;              // [17][64 ND] log2 decays up to the start of every group
 constexpr uint32_t kOffB = kOffG + 17 * 128 * 4;       // beta [64]
-constexpr uint32_t kPrepSmem = kOffB + 256;
+constexpr uint32_t kOffPBar = kOffB + 256;             // loads of q and k, of v; give-up flag
+constexpr uint32_t kPrepSmem = kOffPBar + 64;
 __device__ __forceinline__ void sync_half(int which) { asm volatile("bar.sync %0, 256;" ::"r"(1 + which) : "memory"); }
 }  // namespace
 
@@ -184,7 +175,7 @@ __device__ __forceinline__ void sync_half(int which) { asm volatile("bar.sync %0
 // more than 64 channels a group of tokens is a warp's.
 template <int ND, int TAPS>
 __global__ void __launch_bounds__(kPrepThreads, 2)
-delta_prep_kernel(const DeltaChunkArgs A) {
+delta_prep_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const DeltaChunkArgs A) {
     extern __shared__ __align__(128) unsigned char sm[];
     constexpr int DK = 64 * ND, LN = 16 * ND, kP = DK + 8;         // channels, lanes per token, row pitch in halves
     const DeltaShape& sh = A.sh;
@@ -203,9 +194,17 @@ delta_prep_kernel(const DeltaChunkArgs A) {
     const float* hist = st + (size_t)sh.dim * sh.vt;
     const ConvSource cq{rows + kvh * sh.dp, hist, sh.off_b(), D4, sq.count, sh.dim, sh.dp};
     const ConvSource ck{rows + sh.off_k() + kvh * sh.dp, hist + (taps - 1) * D4, sh.off_b(), D4, sq.count, sh.dim, sh.dp};
-    if constexpr (TAPS > 0) {
-        stage_raw(base + kOffKA, sm + kOffKA, cq, ND + 2, taps, tok0, tid, kPrepThreads);
-        stage_raw(base + kOffQA, sm + kOffQA, ck, ND + 2, taps, tok0, tid, kPrepThreads);
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(sm + kOffPBar + 16);
+    auto bar = [&](int i) { return base + kOffPBar + 8u * i; };
+    if (TAPS > 0 && tid == 0) {
+        mbar_init(bar(0), 1);
+        mbar_init(bar(1), 1);
+        *abort_flag = 0;
+        mbar_fence_init();
+        fence_proxy_async_smem();
+        mbar_arrive_expect_tx(bar(0), 2 * 67 * DK * 2);
+        tma_load_2d(base + kOffKA, &map_k, bar(0), kvh * sh.dp, sq.row0 + tok0 - 3);
+        tma_load_2d(base + kOffQA, &map_k, bar(0), sh.off_k() + kvh * sh.dp, sq.row0 + tok0 - 3);
     }
     const int tg = tid / LN, c4 = tid % LN, ch = 4 * c4, t0 = 4 * tg;
     const bool act = tg < 16, in = act && ch < sh.dp;               // act: whole warps
@@ -226,9 +225,14 @@ delta_prep_kernel(const DeltaChunkArgs A) {
         qh[i][0] = qh[i][1] = kh[i][0] = kh[i][1] = 0u;
         g[i][0] = g[i][1] = g[i][2] = g[i][3] = 1.f;
     }
+    __syncthreads();
     if constexpr (TAPS > 0) {
-        staged();
-        __syncthreads();
+        mbar_wait(bar(0), 0, abort_flag);
+        if (chunk == 0) {
+            put_history(sm + kOffKA, 8 * LN, cq, taps, tid, kPrepThreads);
+            put_history(sm + kOffQA, 8 * LN, ck, taps, tid, kPrepThreads);
+            __syncthreads();
+        }
     }
     if (act) {
 #pragma unroll
@@ -428,16 +432,23 @@ delta_prep_kernel(const DeltaChunkArgs A) {
         put2(q, 16 * I + g4, 8 * n + 2 * t4, d[0], d[1]);
         put2(q, 16 * I + g4 + 8, 8 * n + 2 * t4, d[2], d[3]);
     }
+    fence_proxy_async_smem();
     __syncthreads();
     const int nv = A.item.nv, kVP = 64 * nv + 8;                    // row pitch of V
-    auto load_values = [&](int tile, int vt, int n, int which) {    // the values of a state tile, staged over the queries, go to KB; threads vt of n, half `which`
+    auto fetch_values = [&](int tile) {                             // one thread: the inputs of a state tile's values, over the queries
+        mbar_arrive_expect_tx(bar(1), 67 * 128 * nv);
+        tma_load_2d(base + kOffQA, &map_v, bar(1), sh.off_v() + h * sh.vp + tile * kMlstmTile, sq.row0 + tok0 - 3);
+    };
+    auto load_values = [&](int tile, int vt, int n, int which) {    // .. behind their convolution to KB; threads vt of n (which >= 0: half `which` of the CTA)
         const float* hv = hist + tile * sh.tile_floats() + 2 * (taps - 1) * D4;
         const int c0 = tile * kMlstmTile, left_v = sh.vp - c0;
         const ConvSource c{rows + sh.off_v() + h * sh.vp + c0, hv, sh.off_b(), sh.vt, sq.count, sh.vdim - c0, left_v};
         if constexpr (TAPS > 0) {
-            stage_raw(base + kOffQA, sm + kOffQA, c, nv + 2, taps, tok0, vt, n);
-            staged();
-            if (which < 0) __syncthreads(); else sync_half(which);
+            mbar_wait(bar(1), tile & 1, abort_flag);
+            if (chunk == 0) {
+                put_history(sm + kOffQA, 128 * nv, c, taps, vt, n);
+                if (which < 0) __syncthreads(); else sync_half(which);
+            }
         }
         for (int i = vt; i < 256 * nv; i += n) {
             const int t = 4 * (i >> (nv + 3)), vc = 4 * (i & (16 * nv - 1));
@@ -459,7 +470,11 @@ delta_prep_kernel(const DeltaChunkArgs A) {
         sync_half(0);
         solve_columns(AM, TF, warp, lane);
     } else {          // ---- meanwhile M goes out and the first values come in ----
-        for (int i = tid - 256; i < (int)kTile / 16; i += 256) reinterpret_cast<uint4*>(item + 3 * ND * kTile)[i] = reinterpret_cast<uint4*>(sm + kOffM)[i];
+        if (tid == 256) {
+            if constexpr (TAPS > 0) fetch_values(0);
+            bulk_s2g(item + 3 * ND * kTile, base + kOffM, kTile);
+            bulk_commit_group();
+        }
         load_values(0, tid - 256, 256, 1);
     }
     if (act) {        // the keys decay from the chunk's start
@@ -502,8 +517,12 @@ delta_prep_kernel(const DeltaChunkArgs A) {
             *reinterpret_cast<uint32_t*>(w + sw(16 * i + g4 + 8, (c >> 3) & 7) + 4 * t4) = pack_half2(d[n][2], d[n][3]);
         }
     }
+    fence_proxy_async_smem();
     __syncthreads();
-    for (int i = tid; i < (int)(ND * kTile) / 16; i += kPrepThreads) reinterpret_cast<uint4*>(item)[i] = reinterpret_cast<uint4*>(sm + kOffQA)[i];
+    if (tid == 0) {
+        bulk_s2g(item, base + kOffQA, ND * kTile);
+        bulk_commit_group();
+    }
     // ---- U'^T = V^T (T diag(beta))^T of every state tile: 16 values x every second (fourth) token tile per warp ----
     for (int tile = 0;; ++tile) {
         const int mt = warp & (4 * nv - 1), part = warp >> (nv + 1), parts = 4 / nv;
@@ -524,13 +543,22 @@ delta_prep_kernel(const DeltaChunkArgs A) {
             *reinterpret_cast<uint32_t*>(sm + kOffKA + sw(16 * mt + g4, n) + 4 * t4) = pack_half2(d[0], d[1]);
             *reinterpret_cast<uint32_t*>(sm + kOffKA + sw(16 * mt + g4 + 8, n) + 4 * t4) = pack_half2(d[2], d[3]);
         }
+        fence_proxy_async_smem();
         __syncthreads();
-        uint4* dst = reinterpret_cast<uint4*>(item + A.item.off_u() + tile * nv * kTile);
-        for (int i = tid; i < (int)(nv * kTile) / 16; i += kPrepThreads) dst[i] = reinterpret_cast<uint4*>(sm + kOffKA)[i];
+        if (tid == 0) {
+            bulk_s2g(item + A.item.off_u() + tile * nv * kTile, base + kOffKA, nv * kTile);
+            bulk_commit_group();
+        }
         if (tile + 1 == sh.n_vt) break;
+        if (tid == 0) {                // W and this tile's U' have left their places
+            bulk_wait_group_read0();
+            if constexpr (TAPS > 0) fetch_values(tile + 1);
+        }
         load_values(tile + 1, tid, kPrepThreads, -1);
         __syncthreads();
     }
+    if (tid == 0 || tid == 256) bulk_wait_group0();
+    if (TAPS > 0 && tid == 0 && *abort_flag) atomicExch(A.error, 11);
 }
 
 // ---- the walk over a sequence's chunks -----------------------------------------------------------------------------------------------
@@ -773,12 +801,12 @@ delta_walk_kernel(const DeltaShape sh, const DeltaItem it, const __nv_bfloat16* 
 
 static DeltaItem delta_item(const DeltaShape& sh) { return DeltaItem{ceil_div(sh.dim, 64), sh.vt > 64 ? 2 : 1, sh.n_vt}; }
 
-bool delta_chunk_fits(const DeltaShape& sh) { return sh.dim <= 128; }
+bool delta_chunk_fits(const DeltaShape& sh) { return sh.dim <= 128 && sh.off_b() >= 128; }     // the loads' boxes are up to 128 columns wide
 
 size_t delta_chunk_bytes(const DeltaShape& sh) { return (size_t)sh.heads * delta_item(sh).bytes(); }
 
 int launch_delta_chunk(const DeltaShape& sh, const void* qkv, const float* a, const float* b, const float* conv, const float* a_log, const float* dt_bias,
-                       const LaSeqMeta* d_seqs, int n_seqs, int max_count, int max_seqs, float* state, void* scratch, float* core, int* d_error,
+                       const LaSeqMeta* d_seqs, int n_seqs, int max_count, int rows, int max_seqs, float* state, void* scratch, float* core, int* d_error,
                        cudaStream_t s) {
     const DeltaItem it = delta_item(sh);
     static PerDeviceOnce once;
@@ -787,9 +815,18 @@ int launch_delta_chunk(const DeltaShape& sh, const void* qkv, const float* a, co
             B2_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, kPrepSmem));
         for (auto k : {delta_walk_kernel<1, 1>, delta_walk_kernel<1, 2>, delta_walk_kernel<2, 1>, delta_walk_kernel<2, 2>})
             B2_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, kWalkSmem)));
-    DeltaChunkArgs A{sh, it, (const __nv_bfloat16*)qkv, a, b, conv, a_log, dt_bias, state, d_seqs, max_seqs, (unsigned char*)scratch};
+    const DeltaChunkArgs A{sh, it, (const __nv_bfloat16*)qkv, a, b, conv, a_log, dt_bias, state, d_seqs, max_seqs, (unsigned char*)scratch, d_error};
+    CUtensorMap mk, mv;
+    auto map = [&](CUtensorMap* m, int cols) -> int {          // 67 rows: a chunk and three in front of it
+        const uint64_t dims[2] = {(uint64_t)sh.off_b(), (uint64_t)rows};
+        const uint64_t str[1] = {(uint64_t)sh.off_b() * 2};
+        const uint32_t box[2] = {(uint32_t)cols, 67};
+        return make_tensor_map(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, qkv, dims, str, box, false);
+    };
+    B2_TRY(map(&mk, 64 * it.nd));
+    B2_TRY(map(&mv, 64 * it.nv));
     const dim3 gp(sh.heads, ceil_div(max_count, kDC), n_seqs);
-    auto prep = [&](auto kernel) { kernel<<<gp, kPrepThreads, kPrepSmem, s>>>(A); };
+    auto prep = [&](auto kernel) { kernel<<<gp, kPrepThreads, kPrepSmem, s>>>(mk, mv, A); };
     if (it.nd == 2) { if (sh.taps <= 4) prep(delta_prep_kernel<2, 4>); else prep(delta_prep_kernel<2, 0>); }
     else { if (sh.taps <= 4) prep(delta_prep_kernel<1, 4>); else prep(delta_prep_kernel<1, 0>); }
     B2_LAUNCH_CHECK();

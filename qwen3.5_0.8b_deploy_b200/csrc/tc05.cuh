@@ -135,9 +135,9 @@ __device__ __forceinline__ void tma_prefetch_desc(const CUtensorMap* map) {
 }
 
 // ---- host: tensor maps ----------------------------------------------------------------------------------------------
-// Encodes a tiled map with 128-byte swizzle and zero fill. dims/strides innermost first; strides in bytes
+// Encodes a tiled map with 128-byte swizzle (or none) and zero fill. dims/strides innermost first; strides in bytes
 // for dims 1..rank-1.  Returns 0 or a negative status with the error text set.
 int make_tensor_map(CUtensorMap* out, CUtensorMapDataType dtype, int rank, const void* base, const uint64_t* dims,
-                    const uint64_t* strides_bytes, const uint32_t* box);
+                    const uint64_t* strides_bytes, const uint32_t* box, bool swizzle = true);
 
 }  // namespace b200
