@@ -178,7 +178,7 @@ int delta_forward(BlockModel& m, DeltaOp& op, const LayerRun& run, const PassRow
     }
     B2_TRY(gemm_typed(s, m.xt.p, W, op.w_in.p, m.proj.p, sh.pitch(), op.elem, ELEM_F32, p.rows, sh.pitch(), W));
     B2_TRY(gemm_typed(s, m.low.p, sh.low(), op.w_gate.p, m.gates.p, sh.gate_cols(), op.elem, ELEM_F32, p.rows, sh.gate_cols(), sh.low()));
-    DeltaStepArgs a{sh, m.proj.f(), m.gates.f(), op.conv.f(), op.a_log.f(), op.dt_bias.f(), op.norm_w.f(), state, p.decode ? p.d_slots : nullptr,
+    DeltaStepArgs a{sh, m.proj.f(), m.gates.f(), op.conv.f(), sh.taps <= 4 ? op.conv4.f() : nullptr, op.a_log.f(), op.dt_bias.f(), op.norm_w.f(), state, p.decode ? p.d_slots : nullptr,
                     p.decode ? nullptr : p.d_seqs, m.cfg.max_seqs, m.core.f(), m.mixed.p};
     B2_TRY(launch_delta_step(op.elem, a, p.n_seqs, s));
     if (sh.n_vt > 1)

@@ -200,6 +200,7 @@ struct DeltaStepArgs {                 // the token-serial kernel: decode (one t
     const float* proj;                 // [rows][pitch]
     const float* gates;                // [rows][gate_cols]
     const float* conv;                 // [off_b][taps]
+    const float* conv4;                // [4][off_b] with leading zeros; null with more than four taps
     const float* a_log;                // [heads]
     const float* dt_bias;              // [heads * dp]
     const float* norm_w;               // [vdim]

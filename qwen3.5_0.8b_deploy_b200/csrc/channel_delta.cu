@@ -17,8 +17,10 @@ namespace b200 {
 // grid (sequences, heads, tiles), block 256.  Lane l of every warp owns value columns 4l .. 4l + 3 of the tile, warp w the key
 // rows w, w + 8, ...; with dim <= 8 NR a thread's part of the state stays in registers over the whole run of tokens (decode: one
 // token), else it is streamed through for every token.  Decode loads its state ahead of the wait on the preceding kernel.
-template <int NR, typename T, bool kFuseNorm>
-__global__ void __launch_bounds__(256)
+// kSmall (up to 128 key channels and four taps): threads 0 .. 127 hold the q and k channels with their inputs and weights in
+// registers, the others the values', and everything a token needs is requested before the first use; else they are in shared memory.
+template <int NR, typename T, bool kSmall, bool kFuseNorm>
+__global__ void __launch_bounds__(256, NR <= 16 ? 2 : 1)
 delta_step_kernel(const DeltaStepArgs a, unsigned long long* stamp) {
     extern __shared__ float sm[];
     const DeltaShape& sh = a.sh;
@@ -52,8 +54,34 @@ delta_step_kernel(const DeltaStepArgs a, unsigned long long* stamp) {
             if (d < D) st[i] = __ldcs(reinterpret_cast<const float4*>(S + (size_t)d * sh.vt + c0));
         }
     }
-    for (int i = tid; i < hist_n; i += 256) s_hist[i] = hist[i];
     const int kvh = h / (sh.heads / sh.kv_heads), v0 = h * sh.vp + tile * kMlstmTile;
+    // kSmall: this thread's channels (key channel d, or value column c of the tile), their last three inputs and four weights
+    const bool keys = tid < 128;
+    const int own = keys ? tid : tid - 128, n_own = keys ? D : min(sh.vt, sh.vdim - tile * kMlstmTile);
+    const bool mine_in = own < n_own;
+    const int col0 = keys ? kvh * sh.dp + own : sh.off_v() + v0 + own, col1 = sh.off_k() + kvh * sh.dp + own;
+    float h0[3] = {0.f, 0.f, 0.f}, h1[3] = {0.f, 0.f, 0.f}, w0[4] = {0.f, 0.f, 0.f, 0.f}, w1[4] = {0.f, 0.f, 0.f, 0.f}, dt = 0.f;
+    if constexpr (kSmall) {
+        if (mine_in) {
+            const float* hs = hist + (keys ? own : 2 * (taps - 1) * D4 + own);
+            const int step = keys ? D4 : sh.vt;
+#pragma unroll
+            for (int j = 0; j < 3; ++j) {
+                const int i = j - (4 - taps);
+                if (i < 0) continue;
+                h0[j] = hs[i * step];
+                if (keys) h1[j] = hs[((taps - 1) + i) * D4];
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                w0[j] = a.conv4[j * sh.off_b() + col0];
+                if (keys) w1[j] = a.conv4[j * sh.off_b() + col1];
+            }
+            if (keys) dt = a.dt_bias[h * sh.dp + own];
+        }
+    } else {
+        for (int i = tid; i < hist_n; i += 256) s_hist[i] = hist[i];
+    }
     const float ea = expf(a.a_log[h]), qn = 1.0f / sqrtf((float)D);
     pdl_enter();
     stamp_begin(stamp);
@@ -67,12 +95,34 @@ delta_step_kernel(const DeltaStepArgs a, unsigned long long* stamp) {
         }
         return times_sigmoid<float>(acc, acc);
     };
-    __syncthreads();
+    auto conv4 = [](float x, float (&hs)[3], const float (&w)[4]) {
+        const float acc = hs[0] * w[0] + hs[1] * w[1] + hs[2] * w[2] + x * w[3];
+        hs[0] = hs[1]; hs[1] = hs[2]; hs[2] = x;
+        return times_sigmoid<float>(acc, acc);
+    };
+    if constexpr (!kSmall) __syncthreads();
     for (int t = 0; t < count; ++t) {
         const size_t row = row0 + t;
         const float* pr = a.proj + row * sh.pitch();
         const float* gt = a.gates + row * sh.gate_cols();
         float ssq = 0.f, ssk = 0.f;
+        const float braw = pr[sh.off_b() + h];
+        if constexpr (kSmall) {
+            const float x0 = mine_in ? pr[col0] : 0.f, x1 = mine_in && keys ? pr[col1] : 0.f, z = mine_in && keys ? gt[h * sh.dp + own] : 0.f;
+            const float y0 = conv4(x0, h0, w0);
+            if (keys) {
+                const float y1 = conv4(x1, h1, w1);
+                if (mine_in) {
+                    s_q[own] = y0;
+                    s_k[own] = y1;
+                    s_g[own] = expf(-ea * delta_softplus(z + dt));
+                }
+                ssq = y0 * y0;
+                ssk = y1 * y1;
+            } else if (own < sh.vt) {
+                s_v[own] = y0;
+            }
+        } else {
         for (int d = tid; d < D; d += 256) {
             const int cq = kvh * sh.dp + d, ck = sh.off_k() + cq;
             const float z = gt[h * sh.dp + d] + a.dt_bias[h * sh.dp + d];
@@ -88,7 +138,8 @@ delta_step_kernel(const DeltaStepArgs a, unsigned long long* stamp) {
             const int cv = sh.off_v() + v0 + c;
             s_v[c] = tile * kMlstmTile + c < sh.vdim ? conv(pr[cv], a.conv + (size_t)cv * taps, s_hist + 2 * (taps - 1) * D4 + c, sh.vt) : 0.f;
         }
-        const float beta = 1.0f / (1.0f + expf(-pr[sh.off_b() + h]));
+        }
+        const float beta = 1.0f / (1.0f + expf(-braw));
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) {
             ssq += __shfl_xor_sync(0xffffffffu, ssq, o);
@@ -190,8 +241,23 @@ delta_step_kernel(const DeltaStepArgs a, unsigned long long* stamp) {
             if (d < D) __stcs(reinterpret_cast<float4*>(S + (size_t)d * sh.vt + c0), st[i]);
         }
     }
-    __syncthreads();
-    for (int i = tid; i < hist_n; i += 256) hist[i] = s_hist[i];
+    if constexpr (kSmall) {
+        if (mine_in) {
+            float* hs = hist + (keys ? own : 2 * (taps - 1) * D4 + own);
+            const int step = keys ? D4 : sh.vt;
+#pragma unroll
+            for (int j = 0; j < 3; ++j) {
+                const int i = j - (4 - taps);
+                if (i < 0) continue;
+                hs[i * step] = h0[j];
+                if (keys) hs[((taps - 1) + i) * D4] = h1[j];
+            }
+        }
+        if (stamp) __syncthreads();
+    } else {
+        __syncthreads();
+        for (int i = tid; i < hist_n; i += 256) hist[i] = s_hist[i];
+    }
     if (stamp) stamp_end(stamp);
 }
 
@@ -210,10 +276,10 @@ int launch_delta_step(ElemType t, const DeltaStepArgs& a, int n, cudaStream_t s)
         };
         auto pick = [&](auto fuse) -> int {
             constexpr bool kFuse = decltype(fuse)::value;
-            if (sh.dim <= 32) return go(delta_step_kernel<4, T, kFuse>);
-            if (sh.dim <= 64) return go(delta_step_kernel<8, T, kFuse>);
-            if (sh.dim <= 128) return go(delta_step_kernel<16, T, kFuse>);
-            return go(delta_step_kernel<32, T, kFuse>);
+            if (sh.dim > 128 || !a.conv4) return sh.dim <= 128 ? go(delta_step_kernel<16, T, false, kFuse>) : go(delta_step_kernel<32, T, false, kFuse>);
+            if (sh.dim <= 32) return go(delta_step_kernel<4, T, true, kFuse>);
+            if (sh.dim <= 64) return go(delta_step_kernel<8, T, true, kFuse>);
+            return go(delta_step_kernel<16, T, true, kFuse>);
         };
         rc = sh.n_vt == 1 ? pick(std::true_type{}) : pick(std::false_type{});
     });

@@ -92,8 +92,80 @@ diff_pre_kernel(const DiffPreArgs a) {
     }
 }
 
+// The same for vectors of 4 LPV (64 or 128) columns: LPV lanes per vector, and the loads of all of a warp's first kU rounds of
+// vectors are under way before the first use.
+template <typename T, int LPV>
+__global__ void __launch_bounds__(256)
+diff_pre_vec_kernel(const DiffPreArgs a) {
+    constexpr int kU = 4, kPer = 8 * (32 / LPV);                // vectors per round of a block
+    pdl_enter();
+    const DiffShape& sh = a.sh;
+    const int row = blockIdx.x, slot = a.row_slot[row], pos = a.row_pos[row];
+    if (slot < 0 || slot >= a.cache.max_seqs) return;
+    const int H = sh.heads, G = sh.kv_heads, dp = 4 * LPV, hp = sh.hp(), half = sh.rot / 2, per = H / G, n = 2 * (H + G);
+    const int first = threadIdx.x / LPV, lane = threadIdx.x % LPV, c = 4 * lane;
+    const float* pr = a.proj + (size_t)row * sh.pitch();
+    float4 x[kU];
+    auto fetch = [&](int v0) {
+#pragma unroll
+        for (int i = 0; i < kU; ++i) {
+            const int v = v0 + i * kPer;                        // queries and keys lie behind one another
+            x[i] = v < n ? __ldcs(reinterpret_cast<const float4*>(pr + v * dp + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    };
+    fetch(first);
+    const float4 wq = load4(a.q_norm + c), wk = load4(a.k_norm + c);     // [dp], zero behind dim
+    const float2* cs = a.cs + (size_t)row * half;
+    const float2 one = make_float2(1.f, 0.f), t0 = 2 * lane < half ? cs[2 * lane] : one, t1 = 2 * lane + 1 < half ? cs[2 * lane + 1] : one;
+    const bool fits = pos < a.cache.capacity[slot];
+    if (!fits && threadIdx.x == 0) atomicExch(a.cache.error, 2);         // page not reserved: skip the write
+    T* page = nullptr;
+    if (fits)
+        page = static_cast<T*>(a.cache.rows) + (size_t)a.cache.block_table[slot * a.cache.max_pages_per_seq + pos / kPageTokens] * kPageTokens * sh.row_pitch() +
+               (size_t)(pos % kPageTokens) * hp;
+    for (int i = threadIdx.x; fits && i < G * sh.vp / 4; i += 256) {     // values
+        const int g = 4 * i / sh.vp, cv = 4 * i % sh.vp;
+        store4(page + (size_t)g * kPageTokens * hp + 2 * dp + cv, __ldcs(reinterpret_cast<const float4*>(pr + sh.off_v() + 4 * i)));
+    }
+    if (fits && threadIdx.x < 8 * G) page[(size_t)(threadIdx.x >> 3) * kPageTokens * hp + 2 * dp + sh.vp + (threadIdx.x & 7)] = from_f32<T>(0.f);
+    for (int v0 = first; v0 - first < n; v0 += kU * kPer) {              // the same number of rounds in every lane
+        if (v0 != first) fetch(v0);
+        float ss[kU];
+#pragma unroll
+        for (int i = 0; i < kU; ++i) ss[i] = (x[i].x * x[i].x + x[i].y * x[i].y) + (x[i].z * x[i].z + x[i].w * x[i].w);
+#pragma unroll
+        for (int o = LPV / 2; o > 0; o >>= 1)
+#pragma unroll
+            for (int i = 0; i < kU; ++i) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], o);
+#pragma unroll
+        for (int i = 0; i < kU; ++i) {
+            const int v = v0 + i * kPer;
+            if (v >= n) break;
+            const float inv = 1.0f / sqrtf(ss[i] / (float)sh.dim + sh.eps);
+            const float4 w = v < 2 * H ? wq : wk;
+            const float4 y = make_float4(x[i].x * inv * w.x, x[i].y * inv * w.y, x[i].z * inv * w.z, x[i].w * inv * w.w);
+            const float4 r = make_float4(y.x * t0.x - y.y * t0.y, y.y * t0.x + y.x * t0.y, y.z * t1.x - y.w * t1.y, y.w * t1.x + y.z * t1.y);
+            const int hh = v >> 1, map = v & 1;
+            if (v >= 2 * H) {
+                if (fits) store4(page + (size_t)(hh - H) * kPageTokens * hp + map * dp + c, r);
+            } else if (a.qd) {
+                const int qp = sh.qp();
+                T* dst = static_cast<T*>(a.qd) + (((size_t)row * G + hh / per) * 16 + 8 * map + hh % per) * qp;
+                store4(dst + map * dp + c, r);
+                store4(dst + (1 - map) * dp + c, make_float4(0.f, 0.f, 0.f, 0.f));
+                if (lane < 2) store4(dst + 2 * dp + c, make_float4(0.f, 0.f, 0.f, 0.f));
+            } else {
+                store4(static_cast<T*>(a.q) + ((size_t)row * H * 2 + v) * dp + c, r);
+            }
+        }
+    }
+}
+
 int launch_diff_pre(ElemType t, const DiffPreArgs& a, int rows, cudaStream_t s) {
-    dispatch_elem(t, [&](auto tag) { launch_pdl(diff_pre_kernel<decltype(tag)>, dim3(rows), dim3(256), 0, s, a); });
+    dispatch_elem(t, [&](auto tag) {
+        using T = decltype(tag);
+        launch_pdl(a.sh.dp == 64 ? diff_pre_vec_kernel<T, 16> : a.sh.dp == 128 ? diff_pre_vec_kernel<T, 32> : diff_pre_kernel<T>, dim3(rows), dim3(256), 0, s, a);
+    });
     B2_LAUNCH_CHECK();
     return 0;
 }
