@@ -91,7 +91,7 @@ def gutenex_layers(config: dict, shapes: dict, ops) -> list:
             d.a_rank, d.g_rank = (shapes[f"l{i}.mix.{n}"][0] for n in ("a1", "g1"))
         elif layer["type"] == "attention":
             d.mixer, d.kv_heads, d.scale, d.diff = ops.MIXER_DIFF, m["kv_heads"], m["scale"], m["diff"]
-            d.window, d.keep_first = m["mask"]["size"], m["mask"]["keep_first"]
+            d.window, d.keep_first = m["mask"].get("size") or 0, m["mask"].get("keep_first") or 0
             d.rot_dim, d.rot_base = m["rot"]["dims"], m["rot"]["base"]
         else:
             raise ValueError(f"layer {i}: unknown type {layer['type']!r}")
