@@ -14,7 +14,6 @@
 // Operands are fp16: unit vectors, decays, beta and T are at most 1, and 11 bits are kept of values.
 #include "block_model.cuh"
 #include "channel_delta.cuh"
-#include "delta_inverse.cuh"
 #include "elem.cuh"
 #include "tc05.cuh"
 
@@ -161,13 +160,75 @@ constexpr uint32_t kRegion = 17408;                    // 64 rows of 136 halves
 constexpr uint32_t kOffKA = 0;                         // staged q, decayed keys (rows), e^G K, then the image of U'
 constexpr uint32_t kOffQA = kRegion;                   // staged k, decayed queries (rows), staged v, then the image of W
 constexpr uint32_t kOffKB = 2 * kRegion;               // keys decayed to the end of their group, then V
-constexpr uint32_t kOffCOL = 3 * kRegion;              // 96 rows of decayed keys (columns), then T
-constexpr uint32_t kOffAM = kOffCOL + 26112;           // A, fp32 [64][kLd], then T diag(beta) in fp16
-constexpr uint32_t kOffM = kOffAM + 17408;             // image of M
+constexpr uint32_t kOffCOL = 3 * kRegion;              // 96 rows of decayed keys (columns), then T diag(beta), a swizzled fp16 tile
+constexpr uint32_t kOffAD = kOffCOL + 26112;           // A's diagonal blocks, fp32 [64][kAdP]
+constexpr int kAdP = 20;
+constexpr uint32_t kOffAT = kOffAD + 64 * kAdP * 4;    // A below them, a swizzled fp16 tile
+constexpr uint32_t kOffD = kOffAT + kTile;             // the diagonal blocks' inverses, fp16 [64] rows 48 bytes apart
+constexpr uint32_t kOffM = kOffD + 64 * 48;            // image of M
 constexpr uint32_t kOffG = kOffM + kTile;              // [17][64 ND] log2 decays up to the start of every group
 constexpr uint32_t kOffB = kOffG + 17 * 128 * 4;       // beta [64]
 constexpr uint32_t kOffPBar = kOffB + 256;             // loads of q and k, of v; give-up flag
 constexpr uint32_t kPrepSmem = kOffPBar + 64;
+// T = (I + A)^-1 in blocks of 16.  Threads 0 .. 63 invert the diagonal blocks D_I, a column each by forward substitution in fp32.
+__device__ __forceinline__ void invert_blocks(unsigned char* sm, const float* s_beta, int tid) {
+    const float* AD = reinterpret_cast<const float*>(sm + kOffAD);
+    const int b0 = tid & ~15, col = tid & 15;
+    float t[16];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) t[i] = i == col ? 1.f : 0.f;
+#pragma unroll
+    for (int i = 1; i < 16; ++i) {
+        float acc0 = 0.f, acc1 = 0.f;
+#pragma unroll
+        for (int j = 0; j < i; j += 4) {
+            const float4 a = load4(AD + (b0 + i) * kAdP + j);                 // entries at and above the diagonal are zero
+            acc0 += a.x * t[j] + a.z * t[j + 2];
+            acc1 += a.y * t[j + 1] + a.w * t[j + 3];
+        }
+        t[i] -= acc0 + acc1;
+    }
+    const float beta = s_beta[tid];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+        *reinterpret_cast<__half*>(sm + kOffD + (b0 + i) * 48 + col * 2) = __float2half_rn(t[i]);
+        *reinterpret_cast<__half*>(sm + kOffCOL + sw(b0 + i, tid >> 3) + 2 * (tid & 7)) = __float2half_rn(t[i] * beta);
+    }
+}
+// A warp per block column J: T_IJ^T = -(sum_K T_KJ^T A_IK^T) D_I^T from top to bottom; a product's accumulators are the next one's A operand.
+template <int J>
+__device__ __forceinline__ void solve_block_column(unsigned char* sm, uint32_t base, const float* s_beta, int lane) {
+    const int g4 = lane >> 2, t4 = lane & 3, r8 = (lane & 7) + ((lane >> 4) & 1) * 8, k8 = (lane >> 3) & 1;
+    uint32_t y[4][4];
+    ldm4t(y[J], base + kOffD + (16 * J + r8) * 48 + k8 * 16);
+    const float b0 = -s_beta[16 * J + g4], b1 = -s_beta[16 * J + g4 + 8];
+#pragma unroll
+    for (int I = J + 1; I < 4; ++I) {
+        float z[2][4] = {}, d[2][4] = {};
+        uint32_t b[4];
+#pragma unroll
+        for (int K = J; K < I; ++K) {
+            ldm4(b, base + kOffAT + sw(16 * I + r8, 2 * K + k8));
+            mma_16816(z[0], y[K][0], y[K][1], y[K][2], y[K][3], b[0], b[1]);
+            mma_16816(z[1], y[K][0], y[K][1], y[K][2], y[K][3], b[2], b[3]);
+        }
+        const uint32_t a0 = pack_half2(z[0][0], z[0][1]), a1 = pack_half2(z[0][2], z[0][3]), a2 = pack_half2(z[1][0], z[1][1]), a3 = pack_half2(z[1][2], z[1][3]);
+        ldm4(b, base + kOffD + (16 * I + r8) * 48 + k8 * 16);
+        mma_16816(d[0], a0, a1, a2, a3, b[0], b[1]);
+        mma_16816(d[1], a0, a1, a2, a3, b[2], b[3]);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+            y[I][2 * j] = pack_half2(-d[j][0], -d[j][1]);
+            y[I][2 * j + 1] = pack_half2(-d[j][2], -d[j][3]);
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int t = 16 * I + 8 * j + 2 * t4 + e;
+                *reinterpret_cast<__half*>(sm + kOffCOL + sw(t, 2 * J) + 2 * g4) = __float2half_rn(d[j][e] * b0);
+                *reinterpret_cast<__half*>(sm + kOffCOL + sw(t, 2 * J + 1) + 2 * g4) = __float2half_rn(d[j][2 + e] * b1);
+            }
+        }
+    }
+}
 __device__ __forceinline__ void sync_half(int which) { asm volatile("bar.sync %0, 256;" ::"r"(1 + which) : "memory"); }
 }  // namespace
 
@@ -183,8 +244,7 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
     const int h = blockIdx.x, chunk = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
     if (chunk * kDC >= sq.count || sq.slot < 0 || sq.slot >= A.max_seqs) return;
     const uint32_t base = smem_u32(sm);
-    float* AM = reinterpret_cast<float*>(sm + kOffAM);
-    float* TF = reinterpret_cast<float*>(sm + kOffCOL);
+    float* AD = reinterpret_cast<float*>(sm + kOffAD);
     float* s_g = reinterpret_cast<float*>(sm + kOffG);
     float* s_beta = reinterpret_cast<float*>(sm + kOffB);
     unsigned char* item = A.scratch + ((first_chunk(sq.row0, blockIdx.z) + chunk) * sh.heads + h) * A.item.bytes();
@@ -196,7 +256,7 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
     const ConvSource ck{rows + sh.off_k() + kvh * sh.dp, hist + (taps - 1) * D4, sh.off_b(), D4, sq.count, sh.dim, sh.dp};
     volatile int* abort_flag = reinterpret_cast<volatile int*>(sm + kOffPBar + 16);
     auto bar = [&](int i) { return base + kOffPBar + 8u * i; };
-    if (TAPS > 0 && tid == 0) {
+    if (TAPS > 0 && tid == 480) {
         mbar_init(bar(0), 1);
         mbar_init(bar(1), 1);
         *abort_flag = 0;
@@ -214,9 +274,9 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
 #pragma unroll
         for (int i = 0; i < 4; ++i) z[i] = load4(za + min(t0 + i, left - 1) * (sh.heads * sh.dp));
     }
-    for (int i = tid; i < 64 * kLd / 4; i += kPrepThreads) reinterpret_cast<float4*>(AM)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (tid < (int)kTile / 16) reinterpret_cast<uint4*>(sm + kOffM)[tid] = make_uint4(0u, 0u, 0u, 0u);
-    if (tid < 64) s_beta[tid] = tid < left ? sigmoidc(A.b[(size_t)(sq.row0 + tok0 + tid) * sh.heads + h]) : 0.f;
+    if (tid >= 384 && tid < 448) s_beta[tid - 384] = tid - 384 < left ? sigmoidc(A.b[(size_t)(sq.row0 + tok0 + tid - 384) * sh.heads + h]) : 0.f;
+    if (tid < 16 * kAdP) reinterpret_cast<float4*>(AD)[tid] = make_float4(0.f, 0.f, 0.f, 0.f);
+    reinterpret_cast<uint4*>(sm + kOffM)[tid] = make_uint4(0u, 0u, 0u, 0u);
 
     uint32_t qh[4][2], kh[4][2];                                    // unit vectors, fp16 pairs
     float g[4][4];                                                  // decays of the four tokens
@@ -324,7 +384,7 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
         const uint32_t codes = at < 8 ? 0x40EDC984u : 0xFEDCA985u;
         const int p = (int)(codes >> (4 * (at & 7))) & 15, t = t0 + (p >> 2), s = t0 + (p & 3);
         if (ND == 1 || !(lane & 1)) {
-            if (at < 6) AM[t * kLd + s] = s_beta[t] * acc[0];
+            if (at < 6) AD[t * kAdP + (s & 15)] = s_beta[t] * acc[0];
             else *reinterpret_cast<__half*>(sm + kOffM + sw(t, s >> 3) + 2 * (s & 7)) = __float2half_rn(acc[0]);
         }
     }
@@ -381,9 +441,12 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
     __syncthreads();
     auto a_addr = [&](uint32_t off, int row) { return base + off + ((row + (lane & 15)) * kP + (lane >> 4) * 8) * 2; };
     auto b_addr = [&](uint32_t off, int row) { return base + off + ((row + (lane & 7)) * kP + ((lane >> 3) & 1) * 8) * 2; };
-    auto put2 = [&](bool q, int t, int s, float x, float y) {       // entries (t, s), (t, s + 1) of M or A
-        if (q) *reinterpret_cast<uint32_t*>(sm + kOffM + sw(t, s >> 3) + 2 * (s & 7)) = pack_half2(x, y);
-        else *reinterpret_cast<float2*>(AM + t * kLd + s) = make_float2(s_beta[t] * x, s_beta[t] * y);
+    auto put2 = [&](uint32_t off, int t, int s, float x, float y) {  // entries (t, s), (t, s + 1) of a swizzled tile
+        *reinterpret_cast<uint32_t*>(sm + off + sw(t, s >> 3) + 2 * (s & 7)) = pack_half2(x, y);
+    };
+    auto put_group = [&](bool q, int t, int s, float x, float y) {   // of M or a diagonal block of A
+        if (q) put2(kOffM, t, s, x, y);
+        else *reinterpret_cast<float2*>(AD + t * kAdP + (s & 15)) = make_float2(s_beta[t] * x, s_beta[t] * y);
     };
     auto product = [&](uint32_t aa, uint32_t ba, float (&d)[4]) {   // 16 rows x 8 columns over all channels
         d[0] = d[1] = d[2] = d[3] = 0.f;
@@ -402,8 +465,8 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
         float d[4];
         product(a_addr(q ? kOffQA : kOffKA, 16 * b), b_addr(kOffCOL, 24 * b + 8 * n), d);
         const int c = 8 * n + 2 * t4, i = c < 4 ? 1 : c < 12 ? 2 : 3, s = 16 * b + c - (i == 1 ? 0 : i == 2 ? 4 : 12);
-        if ((g4 >> 2) == i) put2(q, 16 * b + g4, s, d[0], d[1]);
-        if (((g4 + 8) >> 2) == i) put2(q, 16 * b + g4 + 8, s, d[2], d[3]);
+        if ((g4 >> 2) == i) put_group(q, 16 * b + g4, s, d[0], d[1]);
+        if (((g4 + 8) >> 2) == i) put_group(q, 16 * b + g4 + 8, s, d[2], d[3]);
     }
     __syncthreads();
     if (act) {
@@ -429,8 +492,9 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
         const int v = u >> 1, I = v < 2 ? 1 : v < 6 ? 2 : 3, n = v - (I == 1 ? 0 : I == 2 ? 2 : 6);
         float d[4];
         product(a_addr(q ? kOffQA : kOffKA, 16 * I), b_addr(kOffCOL, (I == 1 ? 0 : I == 2 ? 16 : 48) + 8 * n), d);
-        put2(q, 16 * I + g4, 8 * n + 2 * t4, d[0], d[1]);
-        put2(q, 16 * I + g4 + 8, 8 * n + 2 * t4, d[2], d[3]);
+        const float f0 = q ? 1.f : s_beta[16 * I + g4], f1 = q ? 1.f : s_beta[16 * I + g4 + 8];
+        put2(q ? kOffM : kOffAT, 16 * I + g4, 8 * n + 2 * t4, d[0] * f0, d[1] * f0);
+        put2(q ? kOffM : kOffAT, 16 * I + g4 + 8, 8 * n + 2 * t4, d[2] * f1, d[3] * f1);
     }
     fence_proxy_async_smem();
     __syncthreads();
@@ -463,12 +527,12 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
             for (int e = 0; e < 4; ++e) *reinterpret_cast<uint2*>(sm + kOffKB + ((t + e) * kVP + vc) * 2) = r[e];
         }
     };
-    if (warp < 8) {   // ---- T = (I + A)^-1 over the column copies ----
-        if (tid < 64) invert_diagonal(AM, TF, tid);
+    if (warp < 8) {   // ---- T = (I + A)^-1, over the column copies ----
+        if (tid < 64) invert_blocks(sm, s_beta, tid);
         sync_half(0);
-        if (warp < 6) scale_blocks(AM, TF, warp, lane);
-        sync_half(0);
-        solve_columns(AM, TF, warp, lane);
+        if (warp == 0) solve_block_column<0>(sm, base, s_beta, lane);
+        else if (warp == 1) solve_block_column<1>(sm, base, s_beta, lane);
+        else if (warp == 2) solve_block_column<2>(sm, base, s_beta, lane);
     } else {          // ---- meanwhile M goes out and the first values come in ----
         if (tid == 256) {
             if constexpr (TAPS > 0) fetch_values(0);
@@ -483,15 +547,6 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
         for (int i = 0; i < 4; ++i) *piece(kOffKA, t0 + i) = scaled(*piece(kOffKA, t0 + i), f);
     }
     __syncthreads();
-    {   // T diag(beta) as a swizzled fp16 tile over A, eight entries per thread; blocks above the diagonal are never read
-        const int i = tid >> 3, p = tid & 7, s = 8 * p;
-        if ((p >> 1) <= i >> 4) {
-            const float4 a = load4(TF + i * kLd + s), b = load4(TF + i * kLd + s + 4), c = load4(s_beta + s), d = load4(s_beta + s + 4);
-            *reinterpret_cast<uint4*>(sm + kOffAM + sw(i, p)) = make_uint4(pack_half2(a.x * c.x, a.y * c.y), pack_half2(a.z * c.z, a.w * c.w),
-                                                                          pack_half2(b.x * d.x, b.y * d.y), pack_half2(b.z * d.z, b.w * d.w));
-        }
-    }
-    __syncthreads();
     {   // ---- W = (T diag(beta)) (e^G K): 16 rows x 16 ND columns per warp ----
         const int i = warp >> 2, c0 = (warp & 3) * 16 * ND;
         float d[2 * ND][4];
@@ -499,7 +554,7 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
         for (int n = 0; n < 2 * ND; ++n) d[n][0] = d[n][1] = d[n][2] = d[n][3] = 0.f;
         for (int k = 0; k <= i; ++k) {
             uint32_t a[4];
-            ldm4(a, base + kOffAM + sw(16 * i + (lane & 15), 2 * k + (lane >> 4)));
+            ldm4(a, base + kOffCOL + sw(16 * i + (lane & 15), 2 * k + (lane >> 4)));
             const uint32_t ka = base + kOffKA + ((16 * k + (lane & 15)) * kP + c0 + (lane >> 4) * 8) * 2;
 #pragma unroll
             for (int n = 0; n < 2 * ND; n += 2) {
@@ -537,7 +592,7 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
 #pragma unroll
             for (int k = 0; k <= n >> 1; ++k) {
                 uint32_t b0, b1;
-                ldm2(b0, b1, base + kOffAM + sw(8 * n + (lane & 7), 2 * k + ((lane >> 3) & 1)));
+                ldm2(b0, b1, base + kOffCOL + sw(8 * n + (lane & 7), 2 * k + ((lane >> 3) & 1)));
                 mma_16816(d, a[k][0], a[k][1], a[k][2], a[k][3], b0, b1);
             }
             *reinterpret_cast<uint32_t*>(sm + kOffKA + sw(16 * mt + g4, n) + 4 * t4) = pack_half2(d[0], d[1]);
@@ -557,7 +612,7 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
         load_values(tile + 1, tid, kPrepThreads, -1);
         __syncthreads();
     }
-    if (tid == 0 || tid == 256) bulk_wait_group0();
+    if (tid == 0 || tid == 256) bulk_wait_group_read0();            // shared memory may go
     if (TAPS > 0 && tid == 0 && *abort_flag) atomicExch(A.error, 11);
 }
 
