@@ -26,10 +26,9 @@ constexpr int kDC = 64;
 constexpr uint32_t kTile = kDC * 128;                  // 64 rows of 64 fp16, 128-byte swizzle
 constexpr float kDL2e = 1.4426950408889634f;
 
-// An item (chunk and head) of the scratch: W | e^G Q | e^{G_C - G} K (ND tiles each) | M | e^{G_C} | U' per state tile (NV tiles of [64 values][64 tokens])
+// An item (chunk and head) of the scratch: W | e^G Q | e^{G_C - G} K (nd tiles each) | M | e^{G_C} | U' per state tile (nv tiles of [64 values][64 tokens])
 struct DeltaItem {
     int nd, nv, n_vt;
-    __host__ __device__ uint32_t off_q() const { return nd * kTile; }
     __host__ __device__ uint32_t off_k() const { return 2 * nd * kTile; }
     __host__ __device__ uint32_t off_m() const { return 3 * nd * kTile; }
     __host__ __device__ uint32_t off_e() const { return off_m() + kTile; }
@@ -237,7 +236,7 @@ __device__ __forceinline__ void sync_half(int which) { asm volatile("bar.sync %0
 template <int ND, int TAPS>
 __global__ void __launch_bounds__(kPrepThreads, 2)
 delta_prep_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const DeltaChunkArgs A) {
-    extern __shared__ __align__(128) unsigned char sm[];
+    extern __shared__ __align__(1024) unsigned char sm[];
     constexpr int DK = 64 * ND, LN = 16 * ND, kP = DK + 8;         // channels, lanes per token, row pitch in halves
     const DeltaShape& sh = A.sh;
     const LaSeqMeta sq = A.seqs[blockIdx.z];

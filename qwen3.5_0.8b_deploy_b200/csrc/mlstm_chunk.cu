@@ -320,30 +320,31 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap map, const MlstmShape sh,
                     *p = make_uint4(hi[0], hi[1], hi[2], hi[3]);
                     *reinterpret_cast<uint4*>(reinterpret_cast<unsigned char*>(p) + (kMOffKlo - kMOffK)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
                 }
-                if constexpr (!kGated) continue;
-                // eight sums over 32 lanes: halve the values while halving the lanes, lane groups of four end with one column each
+                if constexpr (kGated) {
+                    // eight sums over 32 lanes: halve the values while halving the lanes, lane groups of four end with one column each
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const bool top = lane & 16;
-                    const float x = __shfl_xor_sync(0xffffffffu, top ? cs[e] : cs[e + 4], 16);
-                    cs[e] = (top ? cs[e + 4] : cs[e]) + x;
-                }
+                    for (int e = 0; e < 4; ++e) {
+                        const bool top = lane & 16;
+                        const float x = __shfl_xor_sync(0xffffffffu, top ? cs[e] : cs[e + 4], 16);
+                        cs[e] = (top ? cs[e + 4] : cs[e]) + x;
+                    }
 #pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    const bool top = lane & 8;
-                    const float x = __shfl_xor_sync(0xffffffffu, top ? cs[e] : cs[e + 2], 8);
-                    cs[e] = (top ? cs[e + 2] : cs[e]) + x;
-                }
-                {
-                    const bool top = lane & 4;
-                    const float x = __shfl_xor_sync(0xffffffffu, top ? cs[0] : cs[1], 4);
-                    cs[0] = (top ? cs[1] : cs[0]) + x;
-                }
-                cs[0] += __shfl_xor_sync(0xffffffffu, cs[0], 2);
-                cs[0] += __shfl_xor_sync(0xffffffffu, cs[0], 1);
-                if ((lane & 3) == 0) {
-                    const int d = oct * 8 + ((lane & 16) ? 4 : 0) + ((lane & 8) ? 2 : 0) + ((lane & 4) ? 1 : 0);
-                    s_n(par ^ 1)[d] = keep * s_n(par)[d] + cs[0];
+                    for (int e = 0; e < 2; ++e) {
+                        const bool top = lane & 8;
+                        const float x = __shfl_xor_sync(0xffffffffu, top ? cs[e] : cs[e + 2], 8);
+                        cs[e] = (top ? cs[e + 2] : cs[e]) + x;
+                    }
+                    {
+                        const bool top = lane & 4;
+                        const float x = __shfl_xor_sync(0xffffffffu, top ? cs[0] : cs[1], 4);
+                        cs[0] = (top ? cs[1] : cs[0]) + x;
+                    }
+                    cs[0] += __shfl_xor_sync(0xffffffffu, cs[0], 2);
+                    cs[0] += __shfl_xor_sync(0xffffffffu, cs[0], 1);
+                    if ((lane & 3) == 0) {
+                        const int d = oct * 8 + ((lane & 16) ? 4 : 0) + ((lane & 8) ? 2 : 0) + ((lane & 4) ? 1 : 0);
+                        s_n(par ^ 1)[d] = keep * s_n(par)[d] + cs[0];
+                    }
                 }
             }
             // ---- the state decays to the chunk's end ----
